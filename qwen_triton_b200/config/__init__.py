@@ -4,6 +4,7 @@ from .lederax import LederaxConfig
 from .vunepel import VunepelConfig
 from .bisodra import BisodraConfig
 from .regupel import RegupelConfig
+from .misudra import MisudraConfig
 from .registry import (
     config_from_dict,
     load_config,
@@ -19,9 +20,10 @@ register_architecture("Lederax", LederaxConfig)
 register_architecture("Vunepel", VunepelConfig)
 register_architecture("Bisodra", BisodraConfig)
 register_architecture("Regupel", RegupelConfig)
+register_architecture("Misudra", MisudraConfig)
 
 __all__ = [
-    "BisodraConfig", "ConfigError", "LayerCall", "LayerSpec", "LederaxConfig", "ModelSpec", "PartSpec", "Qwen3Config", "RegupelConfig", "VunepelConfig",
+    "BisodraConfig", "ConfigError", "LayerCall", "LayerSpec", "LederaxConfig", "MisudraConfig", "ModelSpec", "PartSpec", "Qwen3Config", "RegupelConfig", "VunepelConfig",
     "config_from_dict", "load_config", "load_config_dict", "load_preset", "preset_names",
     "register_architecture", "registered_architectures",
 ]

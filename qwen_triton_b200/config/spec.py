@@ -12,7 +12,8 @@ The spec is plain data:
   their sizes and constants as parameters;
 * ``schedule``: the order in which layers run.  It is a list of
   :class:`LayerCall`, so a layer may be named twice, and a call may read the
-  cache that an earlier call wrote instead of owning one.
+  cache that an earlier call wrote instead of owning one, or have the stream
+  rewritten in front of it by one of ``entries``.
 """
 from __future__ import annotations
 
@@ -65,10 +66,14 @@ class LayerCall:
                    mixer asks for one).  An integer ``j``: this call reads the
                    cache entry that schedule position ``j`` (earlier) owns and
                    writes nothing.
+    ``entry``      ``None``, or an index into ``ModelSpec.entries``: that part
+                   rewrites the residual stream right before this call (a pass
+                   of a looped range that starts from a map of the stream).
     """
 
     layer: int
     cache_of: int | None = None
+    entry: int | None = None
 
 
 @dataclass(frozen=True)
@@ -83,6 +88,7 @@ class ModelSpec:
     head: PartSpec
     max_positions: int
     eos_token_ids: tuple[int, ...] = ()
+    entries: Sequence[PartSpec] = ()       # stream maps that calls of the schedule name (``LayerCall.entry``)
 
     def validate(self) -> None:
         if self.vocab_size <= 0 or self.hidden_size <= 0:
@@ -92,6 +98,8 @@ class ModelSpec:
         for pos, call in enumerate(self.schedule):
             if not 0 <= call.layer < len(self.layers):
                 raise ValueError(f"schedule[{pos}] names layer {call.layer}, but there are {len(self.layers)} layers")
+            if call.entry is not None and not 0 <= call.entry < len(self.entries):
+                raise ValueError(f"schedule[{pos}] names stream map {call.entry}, but there are {len(self.entries)}")
             if call.cache_of is not None:
                 if not 0 <= call.cache_of < pos:
                     raise ValueError(f"schedule[{pos}] reads the cache of position {call.cache_of}, which does not run earlier")

@@ -15,7 +15,9 @@
 // the other decode kernels use.  (Where a page's keys are cut among the row groups, see the kernel, both warps of a row
 // group still form the same scores.)
 //
-// Causal: the key at position j is visible to the query at position i iff j <= i.  Takes rows and ranks that are
+// Causal: the key at position j is visible to the query at position i iff j <= i and, under a window, i - j < window; a
+// block's walk then starts at the page of the first key its first row sees, and with `ring_tokens` > 0 (a multiple of the
+// page) position p sits at element p % ring_tokens of the sequence's pages.  Takes rows and ranks that are
 // multiples of 8 (shared-memory rows are padded with zeros to the next multiple of 16), ranks up to 512, a positive
 // scale and pages of 64 tokens; the generic kernels of attention.cu take everything else.
 #include "attention_mma.cuh"
@@ -33,6 +35,7 @@ struct LatentParams {
     const int* seq_start; const int* seq_past;   // prompts: packed sequences with a past (seq_len null)
     const int* seq_len;                          // one-token steps: keys each sequence sees, its own included
     int heads, row, rank;
+    int window, ring_tokens;                     // 0: every earlier key; 0: positions in order
     float scale;
     int n_splits; float* part_acc; float* part_ml;
 };
@@ -85,9 +88,11 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_attention_kernel(const L
         for (int i = tid; i < (int)(3u * tile_bytes / 16u); i += LT_THREADS) reinterpret_cast<uint4*>(smem_raw)[i] = make_uint4(0, 0, 0, 0);
         __syncthreads();
     }
-    const int n_tiles = p_last >= 0 ? p_last / PAGE + 1 : 0;
-    const int per = (n_tiles + p.n_splits - 1) / p.n_splits;
-    const int tile_begin = min(n_tiles, split * per), tile_end = min(n_tiles, tile_begin + per);
+    const int last_tile = p_last >= 0 ? p_last / PAGE + 1 : 0;
+    const int first_tile = p.window > 0 ? min(last_tile, max(0, past + q0 / heads - p.window + 1) / PAGE) : 0;
+    const int per = (last_tile - first_tile + p.n_splits - 1) / p.n_splits;
+    const int tile_begin = min(last_tile, first_tile + split * per), tile_end = min(last_tile, tile_begin + per);
+    const int ring_pages = p.ring_tokens / PAGE;
 
     {
         const int chunks = row >> 3;
@@ -100,7 +105,8 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_attention_kernel(const L
         }
     }
     auto issue = [&](int tile) {
-        if (tile < tile_end) copy_page(kv0 + (uint32_t)((tile - tile_begin) & 1) * tile_bytes, p.cache + (size_t)table[tile] * PAGE * row, row, lds, tid);
+        if (tile < tile_end) copy_page(kv0 + (uint32_t)((tile - tile_begin) & 1) * tile_bytes, p.cache + (size_t)table[ring_pages ? tile % ring_pages : tile] * PAGE * row, row,
+                                         lds, tid);
         cp_async_commit();
     };
     issue(tile_begin);
@@ -118,6 +124,9 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_attention_kernel(const L
     const int last_row = q0 + rows - 1;
     const int qpos[2] = {past + min(q0 + rg * 16 + g, last_row) / heads, past + min(q0 + rg * 16 + g + 8, last_row) / heads};
     const int warp_pos_min = past + min(q0 + rg * 16, last_row) / heads, warp_pos_max = past + min(q0 + rg * 16 + 15, last_row) / heads;
+    // of the keys at and above a warp's first position, those below `low_min` are hidden from its first row, and a page wholly below from all
+    const int low_min = p.window > 0 ? warp_pos_min - p.window + 1 : -1, low_max = p.window > 0 ? warp_pos_max - p.window + 1 : -1;
+    const int low[2] = {p.window > 0 ? qpos[0] - p.window + 1 : -1, p.window > 0 ? qpos[1] - p.window + 1 : -1};
     const uint32_t q_frag = q_s + (uint32_t)((rg * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * lds + (lane >> 4) * 8) * 2u;
     const int mi = lane >> 3;
     const uint32_t k_frag = (uint32_t)((kb + (mi >> 1) * 8 + (lane & 7)) * lds + (mi & 1) * 8) * 2u;
@@ -140,7 +149,7 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_attention_kernel(const L
         if constexpr (KP == 1) {
             // The two warps of a row group form the scores of 32 keys each and hand each other the row maxima (through
             // the padding behind the rows of the query tile) and the weights (through p_s), so no score is formed twice.
-            if (active && pos0 <= warp_pos_max) {
+            if (active && pos0 <= warp_pos_max && pos0 + PAGE > low_min) {
                 const int kc = cg * 32;
                 float s[4][4];
 #pragma unroll
@@ -157,12 +166,14 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_attention_kernel(const L
                         mma_bf16(s[2 * np + 1], a, b[2], b[3]);
                     }
                 }
-                if (pos0 + PAGE - 1 > warp_pos_min) {
+                if (pos0 + PAGE - 1 > warp_pos_min || pos0 < low_max) {
 #pragma unroll
                     for (int nt = 0; nt < 4; ++nt)
 #pragma unroll
-                        for (int e = 0; e < 4; ++e)
-                            if (pos0 + kc + nt * 8 + 2 * t + (e & 1) > qpos[e >> 1]) s[nt][e] = -INFINITY;
+                        for (int e = 0; e < 4; ++e) {
+                            const int key = pos0 + kc + nt * 8 + 2 * t + (e & 1);
+                            if (key > qpos[e >> 1] || key < low[e >> 1]) s[nt][e] = -INFINITY;
+                        }
                 }
                 float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -218,7 +229,7 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_attention_kernel(const L
                     }
                 }
             }
-        } else if (active && pos0 <= warp_pos_max) {
+        } else if (active && pos0 <= warp_pos_max && pos0 + KEYS > low_min) {
             float s[SNT][4];
 #pragma unroll
             for (int i = 0; i < SNT; ++i) { s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f; }
@@ -234,12 +245,14 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_attention_kernel(const L
                     mma_bf16(s[2 * np + 1], a, b[2], b[3]);
                 }
             }
-            if (pos0 + KEYS - 1 > warp_pos_min) {
+            if (pos0 + KEYS - 1 > warp_pos_min || pos0 < low_max) {
 #pragma unroll
                 for (int nt = 0; nt < SNT; ++nt)
 #pragma unroll
-                    for (int e = 0; e < 4; ++e)
-                        if (pos0 + nt * 8 + 2 * t + (e & 1) > qpos[e >> 1]) s[nt][e] = -INFINITY;
+                    for (int e = 0; e < 4; ++e) {
+                        const int key = pos0 + nt * 8 + 2 * t + (e & 1);
+                        if (key > qpos[e >> 1] || key < low[e >> 1]) s[nt][e] = -INFINITY;
+                    }
             }
             float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -335,13 +348,15 @@ int raise_smem(K kernel, size_t bytes, const char* name) {
 // (seq_len given: one query token per sequence).
 extern "C" int qt_attention_latent(const void* q, const void* cache, void* out, const int* block_table, int max_blocks,
                                    const int* seq_start, const int* seq_past, const int* seq_len, int n_seqs, int max_q_len,
-                                   int heads, int row, int rank, int page_tokens, float scale, int n_splits, float* part_acc,
-                                   float* part_ml, void* stream) {
+                                   int heads, int row, int rank, int page_tokens, int window, int ring_tokens, float scale, int n_splits,
+                                   float* part_acc, float* part_ml, void* stream) {
     if (n_seqs == 0 || max_q_len == 0) return QT_OK;
     QT_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && heads > 0, "attention_latent: %d sequences, %d heads", n_seqs, heads);
     QT_REQUIRE(row >= 8 && row % 8 == 0 && rank >= 8 && rank % 8 == 0 && rank <= row && rank <= 512,
                "attention_latent: rows of %d with %d value elements (multiples of 8, values up to 512; use the generic kernel)", row, rank);
     QT_REQUIRE(page_tokens == PAGE, "attention_latent: pages of %d tokens (this kernel walks pages of %d)", page_tokens, PAGE);
+    QT_REQUIRE(window >= 0 && ring_tokens >= 0 && ring_tokens % PAGE == 0 && (ring_tokens == 0 || window > 0),
+               "attention_latent: a window of %d in a ring of %d tokens", window, ring_tokens);
     QT_REQUIRE(scale > 0.f, "attention_latent: the score scale must be positive (the row maximum is taken before scaling)");
     QT_REQUIRE((seq_len != nullptr) != (seq_start != nullptr && seq_past != nullptr), "attention_latent: either seq_len or seq_start and seq_past");
     QT_REQUIRE(n_splits >= 1 && n_splits <= 65535 && (n_splits == 1 || (part_acc && part_ml)), "attention_latent: %d key ranges need scratch memory", n_splits);
@@ -353,7 +368,7 @@ extern "C" int qt_attention_latent(const void* q, const void* cache, void* out, 
     const size_t smem = (size_t)3 * PAGE * lds * 2 + (size_t)4 * 16 * PAGE * 2;      // three tiles and the row groups' weights
     QT_REQUIRE(smem <= 227 * 1024, "attention_latent: rows of %d elements do not fit shared memory (use the generic kernel)", row);
     LatentParams p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, block_table, max_blocks, seq_start, seq_past,
-                   seq_len, heads, row, rank, scale, n_splits / kp, part_acc, part_ml};
+                   seq_len, heads, row, rank, window, ring_tokens, scale, n_splits / kp, part_acc, part_ml};
     const long long most_rows = (long long)(seq_len ? 1 : max_q_len) * heads;
     dim3 grid((unsigned)((most_rows + block_rows - 1) / block_rows), n_splits / kp, n_seqs);
     cudaStream_t s = (cudaStream_t)stream;

@@ -136,12 +136,19 @@ __global__ void conv_keep_kernel(const float* __restrict__ proj, int n_splits, s
 
 // out[t, n] = f(sum_r w[r, n] x[t, r] + bias[n]) for a tile of LR_TOKENS tokens and 256 outputs per block.
 constexpr int LR_TOKENS = 16;
-constexpr int LR_DECAY = 0, LR_SIGMOID = 1;
+constexpr int LR_DECAY = 0, LR_SIGMOID = 1, LR_LOG_SIGMOID = 2;
+
+// f of a narrow projection: a decay's logarithm -rate softplus(z), sigmoid(z), or rate * log(sigmoid(z)) (the logarithm of a
+// decay that is a power of a sigmoid).
+template <int MODE>
+__device__ __forceinline__ float lowrank_value(float z, float rate) {
+    return MODE == LR_SIGMOID ? sigmoidf(z) : -rate * softplusf(MODE == LR_DECAY ? z : -z);
+}
 
 template <int MODE>
 __global__ void __launch_bounds__(256) lowrank_kernel(const float* __restrict__ proj, int n_splits, size_t split_stride, int proj_cols,
                                                       int x_offset, int rank, const float* __restrict__ w, const float* __restrict__ bias,
-                                                      const float* __restrict__ rate_log, int per_rate, float* __restrict__ out,
+                                                      const float* __restrict__ rate_log, int per_rate, float power, float* __restrict__ out,
                                                       int n_tokens, int n_out) {
     pdl_launch_dependents();
     pdl_wait();
@@ -175,12 +182,12 @@ __global__ void __launch_bounds__(256) lowrank_kernel(const float* __restrict__ 
         }
     }
     const float b = bias ? bias[n] : 0.f;
-    const float rate = MODE == LR_DECAY ? expf(rate_log[n / per_rate]) : 0.f;
+    const float rate = MODE == LR_DECAY ? expf(rate_log[n / per_rate]) : power;
 #pragma unroll
     for (int tt = 0; tt < LR_TOKENS; ++tt) {
         if (tt >= count) break;
         const float z = acc[tt] + b;
-        out[(size_t)(t0 + tt) * n_out + n] = MODE == LR_DECAY ? -rate * softplusf(z) : sigmoidf(z);     // the decay's logarithm
+        out[(size_t)(t0 + tt) * n_out + n] = lowrank_value<MODE>(z, rate);
     }
 }
 
@@ -189,7 +196,7 @@ __global__ void __launch_bounds__(256) lowrank_kernel(const float* __restrict__ 
 template <int MODE>
 __global__ void __launch_bounds__(256) lowrank_few_kernel(const float* __restrict__ proj, int n_splits, size_t split_stride, int proj_cols,
                                                           int x_offset, int rank, const float* __restrict__ w, const float* __restrict__ bias,
-                                                          const float* __restrict__ rate_log, int per_rate, float* __restrict__ out,
+                                                          const float* __restrict__ rate_log, int per_rate, float power, float* __restrict__ out,
                                                           int n_tokens, int n_out) {
     pdl_launch_dependents();
     pdl_wait();
@@ -228,11 +235,11 @@ __global__ void __launch_bounds__(256) lowrank_few_kernel(const float* __restric
     __syncthreads();
     if (n >= n_out) return;
     const float b = bias ? bias[n] : 0.f;
-    const float rate = MODE == LR_DECAY ? expf(rate_log[n / per_rate]) : 0.f;
+    const float rate = MODE == LR_DECAY ? expf(rate_log[n / per_rate]) : power;
     for (int tt = slice; tt < n_tokens; tt += 4) {                 // the four ranges' sums in their order
         const float z = part[(0 * LR_TOKENS + tt) * 64 + local] + part[(1 * LR_TOKENS + tt) * 64 + local] +
                         part[(2 * LR_TOKENS + tt) * 64 + local] + part[(3 * LR_TOKENS + tt) * 64 + local] + b;
-        out[(size_t)tt * n_out + n] = MODE == LR_DECAY ? -rate * softplusf(z) : sigmoidf(z);
+        out[(size_t)tt * n_out + n] = lowrank_value<MODE>(z, rate);
     }
 }
 
@@ -817,40 +824,34 @@ extern "C" int qt_delta_prepare(const float* proj, int n_splits, long long split
     return QT_OK;
 }
 
+template <int MODE>
+static int launch_lowrank(const float* proj, int n_splits, size_t split_stride, int proj_cols, int x_offset, int rank, const float* w, const float* bias,
+                          const float* rate_log, int per_rate, float power, float* out, int n_tokens, int n_out, cudaStream_t s) {
+    const size_t few_smem = ((size_t)LR_TOKENS * rank + 4 * LR_TOKENS * 64) * sizeof(float);
+    const unsigned tiles = (unsigned)((n_tokens + LR_TOKENS - 1) / LR_TOKENS);
+    if (n_tokens <= 16 * LR_TOKENS && few_smem <= 48 * 1024)
+        launch_kernel(lowrank_few_kernel<MODE>, dim3((n_out + 63) / 64, tiles), dim3(256), few_smem, s, proj, n_splits, split_stride, proj_cols, x_offset, rank, w,
+                      bias, rate_log, per_rate, power, out, n_tokens, n_out);
+    else
+        launch_kernel(lowrank_kernel<MODE>, dim3((n_out + 255) / 256, tiles), dim3(256), (size_t)LR_TOKENS * rank * sizeof(float), s, proj, n_splits,
+                      split_stride, proj_cols, x_offset, rank, w, bias, rate_log, per_rate, power, out, n_tokens, n_out);
+    QT_CHECK_LAUNCH("lowrank");
+    return QT_OK;
+}
+
 extern "C" int qt_lowrank(const float* proj, int n_splits, long long split_stride, int proj_cols, int x_offset, int rank,
-                          const float* w, const float* bias, const float* rate_log, int per_rate, float* out, int n_tokens,
+                          const float* w, const float* bias, const float* rate_log, int per_rate, float power, float* out, int n_tokens,
                           int n_out, int mode, void* stream) {
     QT_REQUIRE(n_tokens >= 0 && n_out > 0 && rank > 0 && x_offset >= 0 && x_offset + rank <= proj_cols && n_splits >= 1,
                "lowrank: bad sizes T=%d N=%d rank=%d at column %d of %d", n_tokens, n_out, rank, x_offset, proj_cols);
-    QT_REQUIRE(mode == LR_SIGMOID || (mode == LR_DECAY && rate_log && per_rate > 0), "lowrank: mode %d", mode);
+    QT_REQUIRE(mode == LR_SIGMOID || mode == LR_LOG_SIGMOID || (mode == LR_DECAY && rate_log && per_rate > 0), "lowrank: mode %d", mode);
     QT_REQUIRE((size_t)LR_TOKENS * rank * sizeof(float) <= 48 * 1024, "lowrank: %d columns are too many for a tile in shared memory", rank);
     if (n_tokens == 0) return QT_OK;
     cudaStream_t s = (cudaStream_t)stream;
-    if (n_tokens <= 16 * LR_TOKENS) {
-        const size_t few_smem = ((size_t)LR_TOKENS * rank + 4 * LR_TOKENS * 64) * sizeof(float);
-        if (few_smem <= 48 * 1024) {
-            const dim3 few_grid((n_out + 63) / 64, (n_tokens + LR_TOKENS - 1) / LR_TOKENS);
-            if (mode == LR_DECAY)
-                launch_kernel(lowrank_few_kernel<LR_DECAY>, few_grid, dim3(256), few_smem, s, proj, n_splits, (size_t)split_stride, proj_cols, x_offset,
-                              rank, w, bias, rate_log, per_rate, out, n_tokens, n_out);
-            else
-                launch_kernel(lowrank_few_kernel<LR_SIGMOID>, few_grid, dim3(256), few_smem, s, proj, n_splits, (size_t)split_stride, proj_cols, x_offset,
-                              rank, w, bias, rate_log, per_rate, out, n_tokens, n_out);
-            QT_CHECK_LAUNCH("lowrank");
-            return QT_OK;
-        }
-    }
-    const int threads = 256;
-    const dim3 grid((n_out + threads - 1) / threads, (n_tokens + LR_TOKENS - 1) / LR_TOKENS);
-    const size_t smem = (size_t)LR_TOKENS * rank * sizeof(float);
-    if (mode == LR_DECAY)
-        launch_kernel(lowrank_kernel<LR_DECAY>, grid, dim3(threads), smem, s, proj, n_splits, (size_t)split_stride, proj_cols, x_offset, rank, w, bias,
-                      rate_log, per_rate, out, n_tokens, n_out);
-    else
-        launch_kernel(lowrank_kernel<LR_SIGMOID>, grid, dim3(threads), smem, s, proj, n_splits, (size_t)split_stride, proj_cols, x_offset, rank, w, bias,
-                      rate_log, per_rate, out, n_tokens, n_out);
-    QT_CHECK_LAUNCH("lowrank");
-    return QT_OK;
+    const size_t stride = (size_t)split_stride;
+    if (mode == LR_DECAY) return launch_lowrank<LR_DECAY>(proj, n_splits, stride, proj_cols, x_offset, rank, w, bias, rate_log, per_rate, power, out, n_tokens, n_out, s);
+    if (mode == LR_SIGMOID) return launch_lowrank<LR_SIGMOID>(proj, n_splits, stride, proj_cols, x_offset, rank, w, bias, rate_log, per_rate, power, out, n_tokens, n_out, s);
+    return launch_lowrank<LR_LOG_SIGMOID>(proj, n_splits, stride, proj_cols, x_offset, rank, w, bias, rate_log, per_rate, power, out, n_tokens, n_out, s);
 }
 
 template <int R>

@@ -24,15 +24,83 @@ __global__ void embedding_kernel(float* __restrict__ residual, const T* __restri
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) out[i] = valid ? to_float(row[i]) * scale : 0.f;
 }
 
+// The same with an RMS norm behind the gather: residual[t, :] = x / sqrt(mean(x^2) + eps) * norm_w for the scaled row x.
+// `start` (or null) takes a copy of the result in the table's type: the embedding's output, for a model whose layers
+// meet it again.  One block per token; a row is read twice (from L1 the second time).
+template <typename T>
+__global__ void embedding_norm_kernel(float* __restrict__ residual, const T* __restrict__ table, const int* __restrict__ ids, int hidden,
+                                      int vocab, float scale, const float* __restrict__ norm_w, float eps, T* __restrict__ start) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float scratch[32];
+    const int t = blockIdx.x;
+    int id = ids[t];
+    const bool valid = id >= 0 && id < vocab;
+    const T* row = table + (size_t)(valid ? id : 0) * hidden;
+    float inv = scale;
+    if (norm_w) {
+        float sq = 0.f;
+        for (int i = threadIdx.x; i < hidden; i += blockDim.x) { const float x = to_float(row[i]) * scale; sq += x * x; }
+        inv = rsqrtf(block_sum(sq, scratch) / (float)hidden + eps) * scale;
+    }
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        const float y = valid ? to_float(row[i]) * inv * (norm_w ? norm_w[i] : 1.f) : 0.f;
+        residual[(size_t)t * hidden + i] = y;
+        if (start) start[(size_t)t * hidden + i] = from_float<T>(y);
+    }
+}
+
 extern "C" int qt_embedding(float* residual, const void* table, const int* ids, int n_tokens, int hidden, int vocab,
-                            int table_dtype, float scale, void* stream) {
+                            int table_dtype, float scale, const float* norm_w, float eps, void* start, void* stream) {
     QT_REQUIRE(n_tokens >= 0 && hidden > 0 && vocab > 0, "embedding: bad sizes T=%d H=%d V=%d", n_tokens, hidden, vocab);
+    QT_REQUIRE(!norm_w || eps > 0.f, "embedding: eps must be positive");
     if (n_tokens == 0) return QT_OK;
     return QT_DISPATCH_DTYPE(table_dtype, "embedding", {
+        if (norm_w || start) {
+            launch_kernel(embedding_norm_kernel<T>, dim3(n_tokens), dim3(256), 0, (cudaStream_t)stream, residual, (const T*)table, ids, hidden, vocab, scale,
+                          norm_w, eps, (T*)start);
+            QT_CHECK_LAUNCH("embedding_norm");
+            return QT_OK;
+        }
         launch_kernel(embedding_kernel<T>, dim3(n_tokens), dim3(256), 0, (cudaStream_t)stream, residual, (const T*)table, ids, hidden, vocab, scale);
         QT_CHECK_LAUNCH("embedding");
         return QT_OK;
     });
+}
+
+// ----------------------------------------------------------------------------- the stream beside the embedding's output
+// out[t] = [x | start[t]] in the activation type, x = residual[t] + sum_s delta[s][t] in float; the stream is then zero:
+// what a map of these rows returns takes its place by the ordinary addition of the next norm.  One block per token.
+template <typename TD, typename TO>
+__global__ void stream_concat_kernel(float* __restrict__ residual, const TD* __restrict__ delta, int n_splits, size_t split_stride,
+                                     const TO* __restrict__ start, TO* __restrict__ out, int hidden) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t at = (size_t)blockIdx.x * hidden, to = 2 * at;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        float x = residual[at + i];
+        if (delta) x += load_sum(delta, at + i, n_splits, split_stride);
+        residual[at + i] = 0.f;
+        out[to + i] = from_float<TO>(x);
+        out[to + hidden + i] = start[at + i];
+    }
+}
+
+extern "C" int qt_stream_concat(float* residual, const void* delta, int delta_dtype, int n_splits, long long split_stride, const void* start,
+                                void* out, int dtype, int n_tokens, int hidden, void* stream) {
+    QT_REQUIRE(n_tokens >= 0 && hidden > 0 && n_splits >= 1, "stream_concat: bad sizes T=%d H=%d splits=%d", n_tokens, hidden, n_splits);
+    if (n_tokens == 0) return QT_OK;
+    cudaStream_t s = (cudaStream_t)stream;
+#define QT_LAUNCH_CONCAT(TD, TO)                                                                                                  \
+    launch_kernel(stream_concat_kernel<TD, TO>, dim3(n_tokens), dim3(256), 0, s, residual, (const TD*)delta, n_splits, (size_t)split_stride, \
+                  (const TO*)start, (TO*)out, hidden)
+    if (delta_dtype == QT_F32 && dtype == QT_F32) QT_LAUNCH_CONCAT(float, float);
+    else if (delta_dtype == QT_F32 && dtype == QT_BF16) QT_LAUNCH_CONCAT(float, __nv_bfloat16);
+    else if (delta_dtype == QT_BF16 && dtype == QT_BF16) QT_LAUNCH_CONCAT(__nv_bfloat16, __nv_bfloat16);
+    else QT_FAIL(QT_ERR_ARG, "stream_concat: element types %d/%d", delta_dtype, dtype);
+#undef QT_LAUNCH_CONCAT
+    QT_CHECK_LAUNCH("stream_concat");
+    return QT_OK;
 }
 
 // ----------------------------------------------------------------------------- bias of a projection
@@ -908,12 +976,13 @@ extern "C" int qt_qkv_treat_write(const void* qkv, int in_dtype, int n_splits, l
 // ----------------------------------------------------------------------------- gated product
 // out[t, i] = act(g) * u (act: SiLU or another of QT_ACT_*); float inside.  Plain layout (group 0): g = gate_up[t, i], u = gate_up[t, inter + i].
 // Interleaved layout (group G, the fused weight's rows alternate G of gate and G of up, which is what lets a GEMM
-// epilogue see both in one warp): g = gate_up[t, (i / G) * 2G + i % G], u = the element G further on.
+// epilogue see both in one warp): g = gate_up[t, (i / G) * 2G + i % G], u = the element G further on.  `bias` (or null)
+// holds a float per column of gate_up, in its layout, added to the sums.
 __device__ __forceinline__ size_t gate_column(int i, int group) { return group ? (size_t)(i / group) * 2 * group + i % group : (size_t)i; }
 
 template <typename TI, typename TO>
-__global__ void swiglu_kernel(const TI* __restrict__ gate_up, int n_splits, size_t split_stride, TO* __restrict__ out,
-                              long long total, int inter, int group, int act, float limit) {
+__global__ void swiglu_kernel(const TI* __restrict__ gate_up, int n_splits, size_t split_stride, const float* __restrict__ bias,
+                              TO* __restrict__ out, long long total, int inter, int group, int act, float limit) {
     pdl_launch_dependents();
     pdl_wait();
     const int up_offset = group ? group : inter;
@@ -922,8 +991,9 @@ __global__ void swiglu_kernel(const TI* __restrict__ gate_up, int n_splits, size
         const long long t = idx / inter;
         const int i = (int)(idx % inter);
         const size_t base = (size_t)t * 2 * inter + gate_column(i, group);
-        const float g = load_sum(gate_up, base, n_splits, split_stride);
-        const float u = load_sum(gate_up, base + up_offset, n_splits, split_stride);
+        float g = load_sum(gate_up, base, n_splits, split_stride);
+        float u = load_sum(gate_up, base + up_offset, n_splits, split_stride);
+        if (bias) { const int at = (int)gate_column(i, group); g += bias[at]; u += bias[at + up_offset]; }
         out[idx] = from_float<TO>(gated_value<false>(g, u, act, limit));
     }
 }
@@ -957,8 +1027,8 @@ template <typename TO> __device__ __forceinline__ float4 silu_mul4(const float4&
 
 // PT chunks per thread, all loads issued before the first store.
 template <typename TI, typename TO, int PT>
-__global__ void swiglu_vec_kernel(const TI* __restrict__ gate_up, int n_splits, size_t split_stride, TO* __restrict__ out,
-                                  int inter, int group, int act, float limit) {
+__global__ void swiglu_vec_kernel(const TI* __restrict__ gate_up, int n_splits, size_t split_stride, const float* __restrict__ bias,
+                                  TO* __restrict__ out, int inter, int group, int act, float limit) {
     pdl_launch_dependents();
     pdl_wait();
     const int chunks = inter >> 3;
@@ -983,6 +1053,17 @@ __global__ void swiglu_vec_kernel(const TI* __restrict__ gate_up, int n_splits, 
                 }
             }
         }
+        if (bias) {
+#pragma unroll
+            for (int i = 0; i < PT; ++i) {
+                const int c = c0 + i * blockDim.x;
+                if (c < chunks) {
+                    const size_t at = gate_column(8 * c, group);
+                    const Float8 bg = load8(bias + at), bu = load8(bias + at + up_offset);
+                    add4(g[i].a, bg.a); add4(g[i].b, bg.b); add4(u[i].a, bu.a); add4(u[i].b, bu.b);
+                }
+            }
+        }
 #pragma unroll
         for (int i = 0; i < PT; ++i) {
             const int c = c0 + i * blockDim.x;
@@ -991,7 +1072,7 @@ __global__ void swiglu_vec_kernel(const TI* __restrict__ gate_up, int n_splits, 
     }
 }
 
-extern "C" int qt_swiglu(const void* gate_up, int in_dtype, int n_splits, long long split_stride, void* out, int out_dtype,
+extern "C" int qt_swiglu(const void* gate_up, int in_dtype, int n_splits, long long split_stride, const float* bias, void* out, int out_dtype,
                          int n_tokens, int inter, int group, int act, float limit, void* stream) {
     QT_REQUIRE(act >= 0 && act <= QT_ACT_CAPPED, "swiglu: unknown activation code %d", act);
     QT_REQUIRE(n_tokens >= 0 && inter > 0 && n_splits >= 1, "swiglu: bad sizes T=%d I=%d", n_tokens, inter);
@@ -1000,7 +1081,8 @@ extern "C" int qt_swiglu(const void* gate_up, int in_dtype, int n_splits, long l
     const long long total = (long long)n_tokens * inter;
     const int threads = 256;
     cudaStream_t s = (cudaStream_t)stream;
-    const bool vec = inter % 8 == 0 && group % 8 == 0 && split_stride % 8 == 0 && ((uintptr_t)gate_up % 16 == 0) && ((uintptr_t)out % 16 == 0);
+    const bool vec = inter % 8 == 0 && group % 8 == 0 && split_stride % 8 == 0 && ((uintptr_t)gate_up % 16 == 0) && ((uintptr_t)out % 16 == 0) &&
+                     ((uintptr_t)bias % 16 == 0);
     long long blocks = (total + threads - 1) / threads;
     if (blocks > (long long)sm_count() * 16) blocks = (long long)sm_count() * 16;
     // few tokens (decode): one chunk per thread, most blocks; many tokens (prefill): two chunks per thread
@@ -1010,11 +1092,11 @@ extern "C" int qt_swiglu(const void* gate_up, int in_dtype, int n_splits, long l
 #define QT_LAUNCH_SWIGLU(TI, TO)                                                                                              \
     do {                                                                                                                      \
         if (vec && per_thread == 2) launch_kernel(swiglu_vec_kernel<TI, TO, 2>, dim3((unsigned)n_tokens, per_row), dim3(threads), 0, s, \
-                               (const TI*)gate_up, n_splits, (size_t)split_stride, (TO*)out, inter, group, act, limit);              \
+                               (const TI*)gate_up, n_splits, (size_t)split_stride, bias, (TO*)out, inter, group, act, limit);              \
         else if (vec) launch_kernel(swiglu_vec_kernel<TI, TO, 1>, dim3((unsigned)n_tokens, per_row), dim3(threads), 0, s,     \
-                               (const TI*)gate_up, n_splits, (size_t)split_stride, (TO*)out, inter, group, act, limit);              \
+                               (const TI*)gate_up, n_splits, (size_t)split_stride, bias, (TO*)out, inter, group, act, limit);              \
         else launch_kernel(swiglu_kernel<TI, TO>, dim3((unsigned)blocks), dim3(threads), 0, s, (const TI*)gate_up, n_splits,  \
-                           (size_t)split_stride, (TO*)out, total, inter, group, act, limit);                                         \
+                           (size_t)split_stride, bias, (TO*)out, total, inter, group, act, limit);                                         \
     } while (0)
     if (in_dtype == QT_F32 && out_dtype == QT_F32) QT_LAUNCH_SWIGLU(float, float);
     else if (in_dtype == QT_F32 && out_dtype == QT_BF16) QT_LAUNCH_SWIGLU(float, __nv_bfloat16);

@@ -285,10 +285,14 @@ __global__ void expert_combine_kernel(const T* __restrict__ y, const int* __rest
 // A learned router's choice.  logits [splits, T, cols] float (column e < experts: expert e; column `experts`, if
 // shared_gate, the logit of a shared expert's gate).  Scores are sigmoid(logit); the `top` largest are chosen (by their
 // logits; of equal ones the lower expert first), their weights are the scores over their sum (+ 1e-20) times `scale`, or, without `normalize`, the scores themselves times `scale`.
+// `softmax`: the scores are the softmax of the logits over all experts instead.  With `groups` > 1 the experts form that
+// many equal runs of neighbours, a group's score is the largest in it, and only the experts of the `keep` best groups (of
+// equal ones the lower group first) can be chosen.
 // One warp per token; chosen [T, top], weights [T, top], gate [T] = sigmoid of the extra column.
 __global__ void __launch_bounds__(128) route_top_kernel(const float* __restrict__ logits, int n_splits, size_t split_stride, int cols,
                                                         int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ gate,
-                                                        int n_tokens, int experts, int top, float scale, int normalize) {
+                                                        int n_tokens, int experts, int top, float scale, int normalize, int softmax, int groups,
+                                                        int keep) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float route_scores[];                      // [warps][experts]
@@ -300,6 +304,32 @@ __global__ void __launch_bounds__(128) route_top_kernel(const float* __restrict_
     for (int e = lane; e < experts; e += 32) score[e] = load_sum(logits, (size_t)t * cols + e, n_splits, split_stride);
     if (gate && lane == 0) gate[t] = 1.f / (1.f + expf(-load_sum(logits, (size_t)t * cols + experts, n_splits, split_stride)));
     __syncwarp();
+    float highest = 0.f, mass = 1.f;
+    if (softmax) {
+        highest = -INFINITY;
+        for (int e = lane; e < experts; e += 32) highest = fmaxf(highest, score[e]);
+        highest = warp_max(highest);
+        mass = 0.f;
+        for (int e = lane; e < experts; e += 32) mass += expf(score[e] - highest);
+        mass = warp_sum(mass);
+    }
+    if (groups > 1) {
+        float* best_of = route_scores + (size_t)(blockDim.x >> 5) * experts + (size_t)warp * groups;     // [groups] of this warp
+        const int size = experts / groups;
+        for (int g = lane; g < groups; g += 32) {
+            float m = -INFINITY;
+            for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, score[e]);
+            best_of[g] = m;
+        }
+        __syncwarp();
+        for (int g = lane; g < groups; g += 32) {               // a group is dropped if `keep` groups come before it
+            int before = 0;
+            for (int o = 0; o < groups; ++o) before += best_of[o] > best_of[g] || (best_of[o] == best_of[g] && o < g);
+            if (before >= keep)
+                for (int e = g * size; e < (g + 1) * size; ++e) score[e] = -INFINITY;
+        }
+        __syncwarp();
+    }
     float sum = 0.f;
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
@@ -311,7 +341,7 @@ __global__ void __launch_bounds__(128) route_top_kernel(const float* __restrict_
             const int where = __shfl_xor_sync(0xffffffffu, at, off);
             if (where < experts && (at == experts || other > best || (other == best && where < at))) { best = other; at = where; }
         }
-        const float chosen_score = 1.f / (1.f + expf(-best));
+        const float chosen_score = softmax ? expf(best - highest) / mass : 1.f / (1.f + expf(-best));
         sum += chosen_score;
         if (lane == 0) { chosen[(size_t)t * top + k] = at; weights[(size_t)t * top + k] = chosen_score; score[at] = -INFINITY; }
         __syncwarp();
@@ -323,13 +353,15 @@ __global__ void __launch_bounds__(128) route_top_kernel(const float* __restrict_
 }
 
 extern "C" int qt_route_top(const float* logits, int n_splits, long long split_stride, int cols, int* chosen, float* weights, float* gate,
-                            int n_tokens, int experts, int top, float scale, int normalize, void* stream) {
+                            int n_tokens, int experts, int top, float scale, int normalize, int softmax, int groups, int keep, void* stream) {
     QT_REQUIRE(n_tokens >= 0 && experts > 0 && top > 0 && top <= experts && cols >= experts + (gate ? 1 : 0) && n_splits >= 1,
                "route_top: bad sizes T=%d E=%d top=%d cols=%d", n_tokens, experts, top, cols);
-    QT_REQUIRE((size_t)4 * experts * sizeof(float) <= 48 * 1024, "route_top: %d experts are too many for a warp's scores in shared memory", experts);
+    QT_REQUIRE(groups >= 1 && experts % groups == 0 && keep >= 1 && keep <= groups && top <= keep * (experts / groups),
+               "route_top: %d experts out of the best %d of %d groups of %d", top, keep, groups, experts);
+    QT_REQUIRE((size_t)8 * experts * sizeof(float) <= 48 * 1024, "route_top: %d experts are too many for a warp's scores in shared memory", experts);
     if (n_tokens == 0) return QT_OK;
-    launch_kernel(route_top_kernel, dim3((n_tokens + 3) / 4), dim3(128), (size_t)4 * experts * sizeof(float), (cudaStream_t)stream, logits, n_splits,
-                  (size_t)split_stride, cols, chosen, weights, gate, n_tokens, experts, top, scale, normalize);
+    launch_kernel(route_top_kernel, dim3((n_tokens + 3) / 4), dim3(128), (size_t)4 * (experts + groups) * sizeof(float), (cudaStream_t)stream, logits, n_splits,
+                  (size_t)split_stride, cols, chosen, weights, gate, n_tokens, experts, top, scale, normalize, softmax, groups, keep);
     QT_CHECK_LAUNCH("route_top");
     return QT_OK;
 }

@@ -1,7 +1,7 @@
 // What follows a decode step's product, as device functions shared by the kernels that run it in their epilogue
 // (gemm_fused.cu: one launch per product; gemm_chain.cu: one persistent launch for a run of products).
 //
-//   STORE     out[m, n] = s_m * y                       float or bfloat16 (the output head)
+//   STORE     out[m, n] = s_m * y (+ bias[n])           float or bfloat16 (the output head)
 //   RESIDUAL  r = residual[m, n] + y; residual[m, n] = r;  and, for the norm that follows, xw[m, n] = bf16(r * g[n])
 //             and sq_out[tile, m] = sum over the tile's 128 columns of r^2
 //   SWIGLU    act[m, f] = a(s_m * gate) * (s_m * up), a = SiLU or another QT_ACT_*, the weight's rows alternating 16 of gate and 16 of up
@@ -32,6 +32,7 @@ struct EpilogueParams {
     int M, N;
     // the deferred factor of the norm in front of this product
     const float* sq_in; int sq_tiles; float inv_hidden; float eps;
+    const float* bias;                         // STORE / RESIDUAL / SWIGLU: [N] float, added to the (scaled) product; or null
     // STORE / SWIGLU
     void* out; int out_is_float; int act;      // act: the gate's activation, QT_ACT_*
     float limit;                               // of the capped gate (QT_ACT_CAPPED)
@@ -109,17 +110,22 @@ __device__ __forceinline__ Operands load_operands(const EpilogueParams& p, int m
     return o;
 }
 
+__device__ __forceinline__ int swiglu_gate_row(int lane) { const int f = 2 * lane; return (f >> 4) * 32 + (f & 15); }
+
 // SWIGLU: g and u are the gate and up sums of features 2 lane, 2 lane + 1 of tile w_tile (gate rows (f / 16) * 32 + f % 16
 // of the tile, up rows 16 further).
 __device__ __forceinline__ void finish_swiglu(const EpilogueParams& p, const Operands& ops, float2 g, float2 u, int m, int w_tile, int lane) {
     g.x *= ops.scale; g.y *= ops.scale; u.x *= ops.scale; u.y *= ops.scale;
+    if (p.bias) {
+        const int at = w_tile * TILE + swiglu_gate_row(lane);
+        if (at + 17 < p.N) { g.x += p.bias[at]; g.y += p.bias[at + 1]; u.x += p.bias[at + 16]; u.y += p.bias[at + 17]; }
+    }
     const int features = p.N >> 1, feature = w_tile * (TILE / 2) + 2 * lane;
     if (feature < features) {
         const float a0 = gated_value<true>(g.x, u.x, p.act, p.limit), a1 = gated_value<true>(g.y, u.y, p.act, p.limit);
         *reinterpret_cast<uint32_t*>((__nv_bfloat16*)p.out + (size_t)m * features + feature) = pack2(a0, a1);
     }
 }
-__device__ __forceinline__ int swiglu_gate_row(int lane) { const int f = 2 * lane; return (f >> 4) * 32 + (f & 15); }
 
 // The other epilogues: v holds the sums of columns w_tile * 128 + 4 lane .. + 3 of token m.  The whole warp calls.
 template <int EPI>
@@ -127,6 +133,12 @@ __device__ __forceinline__ void finish(const EpilogueParams& p, const Operands& 
     const int n_rows = p.N, n = w_tile * TILE + 4 * lane;
     if (EPI == EPI_STORE) {
         v.x *= ops.scale; v.y *= ops.scale; v.z *= ops.scale; v.w *= ops.scale;
+        if (p.bias) {
+            if (n < n_rows) v.x += p.bias[n];
+            if (n + 1 < n_rows) v.y += p.bias[n + 1];
+            if (n + 2 < n_rows) v.z += p.bias[n + 2];
+            if (n + 3 < n_rows) v.w += p.bias[n + 3];
+        }
         const float e[4] = {v.x, v.y, v.z, v.w};
         if (p.out_is_float) {
             float* dst = (float*)p.out + (size_t)m * n_rows + n;
@@ -141,6 +153,7 @@ __device__ __forceinline__ void finish(const EpilogueParams& p, const Operands& 
         float sq = 0.f;
         if (n < n_rows) {
             v.x += ops.a.x; v.y += ops.a.y; v.z += ops.a.z; v.w += ops.a.w;
+            if (p.bias) { const float4 b = ld4(p.bias + n); v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
             *reinterpret_cast<float4*>(p.residual + (size_t)m * n_rows + n) = v;
             sq = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
             if (p.norm_w)
@@ -196,6 +209,7 @@ inline int check_epilogue(const char* who, int epilogue, const EpilogueParams& p
             break;
         case EPI_RESIDUAL:
             QT_REQUIRE(p.residual != nullptr && p.N % 4 == 0 && (uintptr_t)p.residual % 16 == 0, "%s: the residual epilogue needs an aligned stream whose width is a multiple of 4 (N=%d)", who, p.N);
+            QT_REQUIRE((uintptr_t)p.bias % 16 == 0, "%s: the bias must be 16-byte aligned", who);
             QT_REQUIRE(p.norm_w == nullptr || (p.xw != nullptr && p.sq_out != nullptr && (uintptr_t)p.norm_w % 16 == 0 && (uintptr_t)p.xw % 8 == 0),
                        "%s: preparing the next norm needs its weight, an output for the weighted stream and one for the sums of squares", who);
             break;
@@ -204,6 +218,7 @@ inline int check_epilogue(const char* who, int epilogue, const EpilogueParams& p
             QT_REQUIRE(p.act >= 0 && p.act <= QT_ACT_CAPPED, "%s: unknown activation code %d", who, p.act);
             break;
         case EPI_QKV:
+            QT_REQUIRE(p.bias == nullptr, "%s: the q/k/v epilogue has no bias operand", who);
             QT_REQUIRE(p.d >= 16 && TILE % p.d == 0 && p.d % 4 == 0 && p.N % p.d == 0, "%s: head_dim=%d must divide %d for the fused rotation (N=%d)", who, p.d, TILE, p.N);
             QT_REQUIRE(p.nq > 0 && p.nkv > 0 && (p.N == p.nq * p.d || p.N == (p.nq + 2 * p.nkv) * p.d), "%s: N=%d is neither nq*d nor (nq+2nkv)*d", who, p.N);
             QT_REQUIRE(p.rotary_dim >= 0 && p.rotary_dim <= p.d && p.rotary_dim % 8 == 0, "%s: rotary_dim=%d must be a multiple of 8 within head_dim=%d", who, p.rotary_dim, p.d);

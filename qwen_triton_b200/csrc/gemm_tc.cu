@@ -49,7 +49,7 @@ template <int BX, typename TO, bool GATED>
 __global__ void __launch_bounds__(THREADS) gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w,
                                                           const __grid_constant__ CUtensorMap map_x, TO* __restrict__ out,
                                                           int M, int N, int kb_total, int kb_per_split,
-                                                          size_t split_stride, int stages, int act, float limit, int* status) {
+                                                          size_t split_stride, int stages, int act, float limit, const float* __restrict__ bias, int* status) {
     constexpr uint32_t X_BYTES = BX * BK * 2;
     constexpr uint32_t STAGE_BYTES = W_BYTES + X_BYTES;
     constexpr uint32_t TMEM_COLS = BX < 32 ? 32 : BX;
@@ -138,6 +138,7 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_kernel(const __grid_constant_
         tc_fence_after();
         const int n = w0 + quarter * 32 + lane;
         TO* dst = out + (size_t)split * split_stride;
+        const float add = bias && n < N && split == 0 ? bias[n] : 0.f;      // one plane of a split product carries the bias
         if (ready) {
 #pragma unroll 1
             for (int c = 0; c < BX; c += 16) {
@@ -148,7 +149,7 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_kernel(const __grid_constant_
                     const bool upper = (lane & 16) != 0;
 #pragma unroll
                     for (int j = 0; j < 16; j += 2) {
-                        const float mine0 = __uint_as_float(v[j]), mine1 = __uint_as_float(v[j + 1]);
+                        const float mine0 = __uint_as_float(v[j]) + add, mine1 = __uint_as_float(v[j + 1]) + add;
                         const float got = __shfl_xor_sync(0xffffffffu, upper ? mine0 : mine1, 16);
                         const float g = upper ? got : mine0;          // lower lanes: token j (their gate, the partner's up)
                         const float u = upper ? mine1 : got;          // upper lanes: token j + 1 (the partner's gate, their up)
@@ -159,7 +160,7 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_kernel(const __grid_constant_
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
                         const int m = x0 + c + j;
-                        if (m < M) dst[(size_t)m * N + n] = from_float<TO>(__uint_as_float(v[j]));
+                        if (m < M) dst[(size_t)m * N + n] = from_float<TO>(__uint_as_float(v[j]) + add);
                     }
                 }
             }
@@ -324,7 +325,8 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_tc_pair_kernel(const __grid_c
                                                                   const __grid_constant__ CUtensorMap map_x, TO* __restrict__ out,
                                                                   int M, int N, int kb_total, int kb_per_split, int splits,
                                                                   size_t split_stride, int act, float limit, int vector_stores, int tail_tiles,
-                                                                  float* __restrict__ tail_scratch, int* tail_flags, int* status) {
+                                                                  float* __restrict__ tail_scratch, int* tail_flags, const float* __restrict__ bias,
+                                                                  int* status) {
     // instruction descriptor: float accumulator, bfloat16 A and B, both K-major, N = 256 weight rows, M = 256 tokens over the pair
     constexpr uint32_t IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(PAIR_W >> 3) << 17) | ((uint32_t)(PAIR_X >> 4) << 24);
     constexpr int S = PAIR_STAGES;
@@ -533,6 +535,10 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_tc_pair_kernel(const __grid_c
                 __syncwarp();                                // lanes beyond M skip the stores; the load wants the whole warp
                 tmem_load32(taddr + (uint32_t)c, v);
                 if (m >= M) continue;
+                if (bias && item.split == 0) {               // the same 32 columns for every thread of the warp
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(__uint_as_float(v[j]) + (n0 + c + j < N ? __ldg(bias + n0 + c + j) : 0.f));
+                }
                 if (SWIGLU) {
                     // columns c .. c + 15 are the gate rows of 16 features, c + 16 .. c + 31 the up rows of the same
                     const int f0 = (n0 + c) >> 1;
@@ -616,7 +622,7 @@ int pick_tail_tiles(long long n_tiles, int pairs, int kb_total, int tail, int ta
 
 template <typename TO, bool SWIGLU>
 int launch_pair(const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int M, int N, int kb_total, int splits,
-                size_t split_stride, int act, float limit, int tail, float* tail_scratch, int* tail_flags, int tail_pairs, int* status,
+                size_t split_stride, int act, float limit, int tail, float* tail_scratch, int* tail_flags, int tail_pairs, const float* bias, int* status,
                 cudaStream_t stream) {
     const size_t smem = (size_t)PAIR_STAGES * PAIR_STAGE_BYTES + 1024 + (2 * PAIR_STAGES + 5) * 8 + 16;
     static int resident_pairs = 0;                           // pairs the device runs at once (one per TPC that can host a cluster)
@@ -649,7 +655,7 @@ int launch_pair(const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int
     const int per16 = 16 / (int)sizeof(TO), row_elems = SWIGLU ? N / 2 : N;
     const int vector_stores = ((uintptr_t)out % 16 == 0 && row_elems % per16 == 0 && split_stride % per16 == 0) ? 1 : 0;
     launch_kernel_cluster(gemm_tc_pair_kernel<TO, SWIGLU>, dim3(2 * pairs), dim3(THREADS), smem, stream, 2, map_w, map_x, out, M, N, kb_total,
-                          kb_per_split, splits, split_stride, act, limit, vector_stores, tail_tiles, tail_scratch, tail_flags, status);
+                          kb_per_split, splits, split_stride, act, limit, vector_stores, tail_tiles, tail_scratch, tail_flags, bias, status);
     QT_CHECK_LAUNCH("gemm_tc_pair");
     return QT_OK;
 }
@@ -657,7 +663,7 @@ int launch_pair(const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int
 // ----------------------------------------------------------------------------- host side
 template <int BX, typename TO, bool GATED>
 int launch(const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int M, int N, int kb_total, int splits,
-           size_t split_stride, int stages, int act, float limit, int* status, cudaStream_t stream) {
+           size_t split_stride, int stages, int act, float limit, const float* bias, int* status, cudaStream_t stream) {
     constexpr uint32_t STAGE_BYTES = W_BYTES + BX * BK * 2;
     // Up to 16 tokens a block streams weights through a three-stage ring (54 KB), so that four blocks share an SM and
     // the next product's blocks can move in beside this one's last blocks and fetch their first weight tiles early
@@ -682,7 +688,7 @@ int launch(const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int M, i
     }
     const int kb_per_split = (kb_total + splits - 1) / splits;
     dim3 grid(((N + BW - 1) / BW) * ((M + BX - 1) / BX), 1, splits);
-    launch_kernel(gemm_tc_kernel<BX, TO, GATED>, dim3(grid), dim3(THREADS), smem, stream, map_w, map_x, out, M, N, kb_total, kb_per_split, split_stride, stages, act, limit, status);
+    launch_kernel(gemm_tc_kernel<BX, TO, GATED>, dim3(grid), dim3(THREADS), smem, stream, map_w, map_x, out, M, N, kb_total, kb_per_split, split_stride, stages, act, limit, bias, status);
     QT_CHECK_LAUNCH("gemm_tc");
     return QT_OK;
 }
@@ -690,13 +696,13 @@ int launch(const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int M, i
 
 template <typename TO, bool GATED>
 int dispatch_tile(int bx, const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int M, int N, int kb_total, int splits,
-                  size_t split_stride, int stages, int act, float limit, int* status, cudaStream_t stream) {
+                  size_t split_stride, int stages, int act, float limit, const float* bias, int* status, cudaStream_t stream) {
     switch (bx) {
-        case 16: return launch<16, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, status, stream);
-        case 32: return launch<32, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, status, stream);
-        case 64: return launch<64, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, status, stream);
-        case 128: return launch<128, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, status, stream);
-        case 256: return launch<256, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, status, stream);
+        case 16: return launch<16, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
+        case 32: return launch<32, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
+        case 64: return launch<64, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
+        case 128: return launch<128, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
+        case 256: return launch<256, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
     }
     QT_FAIL(QT_ERR_ARG, "gemm_tc: token tile %d is not one of 16, 32, 64, 128, 256", bx);
 }
@@ -708,10 +714,12 @@ int dispatch_tile(int bx, const CUtensorMap& map_w, const CUtensorMap& map_x, TO
 // blocks: (splits - 1) * ceil(ceil(K/64) / splits) < ceil(K/64).  `status` is a device int that stays
 // 0 unless a wait inside the kernel ran out (1 = producer, 2 = MMA issuer, 3 = epilogue).
 // `stages` > 0 overrides the depth of the shared-memory ring (a tuning knob; 0 picks the default).
+// `bias` (or null): [N] float, added to the sums (to the first plane of split sums; ahead of the gate).
 // With `gated` the weight's rows alternate 16 of a gate and 16 of an up projection and `out` is [M, N / 2] bfloat16 =
 // act(gate) * up (`act`: one of QT_ACT_*; one K range only).
 extern "C" int qt_gemm_tc(const void* x, const void* w, void* out, int out_dtype, int M, int N, int K, int token_tile,
-                          int splits, long long split_stride, int stages, int gated, int act, float limit, int* status, void* stream) {
+                          int splits, long long split_stride, int stages, int gated, int act, float limit, const float* bias, int* status,
+                          void* stream) {
     QT_REQUIRE(!gated || (splits == 1 && out_dtype == QT_BF16 && N % 32 == 0 && act >= 0 && act <= QT_ACT_CAPPED),
                "gemm_tc: the gated epilogue writes bfloat16 from one K range of gate and up rows in groups of 16 (N=%d, splits=%d)", N, splits);
     QT_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_tc: bad sizes M=%d N=%d K=%d", M, N, K);
@@ -731,11 +739,11 @@ extern "C" int qt_gemm_tc(const void* x, const void* w, void* out, int out_dtype
     if (rc) return rc;
     cudaStream_t s = (cudaStream_t)stream;
     if (gated)
-        return dispatch_tile<__nv_bfloat16, true>(token_tile, map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, stages, act, limit, status, s);
+        return dispatch_tile<__nv_bfloat16, true>(token_tile, map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, stages, act, limit, bias, status, s);
     if (out_dtype == QT_BF16)
-        return dispatch_tile<__nv_bfloat16, false>(token_tile, map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, splits, (size_t)split_stride, stages, 0, 0.f, status, s);
+        return dispatch_tile<__nv_bfloat16, false>(token_tile, map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, splits, (size_t)split_stride, stages, 0, 0.f, bias, status, s);
     if (out_dtype == QT_F32)
-        return dispatch_tile<float, false>(token_tile, map_w, map_x, (float*)out, M, N, kb_total, splits, (size_t)split_stride, stages, 0, 0.f, status, s);
+        return dispatch_tile<float, false>(token_tile, map_w, map_x, (float*)out, M, N, kb_total, splits, (size_t)split_stride, stages, 0, 0.f, bias, status, s);
     QT_FAIL(QT_ERR_ARG, "gemm_tc: unknown output type %d", out_dtype);
 }
 
@@ -750,7 +758,7 @@ extern "C" int qt_gemm_tc(const void* x, const void* w, void* out, int out_dtype
 extern "C" int qt_gemm_tc_pair_slots() { return PAIR_SLOT_FLOATS; }
 extern "C" int qt_gemm_tc_pair(const void* x, const void* w, void* out, int out_dtype, int M, int N, int K, int swiglu,
                                int act, float limit, int splits, long long split_stride, int tail, float* tail_scratch, int* tail_flags,
-                               int tail_pairs, int* status, void* stream) {
+                               int tail_pairs, const float* bias, int* status, void* stream) {
     QT_REQUIRE(act >= 0 && act <= QT_ACT_CAPPED, "gemm_tc_pair: unknown activation code %d", act);
     QT_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_tc_pair: bad sizes M=%d N=%d K=%d", M, N, K);
     QT_REQUIRE(K % 8 == 0, "gemm_tc_pair: K=%d must be a multiple of 8 (rows must start on 16-byte boundaries for TMA)", K);
@@ -768,9 +776,9 @@ extern "C" int qt_gemm_tc_pair(const void* x, const void* w, void* out, int out_
     rc = tensor_map(&map_x, x, (uint64_t)M, (uint64_t)K, (uint32_t)PAIR_HALF);
     if (rc) return rc;
     cudaStream_t s = (cudaStream_t)stream;
-    if (out_dtype == QT_BF16 && swiglu) return launch_pair<__nv_bfloat16, true>(map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, act, limit, tail, tail_scratch, tail_flags, tail_pairs, status, s);
-    if (out_dtype == QT_BF16) return launch_pair<__nv_bfloat16, false>(map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, 0, 0.f, tail, tail_scratch, tail_flags, tail_pairs, status, s);
-    if (out_dtype == QT_F32 && !swiglu) return launch_pair<float, false>(map_w, map_x, (float*)out, M, N, kb_total, splits, (size_t)split_stride, 0, 0.f, tail, tail_scratch, tail_flags, tail_pairs, status, s);
+    if (out_dtype == QT_BF16 && swiglu) return launch_pair<__nv_bfloat16, true>(map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, act, limit, tail, tail_scratch, tail_flags, tail_pairs, bias, status, s);
+    if (out_dtype == QT_BF16) return launch_pair<__nv_bfloat16, false>(map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, 0, 0.f, tail, tail_scratch, tail_flags, tail_pairs, bias, status, s);
+    if (out_dtype == QT_F32 && !swiglu) return launch_pair<float, false>(map_w, map_x, (float*)out, M, N, kb_total, splits, (size_t)split_stride, 0, 0.f, tail, tail_scratch, tail_flags, tail_pairs, bias, status, s);
     QT_FAIL(QT_ERR_ARG, "gemm_tc_pair: output type %d%s is not offered", out_dtype, swiglu ? " with the SiLU-gated epilogue" : "");
 }
 

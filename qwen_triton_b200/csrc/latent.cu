@@ -12,7 +12,7 @@
 //                         by the token's position -> the cache row.
 // latent_query_rot_kernel the rotated part of every head's query: rotation by position into the query rows.
 // head_product_kernel     Y[t, h, n] = sum_k X[t, h, k] W[h, n, k] for every head with its own matrix (float sums), with
-//                         strides for X and Y and optionally times sigmoid(gate[t, h * N + n]).
+//                         strides for X and Y and optionally times sigmoid(gate[t, h * N + n]) or sigmoid(gate[t, h]).
 // head_product_mma_kernel the same on the tensor cores (mma.sync m16n8k16) for bfloat16 matrices and results.
 // Rotation: element i of the rotated part turns with element i + rd / 2 by the angle whose cos and sin the table row
 // of the position holds (cos | sin, rd columns); elements beyond the first rd pass unchanged.
@@ -165,7 +165,8 @@ struct HeadProductParams {
     const void* x; int x_splits; size_t x_split_stride; long long x_row, x_head; int x_offset;    // X[t, h, k] at t * x_row + h * x_head + x_offset + k
     const void* w;                                                                                // [heads, N, K]
     void* y; long long y_row, y_head; int y_offset;
-    const float* gate; int gate_splits; size_t gate_split_stride; int gate_cols, gate_offset;      // optional: times sigmoid(gate[t, gate_offset + h * N + n])
+    const float* gate; int gate_splits; size_t gate_split_stride; int gate_cols, gate_offset;      // optional: times sigmoid(gate[t, gate_offset + h * gate_head + n * gate_elem])
+    int gate_head, gate_elem;      // N and 1 (a gate per element), or 1 and 0 (one per head)
     int n_tokens, heads, n, k;
 };
 
@@ -218,7 +219,7 @@ __global__ void __launch_bounds__(256) head_product_kernel(const HeadProductPara
             if (n >= p.n) continue;
             float v = acc[i][j];
             if (p.gate) {
-                const float g = sum_splits(p.gate, (size_t)t * p.gate_cols + p.gate_offset + (size_t)h * p.n + n, p.gate_splits, p.gate_split_stride);
+                const float g = sum_splits(p.gate, (size_t)t * p.gate_cols + p.gate_offset + (size_t)h * p.gate_head + (size_t)n * p.gate_elem, p.gate_splits, p.gate_split_stride);
                 v = v / (1.f + expf(-g));
             }
             y[(size_t)((long long)t * p.y_row + (long long)h * p.y_head + p.y_offset + n)] = from_float<TO>(v);
@@ -331,9 +332,9 @@ __global__ void __launch_bounds__(128) head_product_mma_kernel(const HeadProduct
 #pragma unroll
                 for (int nt = 0; nt < 8; ++nt) {
                     const int n = n0 + nt * 8 + 2 * t;
-                    const size_t at = (size_t)tok * p.gate_cols + p.gate_offset + (size_t)h * p.n + n;
+                    const size_t at = (size_t)tok * p.gate_cols + p.gate_offset + (size_t)h * p.gate_head + (size_t)n * p.gate_elem;
                     if (tok < p.n_tokens && n < p.n) gates[nt][2 * r] += __ldg(gate + at);
-                    if (tok < p.n_tokens && n + 1 < p.n) gates[nt][2 * r + 1] += __ldg(gate + at + 1);
+                    if (tok < p.n_tokens && n + 1 < p.n) gates[nt][2 * r + 1] += __ldg(gate + at + p.gate_elem);
                 }
             }
         }
@@ -365,14 +366,16 @@ __global__ void __launch_bounds__(128) head_product_mma_kernel(const HeadProduct
 extern "C" int qt_head_product(const void* x, int x_dtype, int x_splits, long long x_split_stride, long long x_row, long long x_head, int x_offset,
                                const void* w, int w_dtype, void* y, int y_dtype, long long y_row, long long y_head, int y_offset,
                                const float* gate, int gate_splits, long long gate_split_stride, int gate_cols, int gate_offset,
-                               int n_tokens, int heads, int n, int k, void* stream) {
+                               int gate_per_head, int n_tokens, int heads, int n, int k, void* stream) {
     QT_REQUIRE(n_tokens >= 0 && heads > 0 && n > 0 && k > 0 && x_splits >= 1 && gate_splits >= 1, "head_product: bad sizes");
     QT_REQUIRE(heads <= 65535 && (n_tokens + HP_TM - 1) / HP_TM <= 65535, "head_product: too many heads or tokens for one launch");
-    QT_REQUIRE(!gate || gate_offset + heads * n <= gate_cols, "head_product: the gate needs %d columns at %d of %d", heads * n, gate_offset, gate_cols);
+    QT_REQUIRE(!gate || gate_offset + heads * (gate_per_head ? 1 : n) <= gate_cols, "head_product: the gate needs %d columns at %d of %d",
+               heads * (gate_per_head ? 1 : n), gate_offset, gate_cols);
     if (n_tokens == 0) return QT_OK;
     cudaStream_t s = (cudaStream_t)stream;
     HeadProductParams p{x, x_splits, (size_t)x_split_stride, x_row, x_head, x_offset, w, y, y_row, y_head, y_offset,
-                        gate, gate_splits, (size_t)gate_split_stride, gate_cols, gate_offset, n_tokens, heads, n, k};
+                        gate, gate_splits, (size_t)gate_split_stride, gate_cols, gate_offset, gate_per_head ? 1 : n, gate_per_head ? 0 : 1,
+                        n_tokens, heads, n, k};
     dim3 grid((n + HP_TN - 1) / HP_TN, (n_tokens + HP_TM - 1) / HP_TM, heads);
     // bfloat16 matrices and results whose rows start on 16 bytes take the tensor cores (QT_B200_HEAD_PRODUCT_MMA=0: never)
     static const bool mma_allowed = [] { const char* env = getenv("QT_B200_HEAD_PRODUCT_MMA"); return !(env && env[0] == '0'); }();

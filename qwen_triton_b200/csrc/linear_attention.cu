@@ -11,9 +11,11 @@
 //   transposed, [slots, heads, vdim, dim], so that the 8 lanes of a column read and write 8 RPL consecutive floats.
 //   A sequence's tokens are walked in order, 16 at a time through shared memory; a one-token step is the same kernel
 //   with one token, whose cost is the state's bytes.
-// linear_attention_gate_norm_kernel   one block per token: out = o / sqrt(mean(o^2) + eps) * weight * sigmoid(g) * scale,
-//   the mean over all heads' outputs of the token at once, g the projection's gate columns, rounded once to the
-//   output type.
+// linear_attention_step_kernel   few tokens a sequence; it also takes decays that depend on the token, per head or per key
+//   channel, a factor on v and q/k heads shared by several heads (qt_decayed_attention_steps).
+// group_gate_norm_kernel   out = o / sqrt(mean(o^2) + eps) * weight * gate, the mean over the whole row or over equal parts of it,
+//   the gate (sigmoid or SiLU of projection columns) behind the norm or ahead of it, with an optional skip term; rounded
+//   once to the output type.
 #include "common.cuh"
 
 #include <math.h>
@@ -32,7 +34,13 @@ struct LinAttnParams {
     float* out;                        // [T, heads, vdim]
     const int* seq_start; const int* slots;
     int heads, dim, vdim, act;
+    // decays that depend on the token (null: the constant ones): their logarithms, [T, heads] or [T, heads, dim]
+    const float* log_decay;
+    const float* v_scale;              // [T, heads] or null: a factor on the token's v
+    int heads_per_key;                 // heads that share a q and k head
+    float out_scale;                   // factor on o
 };
+constexpr int LA_CONSTANT = 0, LA_PER_HEAD = 1, LA_PER_CHANNEL = 2;      // what a decay depends on besides its head
 
 __device__ __forceinline__ float la_raw(const LinAttnParams& p, size_t index) {
     float x = __ldg(p.proj + index);
@@ -180,7 +188,7 @@ __global__ void __launch_bounds__(COLS * LA_LANES) linear_attention_scan_kernel(
 // Steps in which no sequence brings more than a few tokens (one-token steps above all): nothing is staged or fetched
 // ahead, a thread reads its rows' q and k from the projection itself (the 32 columns of a block read the same ones, from
 // L1), so the kernel is short and light in registers and many blocks share an SM; its cost is the state's bytes.
-template <int RPL>
+template <int RPL, int MODE>
 __global__ void __launch_bounds__(32 * LA_LANES) linear_attention_step_kernel(const LinAttnParams p) {
     pdl_launch_dependents();
     pdl_wait();
@@ -188,7 +196,8 @@ __global__ void __launch_bounds__(32 * LA_LANES) linear_attention_step_kernel(co
     const int lane = threadIdx.x % LA_LANES, col = blockIdx.x * 32 + threadIdx.x / LA_LANES;
     const int begin = p.seq_start[seq], end = p.seq_start[seq + 1];
     if (begin >= end) return;
-    const float decay = p.decay[head];
+    const float constant = MODE == LA_CONSTANT ? p.decay[head] : 0.f;
+    const int key_head = MODE == LA_CONSTANT ? head : head / p.heads_per_key;
     const bool live = col < p.vdim;
     float* state = p.state + (((size_t)p.slots[seq] * p.heads + head) * p.vdim + (live ? col : 0)) * p.dim;
     const int row0 = lane * RPL;
@@ -213,9 +222,20 @@ __global__ void __launch_bounds__(32 * LA_LANES) linear_attention_step_kernel(co
     const bool quads = p.n_splits == 1 && p.dim % 4 == 0 && p.at_q % 4 == 0 && p.at_k % 4 == 0 && p.proj_cols % 4 == 0 && ((uintptr_t)p.proj & 15) == 0;
     for (int t = begin; t < end; ++t) {
         const size_t row = (size_t)t * p.proj_cols;
-        const float v = live ? la_act(p, la_raw(p, row + p.at_v + (size_t)head * p.vdim + col)) : 0.f;
+        float v = live ? la_act(p, la_raw(p, row + p.at_v + (size_t)head * p.vdim + col)) : 0.f;
+        float decay[MODE == LA_PER_CHANNEL ? RPL : 1];
+        decay[0] = constant;
+        if (MODE != LA_CONSTANT) {
+            const size_t th = (size_t)t * p.heads + head;
+            if (p.v_scale) v *= __ldg(p.v_scale + th);
+            if (MODE == LA_PER_HEAD) decay[0] = expf(__ldg(p.log_decay + th));
+            else {
+#pragma unroll
+                for (int i = 0; i < (MODE == LA_PER_CHANNEL ? RPL : 1); ++i) decay[i] = row0 + i < p.dim ? expf(__ldg(p.log_decay + th * p.dim + row0 + i)) : 0.f;
+            }
+        }
         float q[RPL], k[RPL];
-        const size_t q_at = row + p.at_q + (size_t)head * p.dim + row0, k_at = row + p.at_k + (size_t)head * p.dim + row0;
+        const size_t q_at = row + p.at_q + (size_t)key_head * p.dim + row0, k_at = row + p.at_k + (size_t)key_head * p.dim + row0;
         if (quads) {                                        // 16-byte loads of a row that is finished and aligned
 #pragma unroll
             for (int i = 0; i < RPL; i += 4) {
@@ -236,14 +256,14 @@ __global__ void __launch_bounds__(32 * LA_LANES) linear_attention_step_kernel(co
         float a0 = 0.f, a1 = 0.f;
 #pragma unroll
         for (int i = 0; i < RPL; i += 2) {
-            S[i] = fmaf(decay, S[i], la_act(p, k[i]) * v);             a0 = fmaf(S[i], la_act(p, q[i]), a0);
-            S[i + 1] = fmaf(decay, S[i + 1], la_act(p, k[i + 1]) * v); a1 = fmaf(S[i + 1], la_act(p, q[i + 1]), a1);
+            S[i] = fmaf(decay[MODE == LA_PER_CHANNEL ? i : 0], S[i], la_act(p, k[i]) * v);             a0 = fmaf(S[i], la_act(p, q[i]), a0);
+            S[i + 1] = fmaf(decay[MODE == LA_PER_CHANNEL ? i + 1 : 0], S[i + 1], la_act(p, k[i + 1]) * v); a1 = fmaf(S[i + 1], la_act(p, q[i + 1]), a1);
         }
         float acc = a0 + a1;
         acc += __shfl_xor_sync(0xffffffffu, acc, 1);
         acc += __shfl_xor_sync(0xffffffffu, acc, 2);
         acc += __shfl_xor_sync(0xffffffffu, acc, 4);
-        if (lane == 0 && live) p.out[((size_t)t * p.heads + head) * p.vdim + col] = acc;
+        if (lane == 0 && live) p.out[((size_t)t * p.heads + head) * p.vdim + col] = MODE == LA_CONSTANT ? acc : acc * p.out_scale;
     }
     if (live) {
         if (vec) {
@@ -365,16 +385,17 @@ extern "C" int qt_linear_attention_scan(const float* proj, int n_splits, long lo
     QT_REQUIRE(at_q >= 0 && at_k >= 0 && at_v >= 0 && at_q + heads * dim <= proj_cols && at_k + heads * dim <= proj_cols && at_v + heads * vdim <= proj_cols,
                "linear_attention_scan: q, k or v columns outside the projection's %d", proj_cols);
     if (n_seqs == 0) return QT_OK;
-    LinAttnParams p{proj, n_splits, (size_t)split_stride, proj_cols, at_q, at_k, at_v, decay, state, out, seq_start, slots, heads, dim, vdim, act};
+    LinAttnParams p{proj, n_splits, (size_t)split_stride, proj_cols, at_q, at_k, at_v, decay, state, out, seq_start, slots, heads, dim, vdim, act,
+                    nullptr, nullptr, 1, 1.f};
     cudaStream_t s = (cudaStream_t)stream;
     // blocks of 32 columns where they fill the machine twice over (many sequences: every block stages its head's q and k
     // itself), else of 16, so that one prompt still gives most SMs a block
     const bool wide = (long long)((vdim + 31) / 32) * heads * n_seqs >= 2LL * sm_count();
     if (max_q_len <= 4) {                                  // few tokens a sequence: the short kernel
         const dim3 grid((vdim + 31) / 32, heads, n_seqs), block(32 * LA_LANES);
-        if (dim <= LA_LANES * 8) launch_kernel(linear_attention_step_kernel<8>, grid, block, 0, s, p);
-        else if (dim <= LA_LANES * 16) launch_kernel(linear_attention_step_kernel<16>, grid, block, 0, s, p);
-        else launch_kernel(linear_attention_step_kernel<32>, grid, block, 0, s, p);
+        if (dim <= LA_LANES * 8) launch_kernel(linear_attention_step_kernel<8, LA_CONSTANT>, grid, block, 0, s, p);
+        else if (dim <= LA_LANES * 16) launch_kernel(linear_attention_step_kernel<16, LA_CONSTANT>, grid, block, 0, s, p);
+        else launch_kernel(linear_attention_step_kernel<32, LA_CONSTANT>, grid, block, 0, s, p);
         QT_CHECK_LAUNCH("linear_attention_scan");
         return QT_OK;
     }
@@ -400,43 +421,119 @@ extern "C" int qt_linear_attention_scan(const float* proj, int n_splits, long lo
     return QT_OK;
 }
 
-// ----------------------------------------------------------------------------- norm over all heads, gate, scale
-template <typename TO>
-__global__ void linear_attention_gate_norm_kernel(const float* __restrict__ o, const float* __restrict__ proj, int n_splits, size_t split_stride,
-                                                  int proj_cols, int at_gate, const float* __restrict__ weight, float eps, float scale,
-                                                  TO* __restrict__ out, int width) {
+// The recurrence with decays that depend on the token, token by token: S <- diag(exp(log_decay_t)) S + k_t (v_scale_t v_t)^T,
+// o_t = out_scale S^T q_t.  log_decay is [T, heads] or (per_channel) [T, heads, dim]; q and k have heads / heads_per_key heads.
+// The form for steps of few tokens a sequence (linear_attention_chunk.cu takes long ones).
+extern "C" int qt_decayed_attention_steps(const float* proj, int n_splits, long long split_stride, int proj_cols, int at_q, int at_k, int at_v,
+                                          const float* log_decay, int per_channel, const float* v_scale, float out_scale, float* state, float* out,
+                                          const int* seq_start, const int* slots, int n_seqs, int heads, int heads_per_key, int dim, int vdim,
+                                          void* stream) {
+    QT_REQUIRE(n_seqs >= 0 && heads > 0 && heads_per_key > 0 && heads % heads_per_key == 0 && dim > 0 && vdim > 0 && n_splits >= 1,
+               "decayed_attention: bad sizes B=%d H=%d/%d dim=%d vdim=%d", n_seqs, heads, heads_per_key, dim, vdim);
+    QT_REQUIRE(dim <= LA_LANES * 32, "decayed_attention: %d key channels per head are beyond what a column's lanes hold (%d)", dim, LA_LANES * 32);
+    QT_REQUIRE(at_q >= 0 && at_k >= 0 && at_v >= 0 && at_q + heads / heads_per_key * dim <= proj_cols && at_k + heads / heads_per_key * dim <= proj_cols &&
+               at_v + heads * vdim <= proj_cols, "decayed_attention: q, k or v columns outside the projection's %d", proj_cols);
+    QT_REQUIRE(log_decay != nullptr && heads <= 65535 && n_seqs <= 65535, "decayed_attention: no decays, or too many heads or sequences for one launch");
+    if (n_seqs == 0) return QT_OK;
+    LinAttnParams p{proj, n_splits, (size_t)split_stride, proj_cols, at_q, at_k, at_v, nullptr, state, out, seq_start, slots, heads, dim, vdim, 0,
+                    log_decay, v_scale, heads_per_key, out_scale};
+    cudaStream_t s = (cudaStream_t)stream;
+    const dim3 grid((vdim + 31) / 32, heads, n_seqs), block(32 * LA_LANES);
+#define QT_LAUNCH_STEPS(RPL)                                                                             \
+    do {                                                                                                 \
+        if (per_channel) launch_kernel(linear_attention_step_kernel<RPL, LA_PER_CHANNEL>, grid, block, 0, s, p); \
+        else launch_kernel(linear_attention_step_kernel<RPL, LA_PER_HEAD>, grid, block, 0, s, p);         \
+    } while (0)
+    if (dim <= LA_LANES * 8) QT_LAUNCH_STEPS(8);
+    else if (dim <= LA_LANES * 16) QT_LAUNCH_STEPS(16);
+    else QT_LAUNCH_STEPS(32);
+#undef QT_LAUNCH_STEPS
+    QT_CHECK_LAUNCH("decayed_attention_steps");
+    return QT_OK;
+}
+
+// ----------------------------------------------------------------------------- skip, gate and norm behind a recurrence
+// y = o (+ skip[h] * x, h the head of the element); with gate_first y *= a(g); then y / sqrt(mean(y^2) + eps) * weight * scale over
+// `groups` equal parts of the row, each by its own mean; without gate_first times a(g).  a is the sigmoid or (silu) SiLU of the
+// gate's sums.  weight has an element per column, or (weight_len = the part's width) one per column of a part.  Rounded once.
+struct GroupNormParams {
+    const float* o;                                                    // [T, width]
+    const float* x; int x_cols, at_x; const float* skip; int per_skip;   // x [T, x_cols] from column at_x; skip[i / per_skip]; or null
+    const float* proj; int n_splits; size_t split_stride; int proj_cols, at_gate;    // the gate's sums; or null
+    const float* weight; int weight_len;
+    float eps, scale;
+    int width, part, silu, gate_first;
+};
+
+__device__ __forceinline__ float gn_gate(const GroupNormParams& p, size_t t, int i) {
+    const float* at = p.proj + t * p.proj_cols + p.at_gate + i;
+    float g = at[0];
+    for (int s = 1; s < p.n_splits; ++s) g += at[(size_t)s * p.split_stride];
+    const float sig = 1.f / (1.f + expf(-g));
+    return p.silu ? g * sig : sig;
+}
+__device__ __forceinline__ float gn_value(const GroupNormParams& p, size_t t, int i) {
+    float y = p.o[t * p.width + i];
+    if (p.x) y += p.skip[i / p.per_skip] * p.x[t * p.x_cols + p.at_x + i];
+    if (p.proj && p.gate_first) y *= gn_gate(p, t, i);
+    return y;
+}
+
+// WARP: a part per warp (parts of up to 32 GN_CACHE elements), else a part per block (up to GN_CACHE elements a thread); elements
+// beyond what the registers hold are formed again in the second pass.  grid (tokens, blocks of parts).
+constexpr int GN_CACHE = 8;
+
+template <typename TO, bool WARP>
+__global__ void group_gate_norm_kernel(const GroupNormParams p, TO* __restrict__ out) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float scratch[32];
     const size_t t = blockIdx.x;
-    const float* row = o + t * width;
-    float sq = 0.f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) sq += row[i] * row[i];
-    const float inv = rsqrtf(block_sum(sq, scratch) / (float)width + eps) * scale;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        float y = row[i] * inv * weight[i];
-        if (proj) {
-            const size_t at = t * proj_cols + at_gate + i;
-            float g = proj[at];
-            for (int s = 1; s < n_splits; ++s) g += proj[at + (size_t)s * split_stride];
-            y = y / (1.f + expf(-g));
-        }
-        out[t * width + i] = from_float<TO>(y);
+    const int part = WARP ? blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5) : blockIdx.y;
+    if (WARP && part * p.part >= p.width) return;                       // whole warps leave; a block's threads stay together otherwise
+    const int first = WARP ? threadIdx.x & 31 : threadIdx.x, step = WARP ? 32 : blockDim.x, base = part * p.part;
+    float y[GN_CACHE], sq = 0.f;
+#pragma unroll
+    for (int j = 0; j < GN_CACHE; ++j) {
+        const int i = first + j * step;
+        y[j] = i < p.part ? gn_value(p, t, base + i) : 0.f;
+        sq += y[j] * y[j];
     }
+    for (int i = first + GN_CACHE * step; i < p.part; i += step) { const float v = gn_value(p, t, base + i); sq += v * v; }
+    const float inv = rsqrtf((WARP ? warp_sum(sq) : block_sum(sq, scratch)) / (float)p.part + p.eps) * p.scale;
+    auto finish = [&](float v, int i) {
+        v *= inv * p.weight[p.weight_len == p.part ? i : base + i];
+        if (p.proj && !p.gate_first) v *= gn_gate(p, t, base + i);
+        out[t * p.width + base + i] = from_float<TO>(v);
+    };
+#pragma unroll
+    for (int j = 0; j < GN_CACHE; ++j)
+        if (first + j * step < p.part) finish(y[j], first + j * step);
+    for (int i = first + GN_CACHE * step; i < p.part; i += step) finish(gn_value(p, t, base + i), i);
 }
 
-extern "C" int qt_linear_attention_gate_norm(const float* o, const float* proj, int n_splits, long long split_stride, int proj_cols, int at_gate,
-                                             const float* weight, float eps, float scale, void* out, int out_dtype, int n_tokens, int width,
-                                             void* stream) {
-    QT_REQUIRE(n_tokens >= 0 && width > 0 && eps > 0.f, "linear_attention_gate_norm: bad sizes T=%d width=%d", n_tokens, width);
-    QT_REQUIRE(!proj || (at_gate >= 0 && at_gate + width <= proj_cols && n_splits >= 1), "linear_attention_gate_norm: gate columns outside the projection");
+extern "C" int qt_group_gate_norm(const float* o, const float* x, int x_cols, int at_x, const float* skip, int skips, const float* proj, int n_splits,
+                                  long long split_stride, int proj_cols, int at_gate, const float* weight, int weight_len, float eps, float scale,
+                                  int groups, int silu, int gate_first, void* out, int out_dtype, int n_tokens, int width, void* stream) {
+    QT_REQUIRE(n_tokens >= 0 && width > 0 && groups > 0 && width % groups == 0 && eps > 0.f, "group_gate_norm: bad sizes T=%d width=%d in %d parts", n_tokens, width, groups);
+    QT_REQUIRE(weight_len == width || weight_len == width / groups, "group_gate_norm: a weight of %d for %d columns in %d parts", weight_len, width, groups);
+    QT_REQUIRE(!proj || (at_gate >= 0 && at_gate + width <= proj_cols && n_splits >= 1), "group_gate_norm: gate columns outside the projection");
+    QT_REQUIRE(!x || (skip && skips > 0 && width % skips == 0 && at_x >= 0 && at_x + width <= x_cols), "group_gate_norm: the skip term's operands do not fit");
     if (n_tokens == 0) return QT_OK;
     cudaStream_t s = (cudaStream_t)stream;
-    const int threads = width >= 1024 ? 256 : 128;
-    return QT_DISPATCH_DTYPE(out_dtype, "linear_attention_gate_norm", {
-        launch_kernel(linear_attention_gate_norm_kernel<T>, dim3(n_tokens), dim3(threads), 0, s, o, proj, n_splits, (size_t)split_stride, proj_cols,
-                      at_gate, weight, eps, scale, (T*)out, width);
-        QT_CHECK_LAUNCH("linear_attention_gate_norm");
+    const int part = width / groups;
+    GroupNormParams p{o, x, x_cols, at_x, skip, x ? width / skips : 1, proj, n_splits, (size_t)split_stride, proj_cols, at_gate, weight, weight_len, eps, scale,
+                      width, part, silu, gate_first};
+    return QT_DISPATCH_DTYPE(out_dtype, "group_gate_norm", {
+        if (groups > 1 && part <= 32 * GN_CACHE) {
+            launch_kernel(group_gate_norm_kernel<T, true>, dim3(n_tokens, (groups + 3) / 4), dim3(128), 0, s, p, (T*)out);
+        } else {
+            int threads = ((part + GN_CACHE * 32 - 1) / (GN_CACHE * 32)) * 32;      // 8 elements a thread; few tokens: fewer each
+            if (n_tokens < 256) threads = ((part + 63) / 64) * 32;
+            threads = threads < 128 ? 128 : threads > 1024 ? 1024 : threads;
+            launch_kernel(group_gate_norm_kernel<T, false>, dim3(n_tokens, groups), dim3(threads), 0, s, p, (T*)out);
+        }
+        QT_CHECK_LAUNCH("group_gate_norm");
         return QT_OK;
     });
 }

@@ -7,6 +7,9 @@
 //                        first nq * d channels are the queries (written to q_out), the next nkv * d the keys (written
 //                        into the paged cache at the token's position).  Values are the keys, so nothing else is stored.
 // conv_keep_kernel       kept[slot] <- the raw inputs of the sequence's last n - 1 positions after this step.
+// conv_act_kernel        the same convolution with a bias and SiLU behind it, for a recurrent mixer whose channels lead nothing
+//                        but its recurrence: float rows out.  Beside it the step sizes of the recurrence's heads,
+//                        softplus(. + bias_h), and the logarithms of their decays, -exp(rate_h) times the step size.
 // gate_mul_kernel        x[t][c] *= sigmoid(sum_s gate[s][t][offset + c]): a gate computed from the mixer's input by one
 //                        more block of rows of the first projection.  With `group` > 1 every `group` consecutive
 //                        columns share one gate column (one number per head).
@@ -108,6 +111,120 @@ extern "C" int qt_conv_qk_write(const float* proj, int n_splits, long long split
     if (rc) return rc;
     if (n_taps > 1) {
         launch_kernel(conv_keep_kernel, dim3((channels + 127) / 128, n_seqs), dim3(128), 0, s, proj, n_splits, (size_t)split_stride, proj_cols,
+                      kept, seq_start, slots, channels, n_taps);
+        QT_CHECK_LAUNCH("conv_keep");
+    }
+    return QT_OK;
+}
+
+// ----------------------------------------------------------------------------- convolution, bias and SiLU of a recurrence's channels
+struct ConvActParams {
+    const float* proj; int n_splits; size_t split_stride; int proj_cols;   // [splits, T, proj_cols]
+    int at, channels;                 // the convolved columns
+    const float* taps;                // [channels, n_taps], the last column is the current token's
+    const float* bias;                // [channels] or null
+    float* kept;                      // [slots + 1, max(n_taps - 1, 1), channels]
+    const int* token_seq; const int* seq_start; const int* slots;
+    float* out;                       // [T, channels]
+    int at_step, heads;               // the columns of the heads' step sizes (heads 0: none)
+    const float* step_bias; const float* rate_log;       // [heads]
+    float* step; float* log_decay;    // [T, heads]
+    int n_tokens, n_taps, keep;       // keep: every sequence brings one token, and its kept inputs are shifted here
+};
+
+constexpr int CA_TOKENS = 8;          // consecutive tokens of a channel that one thread walks
+
+__device__ __forceinline__ float conv_silu(float y) { return y / (1.f + expf(-y)); }
+
+// grid (blocks of 128 columns: the channels, then the heads; runs of CA_TOKENS tokens).  TAPS > 0: the inputs of the last TAPS
+// tokens stay in registers from token to token; 0: any number of taps, read again for every token.
+template <int TAPS>
+__global__ void __launch_bounds__(128) conv_act_kernel(const ConvActParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    const int t0 = blockIdx.y * CA_TOKENS, t1 = min(p.n_tokens, t0 + CA_TOKENS);
+    if (c >= p.channels) {
+        const int h = c - p.channels;
+        if (h >= p.heads) return;
+        const float rate = -expf(p.rate_log[h]), b = p.step_bias[h];
+        for (int t = t0; t < t1; ++t) {
+            const float z = sum_splits(p.proj, (size_t)t * p.proj_cols + p.at_step + h, p.n_splits, p.split_stride) + b;
+            const float dt = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+            p.step[(size_t)t * p.heads + h] = dt;
+            p.log_decay[(size_t)t * p.heads + h] = rate * dt;
+        }
+        return;
+    }
+    const int n_taps = TAPS > 0 ? TAPS : p.n_taps, rows = n_taps - 1;
+    const float b = p.bias ? p.bias[c] : 0.f;
+    auto input = [&](int seq, int row0, int from) -> float {          // the channel's input at index `from` of the step's tokens of a sequence
+        return from >= 0 ? sum_splits(p.proj, (size_t)(row0 + from) * p.proj_cols + p.at + c, p.n_splits, p.split_stride)
+                         : p.kept[((size_t)p.slots[seq] * rows + rows + from) * p.channels + c];
+    };
+    if (TAPS > 0) {
+        constexpr int N = TAPS > 0 ? TAPS : 1;
+        float w[N], u[N];
+#pragma unroll
+        for (int j = 0; j < N; ++j) w[j] = p.taps[(size_t)c * N + j];
+        int before = -1;
+        for (int t = t0; t < t1; ++t) {
+            const int seq = p.token_seq[t], row0 = p.seq_start[seq], local = t - row0;
+            if (seq != before) {
+#pragma unroll
+                for (int j = 0; j < N; ++j) u[j] = input(seq, row0, local - (N - 1) + j);
+                before = seq;
+            } else {
+#pragma unroll
+                for (int j = 0; j + 1 < N; ++j) u[j] = u[j + 1];
+                u[N - 1] = input(seq, row0, local);
+            }
+            float y = 0.f;
+#pragma unroll
+            for (int j = 0; j < N; ++j) y += w[j] * u[j];
+            p.out[(size_t)t * p.channels + c] = conv_silu(y + b);
+            if (p.keep) {
+                float* mine = p.kept + (size_t)p.slots[seq] * rows * p.channels + c;
+#pragma unroll
+                for (int j = 0; j + 1 < N; ++j) mine[(size_t)j * p.channels] = u[j + 1];
+            }
+        }
+    } else {
+        for (int t = t0; t < t1; ++t) {
+            const int seq = p.token_seq[t], row0 = p.seq_start[seq], local = t - row0;
+            float y = 0.f;
+            for (int j = 0; j < n_taps; ++j) y += p.taps[(size_t)c * n_taps + j] * input(seq, row0, local - rows + j);
+            p.out[(size_t)t * p.channels + c] = conv_silu(y + b);
+        }
+    }
+}
+
+extern "C" int qt_conv_act(const float* proj, int n_splits, long long split_stride, int proj_cols, int at, int channels, const float* taps,
+                           const float* bias, float* kept, const int* token_seq, const int* seq_start, const int* slots, float* out,
+                           int at_step, int heads, const float* step_bias, const float* rate_log, float* step, float* log_decay, int n_tokens,
+                           int n_seqs, int n_taps, int one_token, void* stream) {
+    QT_REQUIRE(n_tokens >= 0 && n_seqs >= 0 && channels > 0 && heads >= 0 && n_splits >= 1, "conv_act: bad sizes");
+    QT_REQUIRE(n_taps >= 1 && n_taps <= MAX_TAPS, "conv_act: %d taps (1..%d)", n_taps, MAX_TAPS);
+    QT_REQUIRE(at >= 0 && at + channels <= proj_cols && (heads == 0 || (at_step >= 0 && at_step + heads <= proj_cols)),
+               "conv_act: %d channels at %d and %d heads at %d of %d columns", channels, at, heads, at_step, proj_cols);
+    QT_REQUIRE(heads == 0 || (step_bias && rate_log && step && log_decay), "conv_act: step sizes without their operands");
+    QT_REQUIRE(n_seqs <= 65535 && (n_tokens + CA_TOKENS - 1) / CA_TOKENS <= 65535, "conv_act: too many tokens or sequences for one launch");
+    if (n_tokens == 0) return QT_OK;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int keep = one_token && n_taps <= 4 && n_tokens == n_seqs ? 1 : 0;
+    ConvActParams p{proj, n_splits, (size_t)split_stride, proj_cols, at, channels, taps, bias, kept, token_seq, seq_start, slots, out,
+                    at_step, heads, step_bias, rate_log, step, log_decay, n_tokens, n_taps, keep};
+    const dim3 grid((channels + heads + 127) / 128, (n_tokens + CA_TOKENS - 1) / CA_TOKENS);
+    switch (n_taps) {
+        case 1: launch_kernel(conv_act_kernel<1>, grid, dim3(128), 0, s, p); break;
+        case 2: launch_kernel(conv_act_kernel<2>, grid, dim3(128), 0, s, p); break;
+        case 3: launch_kernel(conv_act_kernel<3>, grid, dim3(128), 0, s, p); break;
+        case 4: launch_kernel(conv_act_kernel<4>, grid, dim3(128), 0, s, p); break;
+        default: launch_kernel(conv_act_kernel<0>, grid, dim3(128), 0, s, p);
+    }
+    QT_CHECK_LAUNCH("conv_act");
+    if (n_taps > 1 && !keep) {
+        launch_kernel(conv_keep_kernel, dim3((channels + 127) / 128, n_seqs), dim3(128), 0, s, proj + at, n_splits, (size_t)split_stride, proj_cols,
                       kept, seq_start, slots, channels, n_taps);
         QT_CHECK_LAUNCH("conv_keep");
     }

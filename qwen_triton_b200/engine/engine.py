@@ -99,7 +99,7 @@ class Engine:
         # host than they run on the device.  A part whose step only launches kernels says so (graph_safe = True;
         # a block answers for the parts it runs); one part that does not, or touches the host, and every step
         # launches its kernels one by one.
-        stepped = [self.model.embedding, *self.model.blocks, self.model.final_norm, self.model.head]
+        stepped = [self.model.embedding, *self.model.entries, *self.model.blocks, self.model.final_norm, self.model.head]
         self._graphs_enabled = bool(cuda_graphs) and all(getattr(part, "graph_safe", False) for part in stepped)
         # captured steps by shape, least recently used first; at most ``max_graphs`` are kept (a long generation at
         # many batch sizes and context buckets would otherwise grow device memory without limit), and all of them

@@ -2,7 +2,7 @@
 
 Counterpart: QwenTritonModel / QwenTritonForCausalLM (qwen_triton/models/core.py:156-263), whose
 layer loop (:230-240) runs each layer once in index order; here the order is the spec's
-``schedule``.  The final norm and the head run only on the rows whose logits are wanted (the
+``schedule``, in which a call may have a stream map in front of it.  The final norm and the head run only on the rows whose logits are wanted (the
 reference norms every row and then slices, :242,360-364; RMSNorm is row-wise, so the values agree).
 """
 from __future__ import annotations
@@ -19,6 +19,8 @@ def expected_tensors(spec: ModelSpec) -> dict[str, TensorSpec]:
     out: dict[str, TensorSpec] = {}
     out.update(part_class("embedding", spec.embedding).expected_tensors(spec.embedding.params, spec.vocab_size,
                                                                         spec.hidden_size))
+    for entry in spec.entries:
+        out.update(part_class("stream_map", entry).expected_tensors(entry.params))
     for layer in spec.layers:
         out.update(part_class("block", layer.block).expected_tensors(layer))
     out.update(part_class("norm", spec.final_norm).expected_tensors(spec.final_norm.params, spec.final_norm["name"]))
@@ -34,12 +36,17 @@ class CausalLM:
         self.embedding = part_class("embedding", spec.embedding)(spec.embedding.params, spec.vocab_size,
                                                                  spec.hidden_size, runtime)
         self.blocks = [part_class("block", layer.block)(layer, runtime) for layer in spec.layers]
+        self.entries = [part_class("stream_map", entry)(entry.params, runtime) for entry in spec.entries]
         self.final_norm = part_class("norm", spec.final_norm)(spec.final_norm.params, spec.final_norm["name"], runtime)
         self.head = part_class("head", spec.head)(spec.head.params, spec.vocab_size, spec.hidden_size, runtime)
         runtime.workspace.declare("residual", runtime.max_step_tokens * spec.hidden_size, torch.float32)
+        if self.entries:
+            runtime.workspace.declare("stream_start", runtime.max_step_tokens * spec.hidden_size, runtime.dtype)
 
     def load(self, source) -> None:
         self.embedding.load(source)
+        for entry in self.entries:
+            entry.load(source)
         for block in self.blocks:
             block.load(source)
         self.final_norm.load(source)
@@ -72,15 +79,21 @@ class CausalLM:
                     if key in ("runtime", "cos_sin"):
                         continue
                     yield from walk(value, depth + 1)
-        for part in (self.embedding, *self.blocks, self.final_norm, self.head):
+        for part in (self.embedding, *self.entries, *self.blocks, self.final_norm, self.head):
             yield from walk(part)
 
     def forward(self, ctx, cache, logits: torch.Tensor | None) -> None:
         """Run the tokens of ``ctx`` through every scheduled layer; write the logits of ``ctx.want_rows``."""
         hidden = self.spec.hidden_size
-        stream = ResidualStream(self.runtime.workspace.view("residual", ctx.n_tokens, hidden))
-        self.embedding.forward(ctx.token_ids, stream.residual)
+        ws = self.runtime.workspace
+        stream = ResidualStream(ws.view("residual", ctx.n_tokens, hidden), ws.view("stream_start", ctx.n_tokens, hidden) if self.entries else None)
+        if stream.start is not None:
+            self.embedding.forward(ctx.token_ids, stream.residual, stream.start)
+        else:
+            self.embedding.forward(ctx.token_ids, stream.residual)
         for position, call in enumerate(self.spec.schedule):
+            if call.entry is not None:
+                self.entries[call.entry].apply(stream)
             self.blocks[call.layer].forward(stream, ctx, cache.view(position))
         if logits is not None and ctx.n_want > 0:
             rows = self.final_norm.apply(stream, rows=ctx.want_rows)

@@ -22,7 +22,8 @@ _c_int, _c_ll, _c_float, _c_ptr = ctypes.c_int, ctypes.c_longlong, ctypes.c_floa
 
 _SIGNATURES = {
     "elementwise": {
-        "qt_embedding": [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr],
+        "qt_embedding": [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_float, _c_ptr, _c_ptr],
+        "qt_stream_concat": [_c_ptr, _c_ptr, _c_int, _c_int, _c_ll, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr],
         "qt_add_bias": [_c_ptr, _c_ptr, _c_int, _c_int, _c_ptr],
         "qt_add_rmsnorm": [_c_ptr, _c_ptr, _c_int, _c_int, _c_ll, _c_ptr, _c_float, _c_ptr, _c_int, _c_ptr, _c_int,
                            _c_int, _c_int, _c_ptr],
@@ -32,7 +33,7 @@ _SIGNATURES = {
         "qt_qk_norm_rope_write": [_c_ptr, _c_int, _c_int, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr,
                                   _c_int, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int,
                                   _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr],
-        "qt_swiglu": [_c_ptr, _c_int, _c_int, _c_ll, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr],
+        "qt_swiglu": [_c_ptr, _c_int, _c_int, _c_ll, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr],
         "qt_add_dyt": [_c_ptr, _c_ptr, _c_int, _c_ll, _c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_int, _c_ptr, _c_int,
                        _c_int, _c_ptr],
         "qt_map_difference": [_c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_ptr],
@@ -40,7 +41,7 @@ _SIGNATURES = {
     "delta_rule": {
         "qt_delta_prepare": [_c_ptr, _c_int, _c_ll, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
                              _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr],
-        "qt_lowrank": [_c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr],
+        "qt_lowrank": [_c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_float, _c_ptr, _c_int, _c_int, _c_int, _c_ptr],
         "qt_delta_scan": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
         "qt_gated_head_norm": [_c_ptr, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr],
         "qt_delta_scan_chunked": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
@@ -50,8 +51,18 @@ _SIGNATURES = {
         "qt_linear_attention_scan": [_c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int,
                                      _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
         "qt_linear_attention_prepare": [_c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr],
-        "qt_linear_attention_gate_norm": [_c_ptr, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_ptr, _c_float, _c_float, _c_ptr, _c_int, _c_int,
-                                          _c_int, _c_ptr],
+        "qt_decayed_attention_steps": [_c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_float, _c_ptr, _c_ptr, _c_ptr,
+                                       _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
+        # o, x, x_cols, at_x, skip, skips, proj, n_splits, split_stride, proj_cols, at_gate, weight, weight_len, eps, scale, groups, silu,
+        # gate_first, out, out_dtype, n_tokens, width, stream
+        "qt_group_gate_norm": [_c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_ptr, _c_int, _c_float, _c_float,
+                               _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr],
+    },
+    "linear_attention_chunk": {
+        # rows, cols, at_q, at_k, at_v, log_decay, per_channel, v_scale, out_scale, state, out, seq_start, slots, n_seqs, max_tokens, heads,
+        # heads_per_key, dim, vdim, states, within, whole, q_from, k_to, stream
+        "qt_decayed_attention_chunked": [_c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_float, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
+                                         _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr],
     },
     "attention": {
         "qt_attention_prefill": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int,
@@ -69,6 +80,8 @@ _SIGNATURES = {
     "short_conv": {
         "qt_conv_qk_write": [_c_ptr, _c_int, _c_ll, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr,
                              _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
+        "qt_conv_act": [_c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr,
+                        _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr],
         "qt_gate_mul": [_c_ptr, _c_int, _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
     },
     "latent": {
@@ -77,18 +90,19 @@ _SIGNATURES = {
         "qt_latent_query_rot": [_c_ptr, _c_int, _c_int, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                                 _c_int, _c_ptr],
         "qt_head_product": [_c_ptr, _c_int, _c_int, _c_ll, _c_ll, _c_ll, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ll, _c_ll, _c_int,
-                            _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
+                            _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
     },
     "attention_latent": {
-        # q, cache, out, block_table, max_blocks, seq_start, seq_past, seq_len, n_seqs, max_q_len, heads, row, rank, page_tokens, scale,
-        # n_splits, part_acc, part_ml, stream
+        # q, cache, out, block_table, max_blocks, seq_start, seq_past, seq_len, n_seqs, max_q_len, heads, row, rank, page_tokens, window,
+        # ring_tokens, scale, n_splits, part_acc, part_ml, stream
         "qt_attention_latent": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                                _c_float, _c_int, _c_ptr, _c_ptr, _c_ptr],
+                                _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_ptr],
     },
     "experts": {
         "qt_experts_by_pair": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int,
                                _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_int, _c_float, _c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_ptr],
-        "qt_route_top": [_c_ptr, _c_int, _c_ll, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr],
+        "qt_route_top": [_c_ptr, _c_int, _c_ll, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_int,
+                         _c_ptr],
         "qt_experts_route": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                              _c_int, _c_ptr, _c_ptr],
         "qt_experts_combine": [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr],
@@ -113,14 +127,14 @@ _SIGNATURES = {
         "qt_gemm_simt": [_c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr],
     },
     "gemm_tc": {
-        "qt_gemm_tc": [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_ptr],
+        "qt_gemm_tc": [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_ptr, _c_ptr],
         "qt_gemm_tc_pair": [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_ll, _c_int, _c_ptr,
-                            _c_ptr, _c_int, _c_ptr, _c_ptr],
+                            _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr],
         "qt_gemm_tc_pair_slots": [],
     },
     "gemm_fused": {
         "qt_gemm_fused": [_c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                          _c_ptr, _c_int, _c_int, _c_float,
+                          _c_ptr, _c_int, _c_int, _c_float, _c_ptr,
                           _c_ptr, _c_int, _c_int, _c_float,
                           _c_ptr, _c_ptr, _c_ptr, _c_ptr,
                           _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_float,
@@ -243,16 +257,35 @@ class GemmOut:
 
 
 # ----------------------------------------------------------------------------- elementwise
-def embedding(residual: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, scale: float = 1.0) -> None:
-    """residual[t] = table[ids[t]] * scale in float.  ids: int32 [T]."""
+def embedding(residual: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, scale: float = 1.0, norm_weight: torch.Tensor | None = None,
+              eps: float = 0.0, start: torch.Tensor | None = None) -> None:
+    """residual[t] = table[ids[t]] * scale in float, RMS-normed with ``norm_weight`` [H] where given.  ids: int32 [T].
+    ``start`` [T, H] (the table's type) receives a copy of the result."""
     tokens, hidden = residual.shape
     _need(residual, "residual", torch.float32)
     _need(table, "table")
     _need(ids, "ids", torch.int32, (tokens,))
     if table.shape[1] != hidden:
         raise KernelError(f"embedding: table width {table.shape[1]} != stream width {hidden}")
+    if norm_weight is not None:
+        _need(norm_weight, "norm_weight", torch.float32, (hidden,))
+    if start is not None:
+        _need(start, "start", table.dtype, (tokens, hidden))
     _call("elementwise", "qt_embedding", _ptr(residual), _ptr(table), _ptr(ids), tokens, hidden, table.shape[0],
-          _code(table, "table"), float(scale), _stream())
+          _code(table, "table"), float(scale), _ptr(norm_weight), float(eps), _ptr(start), _stream())
+
+
+def stream_concat(residual: torch.Tensor, delta: GemmOut | None, start: torch.Tensor, out: torch.Tensor) -> None:
+    """out [T, 2 H] = [stream + delta | start] in ``start``'s type, and the stream is set to zero: what a map of these rows
+    returns is added to it as any other addition."""
+    tokens, hidden = residual.shape
+    _need(residual, "residual", torch.float32)
+    _need(start, "start", shape=(tokens, hidden))
+    _need(out, "out", start.dtype, (tokens, 2 * hidden))
+    if delta is not None and (not delta.tensor.is_cuda or (delta.rows, delta.cols) != (tokens, hidden)):
+        raise KernelError(f"stream_concat: delta {tuple(delta.tensor.shape)} does not match the stream {tuple(residual.shape)}")
+    _call("elementwise", "qt_stream_concat", _ptr(residual), _ptr(delta.tensor) if delta else None, _code(delta.tensor, "delta") if delta else F32,
+          delta.n_splits if delta else 1, delta.split_stride if delta else 0, _ptr(start), _ptr(out), _code(start, "start"), tokens, hidden, _stream())
 
 
 def add_bias(out: torch.Tensor, bias: torch.Tensor) -> None:
@@ -496,6 +529,33 @@ def conv_qk_write(proj: GemmOut, taps: torch.Tensor, kept: torch.Tensor, ctx, q_
           1 if write_kv else 0, _stream(), launches=2 if n_taps > 1 else 1)
 
 
+def conv_act(proj: GemmOut, at: int, taps: torch.Tensor, bias: torch.Tensor | None, kept: torch.Tensor, ctx, out: torch.Tensor, at_step: int = 0,
+             step_bias: torch.Tensor | None = None, rate_log: torch.Tensor | None = None, step: torch.Tensor | None = None,
+             log_decay: torch.Tensor | None = None) -> None:
+    """A short causal convolution over time with a bias and SiLU behind it, in float, on columns ``at`` .. of ``proj`` (float
+    sums [*, T, cols]) into ``out`` [T, channels]; taps and kept inputs as for ``conv_qk_write``.  With ``step`` [T, heads] also the
+    step sizes softplus(columns ``at_step`` .. + ``step_bias``) and, in ``log_decay``, -exp(``rate_log``) times them."""
+    tokens, channels = out.shape
+    n_taps = taps.shape[1]
+    heads = step.shape[1] if step is not None else 0
+    _need(proj.tensor, "proj", torch.float32)
+    _need(taps, "taps", torch.float32, (channels, n_taps))
+    _need(out, "out", torch.float32, (proj.rows, channels))
+    if bias is not None:
+        _need(bias, "bias", torch.float32, (channels,))
+    _need(kept, "kept", torch.float32)
+    if tuple(kept.shape[1:]) != (max(n_taps - 1, 1), channels):
+        raise KernelError(f"conv_act: kept inputs {tuple(kept.shape)} are not [slots, {max(n_taps - 1, 1)}, {channels}]")
+    if step is not None:
+        for name, tensor, shape in (("step", step, (tokens, heads)), ("log_decay", log_decay, (tokens, heads)), ("step_bias", step_bias, (heads,)),
+                                    ("rate_log", rate_log, (heads,))):
+            _need(tensor, name, torch.float32, shape)
+    one_token = bool(ctx.is_decode)
+    _call("short_conv", "qt_conv_act", _ptr(proj.tensor), proj.n_splits, proj.split_stride, proj.cols, int(at), channels, _ptr(taps), _ptr(bias), _ptr(kept),
+          _ptr(ctx.token_seq), _ptr(ctx.seq_start), _ptr(ctx.slots), _ptr(out), int(at_step), heads, _ptr(step_bias), _ptr(rate_log), _ptr(step),
+          _ptr(log_decay), tokens, ctx.n_seqs, n_taps, 1 if one_token else 0, _stream(), launches=1 if n_taps == 1 or (one_token and n_taps <= 4) else 2)
+
+
 def gate_mul(x: torch.Tensor, gate: GemmOut, offset: int, group: int = 1) -> None:
     """x [T, N] *= sigmoid(columns ``offset`` .. ``offset + N`` of ``gate``), in float, in place.  With ``group`` > 1 every
     ``group`` consecutive columns of x share one gate column (one number per head): columns ``offset`` .. ``offset + N / group``."""
@@ -556,11 +616,11 @@ def latent_query_rot(q: GemmOut, cos_sin: torch.Tensor | None, token_pos: torch.
 
 
 def head_product(x, weight: torch.Tensor, out: torch.Tensor, *, x_row: int, x_head: int, x_offset: int = 0, out_offset: int = 0,
-                 gate: GemmOut | None = None, gate_offset: int = 0) -> None:
+                 gate: GemmOut | None = None, gate_offset: int = 0, gate_per_head: bool = False) -> None:
     """A product per head: out[t, h, out_offset + n] = sum_k x[t, h, k] weight[h, n, k], every head with a matrix of its own,
     summed in float.  ``x`` is a tensor or a ``GemmOut`` (partial sums are added first) whose element (t, h, k) lies at
     t * x_row + h * x_head + x_offset + k; ``out`` is [T, heads, row].  With ``gate`` (float sums [*, T, cols]) the result
-    is multiplied by sigmoid(gate[t, gate_offset + h * N + n])."""
+    is multiplied by sigmoid(gate[t, gate_offset + h * N + n]), or with ``gate_per_head`` by sigmoid(gate[t, gate_offset + h])."""
     heads, n, k = weight.shape
     _need(weight, "weight")
     _need(out, "out")
@@ -577,7 +637,8 @@ def head_product(x, weight: torch.Tensor, out: torch.Tensor, *, x_row: int, x_he
     _call("latent", "qt_head_product", _ptr(x_tensor), _code(x_tensor, "x"), splits, stride, int(x_row), int(x_head), int(x_offset),
           _ptr(weight), _code(weight, "weight"), _ptr(out), _code(out, "out"), out.shape[1] * out.shape[2], out.shape[2], int(out_offset),
           _ptr(gate.tensor) if gate is not None else None, gate.n_splits if gate is not None else 1,
-          gate.split_stride if gate is not None else 0, gate.cols if gate is not None else 0, int(gate_offset), tokens, heads, n, k, _stream())
+          gate.split_stride if gate is not None else 0, gate.cols if gate is not None else 0, int(gate_offset), 1 if gate_per_head else 0, tokens,
+          heads, n, k, _stream())
 
 
 # ----------------------------------------------------------------------------- the gated delta rule
@@ -607,10 +668,11 @@ def delta_prepare(proj: GemmOut, taps: torch.Tensor, kept: torch.Tensor, ctx, q:
 
 
 def lowrank(proj: GemmOut, offset: int, weight: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None,
-            rate_log: torch.Tensor | None = None, per_rate: int = 0) -> None:
+            rate_log: torch.Tensor | None = None, per_rate: int = 0, power: float | None = None) -> None:
     """out [T, N] (float) = f(weight^T x + bias) for x = columns ``offset`` .. ``offset + rank`` of ``proj`` and
     ``weight`` [rank, N] (float, the second matrix of a projection through a few columns, transposed).  With
-    ``rate_log`` [N / per_rate] f is the logarithm of a decay, -exp(rate_log[n / per_rate]) * softplus(.); else the sigmoid."""
+    ``rate_log`` [N / per_rate] f is the logarithm of a decay, -exp(rate_log[n / per_rate]) * softplus(.); with ``power`` it is the
+    logarithm of sigmoid(.)^power; else the sigmoid."""
     rank, n_out = weight.shape
     _need(proj.tensor, "proj", torch.float32)
     _need(weight, "weight", torch.float32)
@@ -620,7 +682,8 @@ def lowrank(proj: GemmOut, offset: int, weight: torch.Tensor, out: torch.Tensor,
     if rate_log is not None:
         _need(rate_log, "rate_log", torch.float32, (n_out // max(per_rate, 1),))
     _call("delta_rule", "qt_lowrank", _ptr(proj.tensor), proj.n_splits, proj.split_stride, proj.cols, int(offset), rank, _ptr(weight),
-          _ptr(bias), _ptr(rate_log), int(per_rate), _ptr(out), proj.rows, n_out, 0 if rate_log is not None else 1, _stream())
+          _ptr(bias), _ptr(rate_log), int(per_rate), float(power or 0.0), _ptr(out), proj.rows, n_out,
+          0 if rate_log is not None else 2 if power is not None else 1, _stream())
 
 
 def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, state: torch.Tensor,
@@ -712,19 +775,89 @@ def linear_attention_prepare(proj: GemmOut, cols: int, out: torch.Tensor, act: b
     return GemmOut(out.view(1, proj.rows, int(cols)))
 
 
-def linear_attention_gate_norm(o: torch.Tensor, proj: GemmOut | None, at_gate: int, weight: torch.Tensor, eps: float, scale: float,
-                               out: torch.Tensor) -> None:
-    """out [T, N] = o / sqrt(mean(o^2) + eps) * weight * sigmoid(columns ``at_gate`` .. of ``proj``) * scale, the mean over the
-    token's whole row (all heads at once); o float, rounded once to ``out``'s type."""
+DECAY_CHUNK = 64            # tokens per chunk of the chunked recurrence
+_DECAY_FEW_TOKENS = 16      # steps in which no sequence brings more run token by token
+
+
+def decay_chunks(max_step_tokens: int) -> int:
+    """Chunks that a step's scratch holds: every token of a step in chunks, and a chunk of its own for up to 64 sequences' ends."""
+    return max_step_tokens // DECAY_CHUNK + 64
+
+
+def decay_scratch(max_step_tokens: int, heads: int, dim: int, vdim: int, per_channel: bool) -> dict[str, int]:
+    """Floats of the buffers that ``decayed_attention`` wants as scratch, by name."""
+    chunks = decay_chunks(max_step_tokens)
+    wide = dim if per_channel else 1
+    return {"states": chunks * heads * vdim * dim, "within": chunks * heads * DECAY_CHUNK * DECAY_CHUNK, "whole": chunks * heads * wide,
+            "q_from": max_step_tokens * heads * wide, "k_to": max_step_tokens * heads * wide}
+
+
+def decayed_attention(rows: GemmOut, at_q: int, at_k: int, at_v: int, log_decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, ctx,
+                      dim: int, scratch: dict[str, torch.Tensor] | None, heads_per_key: int = 1, v_scale: torch.Tensor | None = None,
+                      out_scale: float = 1.0, impl: str | None = None) -> None:
+    """Linear attention with decays that depend on the token, over the step's packed sequences: per head
+    S <- diag(exp(log_decay_t)) S + k_t (v_scale_t v_t)^T, o_t = out_scale S^T q_t, float throughout.  ``log_decay`` is
+    [T, heads, dim] (a decay per key channel) or [T, heads]; q, k ([heads / heads_per_key, dim]) and v ([heads, vdim]) are the
+    columns of ``rows`` (float sums [*, T, cols]) from ``at_q``, ``at_k``, ``at_v`` on; ``state`` [slots, heads, vdim, dim] (transposed)
+    is read and written at the rows ``ctx.slots`` names; ``out`` [T, heads, vdim].
+
+    Steps of few tokens a sequence run token by token ("steps"); long ones in chunks of 64 tokens ("chunks"), which needs
+    finished rows (one plane) and ``scratch`` (``decay_scratch``)."""
+    tokens, heads, vdim = out.shape
+    per_channel = log_decay.dim() == 3
+    _need(rows.tensor, "rows", torch.float32)
+    _need(out, "out", torch.float32)
+    _need(log_decay, "log_decay", torch.float32, (tokens, heads, dim) if per_channel else (tokens, heads))
+    _need(state, "state", torch.float32)
+    if v_scale is not None:
+        _need(v_scale, "v_scale", torch.float32, (tokens, heads))
+    if rows.rows != tokens or tuple(state.shape[1:]) != (heads, vdim, dim):
+        raise KernelError(f"decayed_attention: state {tuple(state.shape)} is not [slots, {heads}, {vdim}, {dim}], or {rows.rows} rows for {tokens} tokens")
+    needed = tokens // DECAY_CHUNK + ctx.n_seqs
+    fits = scratch is not None and rows.n_splits == 1 and scratch["states"].numel() >= needed * heads * vdim * dim
+    if impl == "chunks" and not fits:
+        raise KernelError("decayed_attention: the chunked form needs finished rows and scratch for every chunk")
+    if impl == "chunks" or (impl is None and fits and ctx.max_q_len > _DECAY_FEW_TOKENS):
+        for name, numel in (("within", needed * heads * DECAY_CHUNK * DECAY_CHUNK), ("whole", needed * heads * (dim if per_channel else 1)),
+                            ("q_from", log_decay.numel()), ("k_to", log_decay.numel())):
+            _need(scratch[name], name, torch.float32)
+            if scratch[name].numel() < numel:
+                raise KernelError(f"decayed_attention: the scratch buffer {name!r} holds {scratch[name].numel()} of {numel} floats")
+        _call("linear_attention_chunk", "qt_decayed_attention_chunked", _ptr(rows.tensor), rows.cols, int(at_q), int(at_k), int(at_v), _ptr(log_decay),
+              1 if per_channel else 0, _ptr(v_scale), float(out_scale), _ptr(state), _ptr(out), _ptr(ctx.seq_start), _ptr(ctx.slots), ctx.n_seqs,
+              int(ctx.max_q_len), heads, int(heads_per_key), int(dim), vdim, _ptr(scratch["states"]), _ptr(scratch["within"]), _ptr(scratch["whole"]),
+              _ptr(scratch["q_from"]), _ptr(scratch["k_to"]), _stream(), launches=4)
+        return
+    _call("linear_attention", "qt_decayed_attention_steps", _ptr(rows.tensor), rows.n_splits, rows.split_stride, rows.cols, int(at_q), int(at_k), int(at_v),
+          _ptr(log_decay), 1 if per_channel else 0, _ptr(v_scale), float(out_scale), _ptr(state), _ptr(out), _ptr(ctx.seq_start), _ptr(ctx.slots),
+          ctx.n_seqs, heads, int(heads_per_key), int(dim), vdim, _stream())
+
+
+def group_gate_norm(o: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, *, groups: int = 1, proj: GemmOut | None = None,
+                    at_gate: int = 0, gate: str = "sigmoid", gate_first: bool = False, x: torch.Tensor | None = None, at_x: int = 0,
+                    skip: torch.Tensor | None = None, scale: float = 1.0) -> None:
+    """What stands between a recurrence's output and the product behind it, for rows ``o`` [T, N] (float): y = o, plus
+    ``skip``[h] * x with ``x`` [T, cols] from column ``at_x`` on (h: which of the ``len(skip)`` equal parts); times the gate if
+    ``gate_first``; divided by the root mean square (``eps`` inside) of each of ``groups`` equal parts, times ``weight`` ([N], or
+    [N / groups] shared by the parts) and ``scale``; times the gate otherwise.  The gate is the sigmoid or ("silu") SiLU of
+    columns ``at_gate`` .. of ``proj`` (None: no gate).  Rounded once to ``out``'s type."""
     tokens, width = o.shape
     _need(o, "o", torch.float32)
-    _need(weight, "weight", torch.float32, (width,))
+    _need(weight, "weight", torch.float32)
     _need(out, "out", shape=(tokens, width))
+    if gate not in ("sigmoid", "silu"):
+        raise KernelError(f"group_gate_norm: gate {gate!r} is neither sigmoid nor silu")
     if proj is not None:
         _need(proj.tensor, "proj", torch.float32)
-    _call("linear_attention", "qt_linear_attention_gate_norm", _ptr(o), _ptr(proj.tensor) if proj is not None else None,
-          proj.n_splits if proj is not None else 1, proj.split_stride if proj is not None else 0, proj.cols if proj is not None else 0,
-          int(at_gate), _ptr(weight), float(eps), float(scale), _ptr(out), _code(out, "out"), tokens, width, _stream())
+    if x is not None:
+        _need(x, "x", torch.float32)
+        _need(skip, "skip", torch.float32)
+        if x.shape[0] != tokens:
+            raise KernelError(f"group_gate_norm: {x.shape[0]} rows of x for {tokens} tokens")
+    _call("linear_attention", "qt_group_gate_norm", _ptr(o), _ptr(x), x.shape[1] if x is not None else 0, int(at_x), _ptr(skip),
+          skip.numel() if skip is not None else 0, _ptr(proj.tensor) if proj is not None else None, proj.n_splits if proj is not None else 1,
+          proj.split_stride if proj is not None else 0, proj.cols if proj is not None else 0, int(at_gate), _ptr(weight), weight.numel(), float(eps),
+          float(scale), int(groups), 1 if gate == "silu" else 0, 1 if gate_first else 0, _ptr(out), _code(out, "out"), tokens, width, _stream())
 
 
 SWIGLU_GROUP = 16      # rows of gate and of up that alternate in a weight laid out for the GEMM's gated epilogue
@@ -756,15 +889,19 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor, group: int) -> torc
     return torch.stack((gate.view(inter // group, group, hidden), up.view(inter // group, group, hidden)), dim=1).reshape(2 * inter, hidden)
 
 
-def swiglu(gate_up: GemmOut, out: torch.Tensor, group: int = 0, activation: str = "silu", limit: float = 0.0) -> None:
+def swiglu(gate_up: GemmOut, out: torch.Tensor, group: int = 0, activation: str = "silu", limit: float = 0.0,
+           bias: torch.Tensor | None = None) -> None:
     """out[t, i] = act(gate[t, i]) * up[t, i] where gate_up[t] holds gate then up (``group`` 0) or alternates
-    ``group`` elements of gate and ``group`` of up; ``activation`` is one of ``ACTIVATIONS``."""
+    ``group`` elements of gate and ``group`` of up; ``activation`` is one of ``ACTIVATIONS``.  ``bias`` (float, one element
+    per column of gate_up) is added to the sums first."""
     tokens, inter = out.shape
+    if bias is not None:
+        _need(bias, "bias", torch.float32, (2 * inter,))
     _need(out, "out")
     if (gate_up.rows, gate_up.cols) != (tokens, 2 * inter):
         raise KernelError(f"swiglu: input {tuple(gate_up.tensor.shape)} does not match output {tuple(out.shape)}")
     _call("elementwise", "qt_swiglu", _ptr(gate_up.tensor), _code(gate_up.tensor, "gate_up"), gate_up.n_splits,
-          gate_up.split_stride, _ptr(out), _code(out, "out"), tokens, inter, int(group), activation_code(activation, True), float(limit),
+          gate_up.split_stride, _ptr(bias), _ptr(out), _code(out, "out"), tokens, inter, int(group), activation_code(activation, True), float(limit),
           _stream())
 
 
@@ -863,9 +1000,9 @@ def attention_latent_supported(q: torch.Tensor, k_cache: torch.Tensor, v_cache: 
                                ring_tokens: int, window, scale: float, penalty, chunk, keep_first: int, sink: bool, v_dim) -> bool:
     """The tensor-core kernel for cached latent rows takes bfloat16, one key head whose rows are the values' source
     too, rows and value sizes that are multiples of 8 (values up to 512, a row within shared memory), a positive
-    scale, pages of 64 tokens and a plain causal softmax."""
-    return (v_dim is not None and v_cache is k_cache and num_kv_heads == 1 and not ring_tokens and not window and penalty is None
-            and not chunk and not keep_first and not sink and scale > 0 and attention_latent_shape(q.dtype, q.shape[2], v_dim, page_tokens))
+    scale, pages of 64 tokens and a plain causal softmax, over all earlier keys or a window of them."""
+    return (v_dim is not None and v_cache is k_cache and num_kv_heads == 1 and ring_tokens % 64 == 0 and (not ring_tokens or bool(window))
+            and penalty is None and not chunk and not keep_first and not sink and scale > 0 and attention_latent_shape(q.dtype, q.shape[2], v_dim, page_tokens))
 
 
 def attention_latent_shape(dtype: torch.dtype, row: int, rank: int, page_tokens: int) -> bool:
@@ -874,12 +1011,12 @@ def attention_latent_shape(dtype: torch.dtype, row: int, rank: int, page_tokens:
             and 3 * 64 * (-(-row // 16) * 16 + 8) * 2 <= 227 * 1024 and not os.environ.get("QT_B200_LATENT_MMA", "1").startswith("0"))
 
 
-def _attention_latent(q, cache, out, block_table, seq_start, seq_past, seq_len, n_seqs, max_q_len, page_tokens, scale, v_dim, n_splits,
-                      part_acc, part_ml) -> None:
+def _attention_latent(q, cache, out, block_table, seq_start, seq_past, seq_len, n_seqs, max_q_len, page_tokens, window, ring_tokens, scale, v_dim,
+                      n_splits, part_acc, part_ml) -> None:
     _call("attention_latent", "qt_attention_latent", _ptr(q), _ptr(cache), _ptr(out), _ptr(block_table), block_table.shape[1],
           _ptr(seq_start) if seq_start is not None else None, _ptr(seq_past) if seq_past is not None else None,
-          _ptr(seq_len) if seq_len is not None else None, n_seqs, int(max_q_len), q.shape[1], q.shape[2], int(v_dim), page_tokens, float(scale),
-          int(n_splits), _ptr(part_acc) if n_splits > 1 else None, _ptr(part_ml) if n_splits > 1 else None, _stream())
+          _ptr(seq_len) if seq_len is not None else None, n_seqs, int(max_q_len), q.shape[1], q.shape[2], int(v_dim), page_tokens,
+          int(window or 0), int(ring_tokens), float(scale), int(n_splits), _ptr(part_acc) if n_splits > 1 else None, _ptr(part_ml) if n_splits > 1 else None, _stream())
 
 
 def attention_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor,
@@ -908,7 +1045,8 @@ def attention_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         _need(seq_past, "seq_past", torch.int32)
         if block_table.shape[0] < n_seqs:
             raise KernelError("attention_prefill: block table has fewer rows than sequences")
-        _attention_latent(q, k_cache, out, block_table, seq_start, seq_past, None, n_seqs, max_q_len, page_tokens, scale, v_dim, 1, None, None)
+        _attention_latent(q, k_cache, out, block_table, seq_start, seq_past, None, n_seqs, max_q_len, page_tokens, window, ring_tokens, scale, v_dim,
+                          1, None, None)
         return
     if impl == "latent":
         raise KernelError("the tensor-core kernel for cached latent rows does not take this call")
@@ -982,7 +1120,8 @@ def attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
             _need(part_ml, "part_ml", torch.float32)
             if part_acc.numel() < n_seqs * num_heads * n_splits * v_dim or part_ml.numel() < n_seqs * num_heads * n_splits * 2:
                 raise KernelError("attention_decode: scratch is too small for this batch and split count")
-        _attention_latent(q, k_cache, out, block_table, None, None, seq_len, n_seqs, 1, page_tokens, scale, v_dim, n_splits, part_acc, part_ml)
+        _attention_latent(q, k_cache, out, block_table, None, None, seq_len, n_seqs, 1, page_tokens, window, ring_tokens, scale, v_dim, n_splits,
+                          part_acc, part_ml)
         return
     if impl == "latent":
         raise KernelError("the tensor-core kernel for cached latent rows does not take this call")
@@ -1022,11 +1161,13 @@ def attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
 
 # ----------------------------------------------------------------------------- experts chosen by a table
 def route_top(logits: GemmOut, chosen: torch.Tensor, weights: torch.Tensor, gate: torch.Tensor | None, experts: int, scale: float,
-              normalize: bool = True) -> None:
+              normalize: bool = True, softmax: bool = False, groups: int = 1, keep_groups: int = 1) -> None:
     """A learned router's choice from float logits [*, T, cols]: scores = sigmoid(logits[:, :experts]); ``chosen``
     [T, top] (int32) the ``top`` largest, ``weights`` [T, top] their scores over their sum (+ 1e-20) times ``scale``;
     ``gate`` [T] = sigmoid(logits[:, experts]) where given (a shared expert's gate, one number per token).  Without
-    ``normalize`` the weights are the chosen scores themselves times ``scale``."""
+    ``normalize`` the weights are the chosen scores themselves times ``scale``.  ``softmax``: the scores are the softmax over
+    all experts.  ``groups`` > 1: only experts of the ``keep_groups`` groups (equal runs of neighbours) whose largest score is
+    largest can be chosen."""
     tokens, top = chosen.shape
     _need(logits.tensor, "logits", torch.float32)
     _need(chosen, "chosen", torch.int32, (logits.rows, top))
@@ -1034,7 +1175,7 @@ def route_top(logits: GemmOut, chosen: torch.Tensor, weights: torch.Tensor, gate
     if gate is not None:
         _need(gate, "gate", torch.float32, (tokens,))
     _call("experts", "qt_route_top", _ptr(logits.tensor), logits.n_splits, logits.split_stride, logits.cols, _ptr(chosen), _ptr(weights),
-          _ptr(gate), tokens, int(experts), top, float(scale), 1 if normalize else 0, _stream())
+          _ptr(gate), tokens, int(experts), top, float(scale), 1 if normalize else 0, 1 if softmax else 0, int(groups), int(keep_groups), _stream())
 
 
 def _expert_extras(tokens: int, top: int, width: int, pair_weights, base: GemmOut | None, row_scale):
@@ -1259,12 +1400,12 @@ def gemm_tc_supported(a: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: GemmOut, token_tile: int | None = None, stages: int = 0,
-            swiglu: bool = False, activation: str = "silu", limit: float = 0.0) -> None:
+            swiglu: bool = False, activation: str = "silu", limit: float = 0.0, bias: torch.Tensor | None = None) -> None:
     """out = a [M, K] @ w [N, K]^T on the tcgen05 tensor cores; bfloat16 inputs, K a multiple of 8.
 
     ``out`` is [1, M, N] bfloat16 or float, or [splits, M, N] float for split-K partial sums.  With ``swiglu`` the
     rows of ``w`` alternate SWIGLU_GROUP of a gate and of an up projection and ``out`` [1, M, N / 2] (bfloat16)
-    receives act(gate) * up from the epilogue.
+    receives act(gate) * up from the epilogue.  ``bias`` [N] (float) is added to the sums (ahead of the gate).
     """
     _need(a, "a", torch.bfloat16)
     _need(w, "w", torch.bfloat16)
@@ -1280,7 +1421,13 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: GemmOut, token_tile: int | No
     tile = token_tile or tc_token_tile(rows)
     _call("gemm_tc", "qt_gemm_tc", _ptr(a), _ptr(w), _ptr(out.tensor), _code(out.tensor, "out"), rows, w.shape[0], k, tile,
           out.n_splits, out.split_stride, int(stages), 1 if swiglu else 0, activation_code(activation, True) if swiglu else 0,
-          float(limit), _ptr(_status_word(a.device)), _stream())
+          float(limit), _ptr(_product_bias(bias, w)), _ptr(_status_word(a.device)), _stream())
+
+
+def _product_bias(bias: torch.Tensor | None, w: torch.Tensor) -> torch.Tensor | None:
+    if bias is not None:
+        _need(bias, "bias", torch.float32, (w.shape[0],))
+    return bias
 
 
 _PAIR_TAIL: dict[int, tuple[torch.Tensor, torch.Tensor, int]] = {}
@@ -1308,14 +1455,15 @@ def pair_tail_mode() -> int:
 
 
 def gemm_tc_pair(a: torch.Tensor, w: torch.Tensor, out: GemmOut, swiglu: bool = False, activation: str = "silu",
-                 tail: int | None = None, limit: float = 0.0) -> None:
+                 tail: int | None = None, limit: float = 0.0, bias: torch.Tensor | None = None) -> None:
     """The same product by pairs of blocks on the two SMs of a TPC (tcgen05 cta_group::2): 256 weight rows x
     256 tokens per tile, each block staging half of both operands; one persistent pair per TPC with two
     accumulators in tensor memory.  Meant for many tokens; ``out`` may be [splits, M, N] float partial sums, which
     pays for a few hundred tokens whose tiles alone do not fill the TPCs.
 
     With ``swiglu`` the rows of ``w`` alternate SWIGLU_GROUP of a gate and of an up projection
-    (``interleave_gate_up``) and ``out`` [1, M, N / 2] receives act(gate) * up from the epilogue."""
+    (``interleave_gate_up``) and ``out`` [1, M, N / 2] receives act(gate) * up from the epilogue.  ``bias`` [N] (float) is
+    added to the sums (ahead of the gate)."""
     _need(a, "a", torch.bfloat16)
     _need(w, "w", torch.bfloat16)
     rows, k = a.shape
@@ -1331,7 +1479,7 @@ def gemm_tc_pair(a: torch.Tensor, w: torch.Tensor, out: GemmOut, swiglu: bool = 
     _call("gemm_tc", "qt_gemm_tc_pair", _ptr(a), _ptr(w), _ptr(out.tensor), _code(out.tensor, "out"), rows, w.shape[0], k,
           1 if swiglu else 0, activation_code(activation, True) if swiglu else 0, float(limit), out.n_splits, out.split_stride,
           tail, _ptr(slots) if slots is not None else None, _ptr(flags) if flags is not None else None, pairs,
-          _ptr(_status_word(a.device)), _stream())
+          _ptr(_product_bias(bias, w)), _ptr(_status_word(a.device)), _stream())
 
 
 def gemm_uses_pairs(a: torch.Tensor, w: torch.Tensor) -> bool:
@@ -1343,16 +1491,18 @@ def gemm_uses_pairs(a: torch.Tensor, w: torch.Tensor) -> bool:
     return a.shape[0] > _TC_TILES[-1] or (a.shape[0] > TC_MAX_BLOCK_TOKENS and w.shape[0] >= 128 * sm_count(a.device))
 
 
-def gemm(a: torch.Tensor, w: torch.Tensor, out: GemmOut) -> None:
-    """out = a @ w^T with the kernel that fits the element type and shape (a static choice):
+def gemm(a: torch.Tensor, w: torch.Tensor, out: GemmOut, bias: torch.Tensor | None = None) -> None:
+    """out = a @ w^T (+ ``bias`` [N], float, for float results) with the kernel that fits the element type and shape (a static choice):
     tensor cores for bfloat16 with 16-byte aligned rows, the FMA kernel for float32 and the rest."""
     if gemm_tc_supported(a, w):
         if gemm_uses_pairs(a, w):
-            gemm_tc_pair(a, w, out)         # more tokens than one block's tile: pairs of blocks, a third less operand traffic
+            gemm_tc_pair(a, w, out, bias=bias)         # more tokens than one block's tile: pairs of blocks, a third less operand traffic
         else:
-            gemm_tc(a, w, out)
+            gemm_tc(a, w, out, bias=bias)
     elif out.n_splits == 1:
         gemm_simt(a, w, out)
+        if bias is not None and out.rows:
+            add_bias(out.tensor[0], bias)
     else:
         raise KernelError("gemm: split-K output is only produced by the tensor-core kernel")
 
@@ -1403,7 +1553,7 @@ def fused_qkv_supported(head_dim: int, rotary_dim: int) -> bool:
 def _fused(x, w: torch.Tensor, splits: int, epilogue: int, *, out=None, residual=None, norm_w=None, xw=None, sq_out=None,
            q_out=None, k_cache=None, v_cache=None, token_seq=None, token_pos=None, block_table=None, q_w=None, k_w=None,
            qk_eps=0.0, cos_sin=None, nq=0, nkv=0, d=0, page_tokens=0, ring_tokens=0, write_kv=False, stages: int = 0,
-           act: int = 0, interleaved: bool = False, limit: float = 0.0) -> None:
+           act: int = 0, interleaved: bool = False, limit: float = 0.0, bias: torch.Tensor | None = None) -> None:
     scaled = x if isinstance(x, ScaledRows) else None
     a = scaled.tensor if scaled is not None else x
     _need(a, "x", torch.bfloat16)
@@ -1420,7 +1570,7 @@ def _fused(x, w: torch.Tensor, splits: int, epilogue: int, *, out=None, residual
     rotary_dim, max_pos = (0, 0) if cos_sin is None else (cos_sin.shape[1], cos_sin.shape[0])
     _call("gemm_fused", "qt_gemm_fused", _ptr(a), _ptr(w), rows, w.shape[0], k, tc_token_tile(rows), int(splits), int(stages), epilogue,
           _ptr(scaled.sq) if scaled is not None else None, scaled.sq.shape[0] if scaled is not None else 0,
-          scaled.width if scaled is not None else 0, float(scaled.eps) if scaled is not None else 0.0,
+          scaled.width if scaled is not None else 0, float(scaled.eps) if scaled is not None else 0.0, _ptr(_product_bias(bias, w)),
           _ptr(out), _CODES.get(out.dtype, -1) if out is not None else 0, int(act), float(limit),
           _ptr(residual), _ptr(norm_w), _ptr(xw), _ptr(sq_out),
           _ptr(q_out), _ptr(k_cache), _ptr(v_cache), _ptr(token_seq), _ptr(token_pos), _ptr(block_table),
@@ -1429,37 +1579,37 @@ def _fused(x, w: torch.Tensor, splits: int, epilogue: int, *, out=None, residual
           1 if interleaved else 0, _ptr(_status_word(a.device)), _stream())
 
 
-def gemm_fused_store(x, w: torch.Tensor, out: torch.Tensor, splits: int = 1, stages: int = 0) -> None:
-    """out [M, N] (float or bfloat16) = x w^T, times the rows' deferred norm factor if ``x`` is ``ScaledRows``."""
+def gemm_fused_store(x, w: torch.Tensor, out: torch.Tensor, splits: int = 1, stages: int = 0, bias: torch.Tensor | None = None) -> None:
+    """out [M, N] (float or bfloat16) = x w^T (+ ``bias``, float), times the rows' deferred norm factor if ``x`` is ``ScaledRows``."""
     _need(out, "out", shape=(x.shape[0], w.shape[0]))
-    _fused(x, w, splits, _EPI_STORE, out=out, stages=stages)
+    _fused(x, w, splits, _EPI_STORE, out=out, stages=stages, bias=bias)
 
 
 def gemm_fused_residual(x, w: torch.Tensor, residual: torch.Tensor, norm_weight: torch.Tensor | None = None,
                         eps: float = 0.0, xw: torch.Tensor | None = None, sq: torch.Tensor | None = None, splits: int = 1,
-                        stages: int = 0) -> "ScaledRows | None":
-    """residual [M, N] (float, in place) += x w^T.  With ``norm_weight`` [N] the RMSNorm that follows is prepared in
+                        stages: int = 0, bias: torch.Tensor | None = None) -> "ScaledRows | None":
+    """residual [M, N] (float, in place) += x w^T (+ ``bias`` [N], float).  With ``norm_weight`` [N] the RMSNorm that follows is prepared in
     the same launch: ``xw`` [M, N] = bf16(residual * norm_weight) and ``sq`` [ceil(N / 128), M] = the rows' sums of
     squares per 128 columns; returns them as ``ScaledRows`` for the product behind the norm."""
     rows, n = x.shape[0], w.shape[0]
     _need(residual, "residual", torch.float32, (rows, n))
     if norm_weight is None:
-        _fused(x, w, splits, _EPI_RESIDUAL, residual=residual, stages=stages)
+        _fused(x, w, splits, _EPI_RESIDUAL, residual=residual, stages=stages, bias=bias)
         return None
     _need(norm_weight, "norm_weight", torch.float32, (n,))
     _need(xw, "xw", torch.bfloat16, (rows, n))
     _need(sq, "sq", torch.float32, (-(-n // 128), rows))
-    _fused(x, w, splits, _EPI_RESIDUAL, residual=residual, norm_w=norm_weight, xw=xw, sq_out=sq, stages=stages)
+    _fused(x, w, splits, _EPI_RESIDUAL, residual=residual, norm_w=norm_weight, xw=xw, sq_out=sq, stages=stages, bias=bias)
     return ScaledRows(xw, sq, n, float(eps))
 
 
 def gemm_fused_swiglu(x, w: torch.Tensor, out: torch.Tensor, splits: int = 1, stages: int = 0, activation: str = "silu",
-                      limit: float = 0.0) -> None:
+                      limit: float = 0.0, bias: torch.Tensor | None = None) -> None:
     """out [M, N / 2] (bfloat16) = act(gate) * up for a weight whose rows alternate SWIGLU_GROUP of gate and of up."""
     if w.shape[0] % (2 * SWIGLU_GROUP):
         raise KernelError(f"gemm_fused_swiglu: {w.shape[0]} rows are not gate and up rows in groups of {SWIGLU_GROUP}")
     _need(out, "out", torch.bfloat16, (x.shape[0], w.shape[0] // 2))
-    _fused(x, w, splits, _EPI_SWIGLU, out=out, stages=stages, act=activation_code(activation, True), limit=limit)
+    _fused(x, w, splits, _EPI_SWIGLU, out=out, stages=stages, act=activation_code(activation, True), limit=limit, bias=bias)
 
 
 def gemm_fused_qkv(x, w: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor | None, v_cache: torch.Tensor | None,

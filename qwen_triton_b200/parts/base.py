@@ -22,6 +22,8 @@ Interfaces (what a new part must offer):
 * block:       ``forward(stream, ctx, cache) -> None``: arranges norm, mixer and feed-forward
   around the residual stream; ``cache_requests()`` says what it keeps per sequence: its mixer's
   request, or a list of requests if it has several such parts (``cache`` is then a tuple of views).
+* stream map:  ``apply(stream) -> None``: rewrites the residual stream in front of a scheduled call (``LayerCall.entry``), folding
+  what is pending; ``stream.start`` holds a copy of what the embedding put into the stream, in the activation dtype.
 * a part whose work in a step is kernel launches only (no host reads, no shapes that depend on data) may set
   ``graph_safe = True``; a block reports it for the parts it runs.  One-token steps are captured in CUDA graphs
   only if the embedding, every block, the final norm and the head say so.
@@ -37,7 +39,7 @@ from ..config.spec import PartSpec
 from ..ops.kernels import GemmOut, ScaledRows
 
 _REGISTRIES: dict[str, dict[str, type]] = {"norm": {}, "position": {}, "mixer": {}, "feed_forward": {}, "block": {},
-                                           "embedding": {}, "head": {}}
+                                           "embedding": {}, "head": {}, "stream_map": {}}
 
 
 def _register(family: str, kind: str, cls: type | None = None):
@@ -58,6 +60,7 @@ def register_feed_forward(kind: str, cls: type | None = None): return _register(
 def register_block(kind: str, cls: type | None = None): return _register("block", kind, cls)
 def register_embedding(kind: str, cls: type | None = None): return _register("embedding", kind, cls)
 def register_head(kind: str, cls: type | None = None): return _register("head", kind, cls)
+def register_stream_map(kind: str, cls: type | None = None): return _register("stream_map", kind, cls)
 
 
 def part_class(family: str, spec: PartSpec) -> type:
@@ -188,8 +191,9 @@ class ResidualStream:
     ``pending`` launches it and gives its result.
     """
 
-    def __init__(self, residual: torch.Tensor) -> None:
+    def __init__(self, residual: torch.Tensor, start: torch.Tensor | None = None) -> None:
         self.residual = residual
+        self.start = start                 # the stream as the embedding left it [T, H] (activation dtype), for models whose stream maps read it
         self._pending: GemmOut | DeferredProduct | None = None
         self.more: list[GemmOut] = []      # further additions beside ``pending`` (a block whose parts run side by side)
         self.post = None                   # a norm that the pending addition passes before it is added (``add(..., post=)``)

@@ -2,7 +2,8 @@
 here it is a parameter: any of ``kernels.ACTIVATIONS``, or ``kernels.CAPPED_GATE`` with ``limit``:
 g' = min(g, limit), u' = clamp(u, -limit, limit), y = g' sigmoid(1.702 g') (u' + 1), computed by the gate kernel
 in the same places as the other activations: the products' epilogues, or the gate kernel).  ``weight_suffix`` is what the tensor names add to the projections' names (default
-".weight"); ``float_out`` makes the down projection hand on float sums.
+".weight"); with ``bias`` the three projections have biases (tensor names: the projection's plus ``bias_suffix``, default
+".bias"), added in float ahead of the gate and to the down product's sums; ``float_out`` makes the down projection hand on float sums.
 
 gate and up run as one product over the fused weight [gate; up].  In bfloat16 its rows alternate 16 of gate and
 16 of up, so that the GEMM for many tokens can apply the SiLU gate in its epilogue (one warp then holds both halves
@@ -43,8 +44,10 @@ class GatedMLP:
         float_out = bool(params.get("float_out", False))
         key = str(params.get("buffers", "mlp"))           # several such parts in one layer keep their buffers apart
         self.gate_up = Linear(f"{key}.gate_up", 2 * self.inter, self.hidden, runtime, role="gate" if fused else "")
-        self.down = Linear(f"{key}.down" + (".float" if float_out else ""), self.hidden, self.inter, runtime,
-                           role="mlp_out", float_out=float_out)
+        self.biased = bool(params.get("bias", False))
+        self.down = Linear(f"{key}.down" + (".float" if float_out or self.biased else ""), self.hidden, self.inter, runtime,
+                           role="mlp_out", float_out=float_out, bias=self.biased)
+        self.gate_bias: torch.Tensor | None = None        # gate's and up's, in the layout of the fused weight's rows
         self.act_buffer = f"{key}.act"
         runtime.workspace.declare(self.act_buffer, runtime.max_step_tokens * self.inter, runtime.dtype)
         # few tokens: the gate in the epilogue of the gate/up product, which then also applies the factor of the norm
@@ -56,17 +59,26 @@ class GatedMLP:
         hidden, inter = int(params["hidden_size"]), int(params["intermediate_size"])
         n = cls._names(params)
         std = float(params.get("init_std", 0.02))
-        return {f"{prefix}.{n['gate']}": TensorSpec((inter, hidden), init_std=std),
-                f"{prefix}.{n['up']}": TensorSpec((inter, hidden), init_std=std),
-                f"{prefix}.{n['down']}": TensorSpec((hidden, inter), init_std=std)}
+        out = {f"{prefix}.{n['gate']}": TensorSpec((inter, hidden), init_std=std),
+               f"{prefix}.{n['up']}": TensorSpec((inter, hidden), init_std=std),
+               f"{prefix}.{n['down']}": TensorSpec((hidden, inter), init_std=std)}
+        if params.get("bias", False):
+            for key, size in (("gate_bias", inter), ("up_bias", inter), ("down_bias", hidden)):
+                out[f"{prefix}.{n[key]}"] = TensorSpec((size,), role="vector", init_std=0.1)
+        return out
 
     @staticmethod
     def _names(params) -> dict[str, str]:
-        suffix = str(params.get("weight_suffix", ".weight"))
-        return {k: params.get(k, f"{k}_proj") + suffix for k in ("gate", "up", "down")}
+        suffix, bias = str(params.get("weight_suffix", ".weight")), str(params.get("bias_suffix", ".bias"))
+        names = {k: params.get(k, f"{k}_proj") + suffix for k in ("gate", "up", "down")}
+        return {**names, **{f"{k}_bias": params.get(k, f"{k}_proj") + bias for k in ("gate", "up", "down")}}
 
     def load(self, source) -> None:
         n, p = self.names, self.prefix
+        if self.biased:
+            gate_b, up_b = (source(f"{p}.{n[k]}").float().reshape(-1, 1) for k in ("gate_bias", "up_bias"))
+            self.gate_bias = to_device(kernels.interleave_gate_up(gate_b, up_b, self.group).reshape(-1), torch.float32, self.runtime.device)
+            self.down.set_bias(source(f"{p}.{n['down_bias']}"))
         gate, up = source(f"{p}.{n['gate']}"), source(f"{p}.{n['up']}")
         self.gate_up.set_weight(kernels.interleave_gate_up(gate.to(self.runtime.dtype), up.to(self.runtime.dtype), self.group))
         self.down.set_weight(source(f"{p}.{n['down']}"))
@@ -75,16 +87,16 @@ class GatedMLP:
         tokens = x.shape[0]
         act = self.runtime.workspace.view(self.act_buffer, tokens, self.inter)
         if self.takes_scaled_rows and self.gate_up.fusable(tokens):
-            self.gate_up.into_swiglu(x, act, self.activation, self.limit)
+            self.gate_up.into_swiglu(x, act, self.activation, self.limit, self.gate_bias)
         elif self.group and kernels.gemm_uses_pairs(x, self.gate_up.weight):
             kernels.gemm_tc_pair(x, self.gate_up.weight, GemmOut(act.view(1, tokens, self.inter)), swiglu=True, activation=self.activation,
-                                 limit=self.limit)
+                                 limit=self.limit, bias=self.gate_bias)
         elif self.group and kernels.gemm_tc_supported(x, self.gate_up.weight) and self.gate_up.plan_splits(tokens) == 1:
             # a weight whose tiles fill the machine unsplit: the gate in the plain product's epilogue
             kernels.gemm_tc(x, self.gate_up.weight, GemmOut(act.view(1, tokens, self.inter)), swiglu=True, activation=self.activation,
-                            limit=self.limit)
+                            limit=self.limit, bias=self.gate_bias)
         else:
-            kernels.swiglu(self.gate_up(x), act, self.group, self.activation, self.limit)
+            kernels.swiglu(self.gate_up(x), act, self.group, self.activation, self.limit, self.gate_bias)
         # few tokens: the down projection is left to the norm behind it, which launches it with the residual addition
         # (and its own preparation) in the product's epilogue
         return DeferredProduct(self.down, act) if self.down.fusable(tokens) else self.down(act)
@@ -248,6 +260,9 @@ class RoutedExperts:
     ``shared`` (a dict: ``intermediate_size``, ``limit``) a further expert of the same form runs for every token and is
     added, times sigmoid(w_gate . h), one number per token; its gate is one more row of the router's product.
 
+    ``score`` = "softmax": the scores are softmax(z) over all experts.  ``groups`` > 1 (with ``keep_groups``): the experts form that
+    many equal groups of neighbours, a group's score is the largest in it, and only experts of the best ``keep_groups`` groups
+    can be chosen.
     ``normalize`` = False: the weights are the chosen scores themselves (times ``route_scale``), not divided by their sum.
     ``weight_on`` = "input": a pair's weight multiplies what its expert reads, not what it returns: the output is the sum of
     expert_e(w_e h), which for a gated expert is another function of w_e.  ``shared_gated`` = False: the shared expert is
@@ -280,6 +295,13 @@ class RoutedExperts:
             raise ValueError(f"{prefix}: gate activation {self.activation!r} is not one of {sorted(kernels.ACTIVATIONS) + [kernels.CAPPED_GATE]}")
         if not 0 < self.top <= self.experts:
             raise ValueError(f"{prefix}: {self.top} experts per token out of {self.experts}")
+        self.score = str(params.get("score", "sigmoid"))
+        if self.score not in ("sigmoid", "softmax"):
+            raise ValueError(f"{prefix}: router scores {self.score!r} are neither 'sigmoid' nor 'softmax'")
+        self.groups, self.keep_groups = int(params.get("groups", 1)), int(params.get("keep_groups", 1))
+        if self.groups < 1 or self.experts % self.groups or not 0 < self.keep_groups <= self.groups \
+                or self.top > self.keep_groups * (self.experts // self.groups):
+            raise ValueError(f"{prefix}: {self.top} experts out of the best {self.keep_groups} of {self.groups} groups of {self.experts}")
         self.normalize = bool(params.get("normalize", True))
         self.weight_on = str(params.get("weight_on", "output"))
         if self.weight_on not in ("output", "input"):
@@ -362,7 +384,8 @@ class RoutedExperts:
         chosen = ws.view("experts.chosen", tokens, self.top)
         weights = ws.view("experts.weights", tokens, self.top)
         gate = ws.view("experts.shared_gate", tokens) if self.shared is not None and self.shared_gated else None
-        kernels.route_top(self.router(x), chosen, weights, gate, self.experts, self.route_scale, self.normalize)
+        kernels.route_top(self.router(x), chosen, weights, gate, self.experts, self.route_scale, self.normalize, self.score == "softmax", self.groups,
+                          self.keep_groups)
         on_input = self.weight_on == "input"
         out_weights, in_weights = (None, weights) if on_input else (weights, None)
         base = None

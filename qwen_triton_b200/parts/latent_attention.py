@@ -4,8 +4,9 @@ all heads share, and every head expands its keys and values from the latent with
 From the mixer's input h: the query latent c_q = rms(W_dq h) w_q and q = W_uq c_q, laid out head by head as
 [``head_dim`` plain | ``rot_dim`` rotated]; W_dkv h = [``kv_rank`` | ``rot_dim``] rows, of which the first, RMS-normed with a
 weight, are the latent c and the last, rotated by the position encoding, the key part k_r shared by the heads.  Head h has
-k_h = W_uk_h c and v_h = W_uv_h c; its score is (q_plain_h . k_h + q_rot_h . k_r) * ``scale``, causal, plain softmax; the
-concatenated heads are multiplied by sigmoid(W_g h) and projected by W_o.  Only c and k_r are cached.
+k_h = W_uk_h c and v_h = W_uv_h c; its score is (q_plain_h . k_h + q_rot_h . k_r) * ``scale``, causal, over all earlier keys or
+the last ``window`` of them, plain softmax; the concatenated heads are multiplied by sigmoid(W_g h) (``gate`` true: one number
+per element; "head": one per head; false: none) and projected by W_o.  Only c and k_r are cached, under a window in a ring.
 
 What runs: since q_plain_h . (W_uk_h c) = (W_uk_h^T q_plain_h) . c, every head's query becomes
 [W_uk_h^T q_plain_h | q_rot_h] (a product per head, ``kernels.head_product``) and the attention kernels run all heads
@@ -20,7 +21,7 @@ Norms, rotation (float cos/sin table), scores, softmax and the gate are float; t
 rows and the heads' outputs are rounded to the activation type between the products.
 
 Parameters: ``hidden_size``, ``num_heads``, ``head_dim``, ``rot_dim``, ``v_head_dim``, ``q_rank``, ``kv_rank``, ``scale``, ``eps``,
-``position`` (a position part over ``rot_dim``), ``own_kv``, ``gate``, ``float_out``, and the tensor-name pieces ``dq``, ``uq``,
+``position`` (a position part over ``rot_dim``), ``window``, ``own_kv``, ``gate``, ``float_out``, and the tensor-name pieces ``dq``, ``uq``,
 ``dkv``, ``uk``, ``uv``, ``g``, ``o``, ``weight_suffix``, ``norm_suffix``.
 """
 from __future__ import annotations
@@ -30,7 +31,7 @@ import torch
 from ..ops import kernels
 from ..weights.tensors import TensorSpec
 from .attention import _MAX_SPLIT_PAIRS, _MIN_KEYS_PER_SPLIT
-from .base import KVRequest, Runtime, part_class, register_mixer, to_device
+from .base import DeferredProduct, KVRequest, Runtime, part_class, register_mixer, to_device
 from .linear import Linear
 
 
@@ -50,6 +51,8 @@ class LatentAttention:
         self.eps = float(params.get("eps", 1e-6))
         self.own_kv = bool(params.get("own_kv", True))
         self.gated = bool(params.get("gate", True))
+        self.head_gate = params.get("gate") == "head"
+        self.window = int(params["window"]) if params.get("window") else None
         position_spec = params["position"]
         self.position = part_class("position", position_spec)(position_spec.params, runtime)
         if getattr(self.position, "interleaved", False):
@@ -57,12 +60,12 @@ class LatentAttention:
         self.cos_sin = None
         self.at_kv = self.q_rank
         self.at_gate = self.q_rank + (self.row if self.own_kv else 0)
-        used = self.at_gate + (self.heads * self.dv if self.gated else 0)
+        used = self.at_gate + (self.heads * (1 if self.head_gate else self.dv) if self.gated else 0)
         self.proj_rows = -(-used // 8) * 8
         self.proj = Linear("latent.proj" + ("" if self.own_kv else ".reader"), self.proj_rows, self.hidden, runtime, float_out=True)
         self.uq = Linear("latent.uq", self.heads * (self.d + self.rot), self.q_rank, runtime)
         float_out = bool(params.get("float_out", False))
-        self.o = Linear("latent.o" + (".float" if float_out else ""), self.hidden, self.heads * self.dv, runtime, float_out=float_out)
+        self.o = Linear("latent.o" + (".float" if float_out else ""), self.hidden, self.heads * self.dv, runtime, float_out=float_out, role="attn_out")
         ws = runtime.workspace
         tokens = runtime.max_step_tokens
         ws.declare("latent.cq", tokens * self.q_rank, runtime.dtype)
@@ -91,7 +94,7 @@ class LatentAttention:
                n["uq"]: TensorSpec((heads * (d + rot), q_rank), init_std=std), n["uk"]: TensorSpec((heads * d, rank), init_std=std),
                n["uv"]: TensorSpec((heads * dv, rank), init_std=std), n["o"]: TensorSpec((hidden, heads * dv), init_std=std)}
         if params.get("gate", True):
-            out[n["g"]] = TensorSpec((heads * dv, hidden), init_std=std)
+            out[n["g"]] = TensorSpec((heads * (1 if params.get("gate") == "head" else dv), hidden), init_std=std)
         if params.get("own_kv", True):
             out[n["dkv"]] = TensorSpec((rank + rot, hidden), init_std=std)
             out[n["dkv_norm"]] = TensorSpec((rank,), role="vector", init_std=0.1, init_mean=1.0)
@@ -126,22 +129,23 @@ class LatentAttention:
 
     # ------------------------------------------------------------------ what it keeps per sequence
     def cache_request(self):
-        return KVRequest(1, self.row, None, shared_values=True)
+        return KVRequest(1, self.row, self.window, shared_values=True)
 
     def _splits(self, ctx, page_tokens: int) -> int:
         """Partial results per (sequence, head) of a one-token step.  The tensor-core kernel runs one block per SM, each
         with up to 64 heads of a sequence and a range of its pages; with at most 16 (32) heads a block cuts the keys of
         every page into 4 (2) parts, each a partial result of its own.  The generic kernel runs four heads a block,
         several blocks per SM."""
+        keys = min(ctx.max_context, self.window) if self.window else ctx.max_context
         if kernels.attention_latent_shape(self.runtime.dtype, self.row, self.rank, page_tokens) and self.scale > 0:
             parts = 4 if self.heads <= 16 else 2 if self.heads <= 32 else 1
             if parts * ctx.n_seqs > _MAX_SPLIT_PAIRS:
                 parts = 1
             blocks = ctx.n_seqs * -(-self.heads // 64)
-            most = max(1, min(ctx.max_context // _MIN_KEYS_PER_SPLIT, _MAX_SPLIT_PAIRS // (ctx.n_seqs * parts), 32))
+            most = max(1, min(keys // _MIN_KEYS_PER_SPLIT, _MAX_SPLIT_PAIRS // (ctx.n_seqs * parts), 32))
             return parts * max(1, min(most, self.runtime.sm_count // max(blocks, 1)))
         blocks = ctx.n_seqs * -(-self.heads // 4)
-        most = max(1, min(ctx.max_context // _MIN_KEYS_PER_SPLIT, _MAX_SPLIT_PAIRS // ctx.n_seqs, 32))
+        most = max(1, min(keys // _MIN_KEYS_PER_SPLIT, _MAX_SPLIT_PAIRS // ctx.n_seqs, 32))
         return max(1, min(most, (2 * self.runtime.sm_count) // max(blocks, 1)))
 
     # ------------------------------------------------------------------ run
@@ -162,13 +166,15 @@ class LatentAttention:
         kernels.latent_query_rot(q_full, self.cos_sin, ctx.token_pos, q, self.heads, self.d, self.rot, self.rank)
         out = ws.view("latent.ctx", tokens, self.heads, self.rank)
         if ctx.is_decode:
-            kernels.attention_decode(q, cache.k, cache.k, out, table, ctx.seq_len, 1, cache.page_tokens, cache.ring_tokens, None, self.scale,
+            kernels.attention_decode(q, cache.k, cache.k, out, table, ctx.seq_len, 1, cache.page_tokens, cache.ring_tokens, self.window, self.scale,
                                      self._splits(ctx, cache.page_tokens), ws.view("attn.part_acc", _MAX_SPLIT_PAIRS * self.heads * self.rank),
                                      ws.view("attn.part_ml", _MAX_SPLIT_PAIRS * self.heads * 2), v_dim=self.rank)
         else:
             kernels.attention_prefill(q, cache.k, cache.k, out, table, ctx.seq_start, ctx.seq_past, ctx.max_q_len, 1, cache.page_tokens,
-                                      cache.ring_tokens, None, self.scale, v_dim=self.rank)
+                                      cache.ring_tokens, self.window, self.scale, v_dim=self.rank)
         heads = ws.view("latent.heads", tokens, self.heads, self.dv)
         kernels.head_product(out, self.uv, heads, x_row=self.heads * self.rank, x_head=self.rank,
-                             gate=proj if self.gated else None, gate_offset=self.at_gate)
-        return self.o(heads.view(tokens, self.heads * self.dv))
+                             gate=proj if self.gated else None, gate_offset=self.at_gate, gate_per_head=self.head_gate)
+        heads = heads.view(tokens, self.heads * self.dv)
+        # few tokens: the product is left to the block, whose next norm launches it with the residual addition in its epilogue
+        return DeferredProduct(self.o, heads) if self.o.fusable(tokens) else self.o(heads)

@@ -109,7 +109,7 @@ class Linear:
         self.in_features = in_features
         self.runtime = runtime
         # a bias is added to the float sums (the first plane of a product split over K), so such a product stays float
-        # up to its consumer, and it keeps to the plain kernels: the fused products have no bias operand
+        # up to its consumer; the q/k/v product's fused epilogue has no bias operand, the others have
         self.has_bias = bias
         float_out = float_out or bias
         self.float_out = float_out
@@ -157,14 +157,14 @@ class Linear:
     @property
     def fused_capable(self) -> bool:
         """Whether this product has a fused form at all (known before the weight is loaded)."""
-        return bool(self.fused_plans) and bool(self.role) and kernels.fused_enabled(self.role) and not self.has_bias
+        return bool(self.fused_plans) and bool(self.role) and kernels.fused_enabled(self.role) and not (self.has_bias and self.role == "qkv")
 
     def fusable(self, rows: int) -> bool:
         """Whether ``rows`` tokens take the fused product (a static choice: element type, sizes, row count), in which
         what follows the product (residual add and norm preparation, SiLU gate, q/k-norm + rotation + cache write)
         runs in its epilogue.  ``QT_B200_FUSED=0`` in the environment turns it off."""
         return self.fused_capable and 0 < rows <= _FUSED_ROWS and self.weight is not None \
-            and kernels.fused_supported(self.weight)
+            and kernels.fused_supported(self.weight) and (self.role not in ("attn_out", "mlp_out") or self.out_features % 4 == 0)
 
     def _fused_splits(self, rows: int) -> int:
         return next(n for most, n in self.fused_plans if rows <= most)
@@ -188,11 +188,12 @@ class Linear:
     def into_residual(self, x: torch.Tensor, residual: torch.Tensor, norm_weight: torch.Tensor | None = None, eps: float = 0.0,
                       xw: torch.Tensor | None = None, sq: torch.Tensor | None = None) -> "ScaledRows | None":
         """residual += x W^T, and the norm behind it prepared (see ``kernels.gemm_fused_residual``)."""
-        return kernels.gemm_fused_residual(x, self.weight, residual, norm_weight, eps, xw, sq, splits=self._fused_splits(x.shape[0]), stages=self._fused_stages(x.shape[0]))
+        return kernels.gemm_fused_residual(x, self.weight, residual, norm_weight, eps, xw, sq, splits=self._fused_splits(x.shape[0]),
+                                           stages=self._fused_stages(x.shape[0]), bias=self._loaded_bias())
 
-    def into_swiglu(self, x, out: torch.Tensor, activation: str = "silu", limit: float = 0.0) -> None:
+    def into_swiglu(self, x, out: torch.Tensor, activation: str = "silu", limit: float = 0.0, bias: torch.Tensor | None = None) -> None:
         kernels.gemm_fused_swiglu(x, self.weight, out, splits=self._fused_splits(x.shape[0]), stages=self._fused_stages(x.shape[0]),
-                                  activation=activation, limit=limit)
+                                  activation=activation, limit=limit, bias=bias)
 
     def into_qkv(self, x, *args, **kwargs) -> None:
         kernels.gemm_fused_qkv(x, self.weight, *args, splits=self._fused_splits(x.shape[0]), stages=self._fused_stages(x.shape[0]), **kwargs)
@@ -206,8 +207,8 @@ class Linear:
         if isinstance(x, ScaledRows):
             # rows whose norm factor is still to be applied: the fused product's plain store applies it
             if out is None:
-                out = self.runtime.workspace.view(f"{self.key}.wide", rows, self.out_features)
-            kernels.gemm_fused_store(x, self.weight, out.view(rows, self.out_features), splits=self._fused_splits(rows))
+                out = self.runtime.workspace.view(f"{self.key}.out" if self.float_out else f"{self.key}.wide", rows, self.out_features)
+            kernels.gemm_fused_store(x, self.weight, out.view(rows, self.out_features), splits=self._fused_splits(rows), bias=self._loaded_bias())
             return GemmOut(out.view(1, rows, self.out_features))
         splits = self.plan_splits(rows)
         if out is None and splits > 1:
@@ -216,9 +217,10 @@ class Linear:
             result = GemmOut(self.runtime.workspace.view(f"{self.key}.out", 1, rows, self.out_features))
         else:
             result = GemmOut(out.view(1, rows, self.out_features))
-        kernels.gemm(x, self.weight, result)
-        if self.has_bias and rows:
-            if self.bias is None:
-                raise ValueError(f"{self.key}: the bias was not loaded")
-            kernels.add_bias(result.tensor[0], self.bias)
+        kernels.gemm(x, self.weight, result, self._loaded_bias())
         return result
+
+    def _loaded_bias(self) -> torch.Tensor | None:
+        if self.has_bias and self.bias is None:
+            raise ValueError(f"{self.key}: the bias was not loaded")
+        return self.bias

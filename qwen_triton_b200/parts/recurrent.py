@@ -31,6 +31,7 @@ from __future__ import annotations
 import torch
 
 from ..ops import kernels
+from ..ops.kernels import GemmOut
 from ..weights.tensors import TensorSpec
 from .base import DeferredProduct, Runtime, StateRequest, register_mixer, to_device
 from .linear import Linear
@@ -273,6 +274,230 @@ class LinearAttention:
         ready = kernels.linear_attention_prepare(proj, self.at_gate, ws.view("linattn.qkv", tokens, self.at_gate), self.act)
         kernels.linear_attention_scan(ready, 0, self.at_k, self.at_v, self.decay, cache.state, read, ctx, self.dim, False)
         normed = ws.view("linattn.normed", tokens, self.heads * self.vdim)
-        kernels.linear_attention_gate_norm(read.view(tokens, self.heads * self.vdim), proj if self.gated else None, self.at_gate, self.norm,
-                                           self.eps, 1.0, normed)
+        kernels.group_gate_norm(read.view(tokens, self.heads * self.vdim), self.norm, self.eps, normed, proj=proj if self.gated else None, at_gate=self.at_gate)
         return self.o(normed)
+
+
+class _DecayedMixer:
+    """What the mixers around ``kernels.decayed_attention`` share: its scratch, their output product and their checks."""
+
+    graph_safe = True
+
+    def _declare_scratch(self, per_channel: bool) -> None:
+        ws, tokens = self.runtime.workspace, self.runtime.max_step_tokens
+        self._scratch = {f"decayed.{name}": numel for name, numel in kernels.decay_scratch(tokens, self.heads, self.dim, self.vdim, per_channel).items()}
+        for name, numel in self._scratch.items():
+            ws.declare(name, numel, torch.float32)
+        ws.declare("decayed.read", tokens * self.heads * self.vdim, torch.float32)
+        ws.declare("decayed.normed", tokens * self.heads * self.vdim, self.runtime.dtype)
+
+    def _scratch_views(self) -> dict:
+        return {name.split(".", 1)[1]: self.runtime.workspace.view(name, numel) for name, numel in self._scratch.items()}
+
+    def _check(self, states) -> None:
+        if not states.writable:
+            raise ValueError(f"{self.prefix}: a recurrent mixer cannot read another layer's state")
+
+    def _output(self, normed, tokens: int):
+        # few tokens: the product is left to the block, whose next norm launches it with the residual addition in its epilogue
+        return DeferredProduct(self.o, normed) if self.o.fusable(tokens) else self.o(normed)
+
+
+@register_mixer("gated_linear_attention")
+class GatedLinearAttention(_DecayedMixer):
+    """Linear attention with a decay per key channel and token ("gated linear attention"):
+
+        S <- diag(alpha_t) S + k_t v_t^T;   o_t = dim^-1/2 S^T q_t
+
+    with q = W_q h, k = W_k h ([heads, dim]), v = W_v h ([heads, vdim]) and alpha = sigmoid(W_a2 (W_a1 h) + b)^(1/tau), [heads,
+    dim], a projection through few columns (the kernels pass its logarithm on).  Every head's o is RMS-normed over vdim with
+    a weight shared by the heads (``eps`` inside the root), the concatenated heads are multiplied by silu(W_g h) and projected
+    by W_o.  Per sequence the mixer keeps the states, float, zero for a new sequence, in the cache's per-slot state rows
+    (stored transposed, [heads, vdim, dim]).  The five projections of h run as one product with float sums; everything between
+    it and the output projection is float (``csrc/linear_attention.cu``, ``csrc/linear_attention_chunk.cu``, the narrow
+    projection in ``csrc/delta_rule.cu``).
+
+    Parameters: ``hidden_size``, ``num_heads``, ``head_dim``, ``v_head_dim``, ``tau``, ``decay_rank``, ``eps``, ``float_out``,
+    ``init_std``, and the tensor-name pieces ``q``, ``k``, ``v``, ``g``, ``o``, ``norm``, ``decay_in``, ``decay_out``, ``weight_suffix``,
+    ``bias_suffix``."""
+
+    def __init__(self, params, prefix: str, runtime: Runtime) -> None:
+        self.prefix, self.runtime, self.params = prefix, runtime, dict(params)
+        self.hidden = int(params["hidden_size"])
+        self.heads, self.dim = int(params["num_heads"]), int(params["head_dim"])
+        self.vdim = int(params.get("v_head_dim") or self.dim)
+        self.tau = float(params["tau"])
+        self.rank = int(params["decay_rank"])
+        self.eps = float(params.get("eps", 1e-6))
+        if self.dim > kernels.LINEAR_ATTENTION_MAX_DIM:
+            raise ValueError(f"{prefix}: {self.dim} key channels per head are beyond what the recurrence kernels hold "
+                             f"({kernels.LINEAR_ATTENTION_MAX_DIM})")
+        self.at_k = self.heads * self.dim
+        self.at_v = 2 * self.heads * self.dim
+        self.at_gate = self.at_v + self.heads * self.vdim
+        self.at_decay = self.at_gate + self.heads * self.vdim
+        self.proj_rows = -(-(self.at_decay + self.rank) // 8) * 8
+        self.proj = Linear("gla.proj", self.proj_rows, self.hidden, runtime, float_out=True)
+        float_out = bool(params.get("float_out", False))
+        self.o = Linear("gla.o" + (".float" if float_out else ""), self.hidden, self.heads * self.vdim, runtime, float_out=float_out, role="attn_out")
+        ws = runtime.workspace
+        ws.declare("gla.decay", runtime.max_step_tokens * self.heads * self.dim, torch.float32)
+        ws.declare("gla.qkv", runtime.max_step_tokens * self.at_gate, torch.float32)
+        self._declare_scratch(per_channel=True)
+        self.norm = self.decay_out = self.decay_bias = None
+
+    @staticmethod
+    def _names(params, prefix: str) -> dict[str, str]:
+        w, b = str(params.get("weight_suffix", ".weight")), str(params.get("bias_suffix", ".bias"))
+        n = {key: f"{prefix}.{params.get(key, key)}{w}" for key in ("q", "k", "v", "g", "o", "decay_in", "decay_out")}
+        n["decay_bias"] = f"{prefix}.{params.get('decay_out', 'decay_out')}{b}"
+        n["norm"] = f"{prefix}.{params.get('norm', 'norm')}"
+        return n
+
+    @classmethod
+    def expected_tensors(cls, params, prefix: str) -> dict[str, TensorSpec]:
+        hidden, heads, dim = int(params["hidden_size"]), int(params["num_heads"]), int(params["head_dim"])
+        vdim, rank = int(params.get("v_head_dim") or dim), int(params["decay_rank"])
+        n = cls._names(params, prefix)
+        std, narrow = float(params.get("init_std", 0.02)), float(params.get("narrow_init_std", 0.2))
+        return {n["q"]: TensorSpec((heads * dim, hidden), init_std=std), n["k"]: TensorSpec((heads * dim, hidden), init_std=std),
+                n["v"]: TensorSpec((heads * vdim, hidden), init_std=std), n["g"]: TensorSpec((heads * vdim, hidden), init_std=std),
+                n["o"]: TensorSpec((hidden, heads * vdim), init_std=std), n["norm"]: TensorSpec((vdim,), role="vector", init_std=0.1, init_mean=1.0),
+                n["decay_in"]: TensorSpec((rank, hidden), init_std=std), n["decay_out"]: TensorSpec((heads * dim, rank), init_std=narrow),
+                n["decay_bias"]: TensorSpec((heads * dim,), role="vector", init_std=0.5, init_mean=1.0)}
+
+    def load(self, source) -> None:
+        n = self._names(self.params, self.prefix)
+        dtype, device = self.runtime.dtype, self.runtime.device
+        rows = [source(n[key]).to(dtype) for key in ("q", "k", "v", "g", "decay_in")]
+        used = sum(r.shape[0] for r in rows)
+        if self.proj_rows > used:
+            rows.append(torch.zeros(self.proj_rows - used, self.hidden, dtype=dtype, device=rows[0].device))
+        self.proj.set_weight(torch.cat(rows, dim=0))
+        self.o.set_weight(source(n["o"]))
+        # the narrow projection's second matrix: float, transposed to [rank, N] so that neighbouring threads read neighbouring outputs
+        self.decay_out = to_device(source(n["decay_out"]).float().t(), torch.float32, device)
+        self.decay_bias = to_device(source(n["decay_bias"]), torch.float32, device)
+        self.norm = to_device(source(n["norm"]), torch.float32, device)
+
+    def cache_request(self):
+        return StateRequest((self.heads, self.vdim, self.dim), torch.float32)
+
+    def forward(self, x, ctx, cache):
+        self._check(cache)
+        tokens, width = x.shape[0], self.heads * self.vdim
+        ws = self.runtime.workspace
+        proj = self.proj(x)
+        decay = ws.view("gla.decay", tokens, self.heads, self.dim)
+        kernels.lowrank(proj, self.at_decay, self.decay_out, decay.view(tokens, self.heads * self.dim), self.decay_bias, power=1.0 / self.tau)
+        # split sums are added once, not by every block of the recurrence that reads them
+        rows = proj if proj.n_splits == 1 else kernels.linear_attention_prepare(proj, self.at_gate, ws.view("gla.qkv", tokens, self.at_gate), False)
+        read = ws.view("decayed.read", tokens, self.heads, self.vdim)
+        kernels.decayed_attention(rows, 0, self.at_k, self.at_v, decay, cache.state, read, ctx, self.dim, self._scratch_views(),
+                                  out_scale=self.dim ** -0.5)
+        normed = ws.view("decayed.normed", tokens, width)
+        kernels.group_gate_norm(read.view(tokens, width), self.norm, self.eps, normed, groups=self.heads, proj=proj, at_gate=self.at_gate, gate="silu")
+        return self._output(normed, tokens)
+
+
+@register_mixer("state_space")
+class StateSpace(_DecayedMixer):
+    """A state-space recurrence with a decay per head and token ("Mamba-2"):
+
+        S <- exp(-exp(A_h) d_t) S + d_t B_t x_t^T;   y_t = S^T C_t + D_h x_t
+
+    W_in h is laid out as [z | x | B | C | d]: z and x [heads, vdim], B and C [groups, state] (head h reads group
+    h // (heads / groups)), d one number per head.  x, B and C together pass a causal convolution per channel (``conv`` taps,
+    the last one the current token's, zeros before the sequence's start; with a bias) and SiLU; d is softplus(d + bias).  The
+    heads' y are concatenated, multiplied by silu(z), divided by the root mean square of each of ``norm_groups`` equal parts
+    (``eps`` inside the root), times a weight, and projected by W_o.  Per sequence the mixer keeps the states [heads, vdim,
+    state] and the convolution's last ``conv`` - 1 inputs, both float, zero for a new sequence, in the cache's per-slot state
+    rows.  The first product hands on float sums and everything between it and the output projection is float
+    (``csrc/short_conv.cu``, ``csrc/linear_attention.cu``, ``csrc/linear_attention_chunk.cu``).
+
+    Parameters: ``hidden_size``, ``num_heads``, ``v_head_dim``, ``state``, ``groups``, ``conv``, ``norm_groups``, ``eps``, ``float_out``,
+    ``init_std``, and the tensor-name pieces ``in``, ``conv_name``, ``step_bias``, ``decay_rate``, ``skip``, ``norm``, ``o``,
+    ``weight_suffix``, ``bias_suffix``."""
+
+    def __init__(self, params, prefix: str, runtime: Runtime) -> None:
+        self.prefix, self.runtime, self.params = prefix, runtime, dict(params)
+        self.hidden = int(params["hidden_size"])
+        self.heads, self.vdim, self.dim = int(params["num_heads"]), int(params["v_head_dim"]), int(params["state"])
+        self.groups, self.taps = int(params.get("groups", 1)), int(params.get("conv", 1))
+        self.norm_groups, self.eps = int(params.get("norm_groups", 1)), float(params.get("eps", 1e-6))
+        self.inner = self.heads * self.vdim
+        if self.heads % self.groups or self.inner % self.norm_groups:
+            raise ValueError(f"{prefix}: {self.groups} groups for {self.heads} heads, {self.norm_groups} norm groups for {self.inner} columns")
+        if not 1 <= self.taps <= 16:
+            raise ValueError(f"{prefix}: a convolution of {self.taps} taps (1..16)")
+        if self.dim > kernels.LINEAR_ATTENTION_MAX_DIM:
+            raise ValueError(f"{prefix}: states of {self.dim} rows per head are beyond what the recurrence kernels hold ({kernels.LINEAR_ATTENTION_MAX_DIM})")
+        self.channels = self.inner + 2 * self.groups * self.dim
+        self.at_step = self.inner + self.channels
+        self.rows = self.at_step + self.heads
+        self.proj_rows = -(-self.rows // 8) * 8
+        self.proj = Linear("ssm.proj", self.proj_rows, self.hidden, runtime, float_out=True)
+        float_out = bool(params.get("float_out", False))
+        self.o = Linear("ssm.o" + (".float" if float_out else ""), self.hidden, self.inner, runtime, float_out=float_out, role="attn_out")
+        ws, tokens = runtime.workspace, runtime.max_step_tokens
+        ws.declare("ssm.mixed", tokens * self.channels, torch.float32)
+        ws.declare("ssm.step", tokens * self.heads, torch.float32)
+        ws.declare("ssm.decay", tokens * self.heads, torch.float32)
+        self._declare_scratch(per_channel=False)
+        self.conv = self.conv_bias = self.step_bias = self.rate_log = self.skip = self.norm = None
+
+    @staticmethod
+    def _names(params, prefix: str) -> dict[str, str]:
+        w, b = str(params.get("weight_suffix", ".weight")), str(params.get("bias_suffix", ".bias"))
+        conv = str(params.get("conv_name", "conv"))
+        n = {key: f"{prefix}.{params.get(key, key)}{w}" for key in ("in", "o")}
+        n.update({key: f"{prefix}.{params.get(key, key)}" for key in ("step_bias", "decay_rate", "skip", "norm")})
+        n["conv"], n["conv_bias"] = f"{prefix}.{conv}{w}", f"{prefix}.{conv}{b}"
+        return n
+
+    @classmethod
+    def expected_tensors(cls, params, prefix: str) -> dict[str, TensorSpec]:
+        hidden, heads, vdim, state = (int(params[key]) for key in ("hidden_size", "num_heads", "v_head_dim", "state"))
+        groups, taps = int(params.get("groups", 1)), int(params.get("conv", 1))
+        inner = heads * vdim
+        channels = inner + 2 * groups * state
+        n = cls._names(params, prefix)
+        std = float(params.get("init_std", 0.02))
+        return {n["in"]: TensorSpec((inner + channels + heads, hidden), init_std=std), n["o"]: TensorSpec((hidden, inner), init_std=std),
+                n["conv"]: TensorSpec((channels, taps), role="vector", init_std=0.3, init_mean=0.3),
+                n["conv_bias"]: TensorSpec((channels,), role="vector", init_std=0.1), n["step_bias"]: TensorSpec((heads,), role="vector", init_std=0.5, init_mean=-1.0),
+                n["decay_rate"]: TensorSpec((heads,), role="vector", init_std=0.5, init_mean=-1.0),
+                n["skip"]: TensorSpec((heads,), role="vector", init_std=0.3, init_mean=1.0),
+                n["norm"]: TensorSpec((inner,), role="vector", init_std=0.1, init_mean=1.0)}
+
+    def load(self, source) -> None:
+        n = self._names(self.params, self.prefix)
+        dtype, device = self.runtime.dtype, self.runtime.device
+        weight = source(n["in"]).to(dtype)
+        if self.proj_rows > self.rows:
+            weight = torch.cat((weight, torch.zeros(self.proj_rows - self.rows, self.hidden, dtype=dtype, device=weight.device)), dim=0)
+        self.proj.set_weight(weight)
+        self.o.set_weight(source(n["o"]))
+        self.conv, self.conv_bias, self.step_bias, self.rate_log, self.skip, self.norm = (
+            to_device(source(n[key]), torch.float32, device) for key in ("conv", "conv_bias", "step_bias", "decay_rate", "skip", "norm"))
+
+    def cache_request(self):
+        return [StateRequest((self.heads, self.vdim, self.dim), torch.float32), StateRequest((max(self.taps - 1, 1), self.channels), torch.float32)]
+
+    def forward(self, x, ctx, cache):
+        states, kept = cache
+        self._check(states)
+        tokens = x.shape[0]
+        ws = self.runtime.workspace
+        proj = self.proj(x)
+        mixed = ws.view("ssm.mixed", tokens, self.channels)
+        step, decay = ws.view("ssm.step", tokens, self.heads), ws.view("ssm.decay", tokens, self.heads)
+        kernels.conv_act(proj, self.inner, self.conv, self.conv_bias, kept.state, ctx, mixed, self.at_step, self.step_bias, self.rate_log, step, decay)
+        read = ws.view("decayed.read", tokens, self.heads, self.vdim)
+        at_b, at_c = self.inner, self.inner + self.groups * self.dim
+        kernels.decayed_attention(GemmOut(mixed.view(1, tokens, self.channels)), at_c, at_b, 0, decay, states.state, read, ctx, self.dim,
+                                  self._scratch_views(), heads_per_key=self.heads // self.groups, v_scale=step)
+        normed = ws.view("decayed.normed", tokens, self.inner)
+        kernels.group_gate_norm(read.view(tokens, self.inner), self.norm, self.eps, normed, groups=self.norm_groups, proj=proj, at_gate=0, gate="silu",
+                                gate_first=True, x=mixed, at_x=0, skip=self.skip)
+        return self._output(normed, tokens)

@@ -421,7 +421,7 @@ def test_linear_attention_with_a_decay_per_head_in_portions(heads, dim, vdim):
     wanted = plain.rms_divide(o.double(), 1e-5) * weight.double() * torch.sigmoid(gate.double())
     for store in (torch.float32, torch.bfloat16):
         out = torch.empty(lengths[0], heads * vdim, dtype=store, device=DEV)
-        kernels.linear_attention_gate_norm(o.to(DEV), GemmOut(rows[0].to(DEV)), at_gate, weight.to(DEV), 1e-5, 1.0, out)
+        kernels.group_gate_norm(o.to(DEV), weight.to(DEV), 1e-5, out, proj=GemmOut(rows[0].to(DEV)), at_gate=at_gate)
         torch.testing.assert_close(out.float().cpu().double(), wanted, atol=1e-4 if store == torch.float32 else 3e-2, rtol=1e-2)
 
 
