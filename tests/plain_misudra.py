@@ -186,7 +186,7 @@ def experts(h, t, prefix, m, margins=None):
     logits = h @ t[prefix + ".router"].T
     chosen, weights = route(logits, router["top"], router.get("groups"))
     if margins is not None:
-        margins.append(choice_margin(logits, router["top"], router.get("groups")) / logits.std().clamp(min=1e-9))
+        margins.append(choice_margin(logits, router["top"], router.get("groups")) / logits.std(unbiased=False).clamp(min=1e-9))
     out = torch.zeros_like(h)
     for e in range(router["experts"]):
         rows, place = (chosen == e).nonzero(as_tuple=True)

@@ -1,0 +1,130 @@
+"""Misudra models drawn at random from what config.json allows (widths, head counts, ranks and sizes off 8 and off 16 among
+them, values narrower and wider than keys, the order and number of layers, loops of any range and count and none, windows down to
+one position and none, 1 to 12 experts in 1 to 4 groups, dense layers and layers without a feed-forward, 1 to 9 taps), each
+run whole, token by token, in portions and as an unequal batch in both types against the plain implementation."""
+import random
+import tempfile
+from pathlib import Path
+
+import pytest
+import torch
+
+import plain_misudra as plain
+from qwen_triton_b200 import Engine, StepEntry, config_from_dict, write_random_model
+from qwen_triton_b200.weights import Checkpoint, write_safetensors
+from test_gpu_vunepel import STORE, close as close_all
+
+CLOSE_CALL = 0.15      # a router's gap, over the scale of its logits, below which bfloat16 may choose otherwise
+
+pytestmark = pytest.mark.gpu
+
+
+def draw_mixer(rng, kind: str) -> dict:
+    heads = rng.choice([1, 2, 3, 4, 6, 8])
+    vdim = rng.choice([4, 8, 20, 32, 33, 64, 72])
+    if kind == "gla":
+        return {"heads": heads, "dim": rng.choice([3, 8, 16, 20, 64, 100, 128]), "vdim": vdim, "tau": rng.choice([0.7, 1.0, 4.0, 16.0]),
+                "ranks": {"decay": rng.choice([1, 4, 8, 16, 30])}}
+    if kind == "mamba2":
+        groups = rng.choice([g for g in (1, 2, 3, heads) if heads % g == 0])
+        return {"heads": heads, "vdim": vdim, "state": rng.choice([4, 16, 33, 64, 100, 128, 200]), "groups": groups, "conv": rng.choice([1, 2, 3, 4, 4, 9]),
+                "norm_groups": rng.choice([g for g in (1, 2, heads, heads * vdim // 2) if g > 0 and heads * vdim % g == 0])}
+    rot_dim = rng.choice([2, 6, 8, 16, 32])
+    mixer = {"heads": rng.choice([heads, 20, 34]) if rng.random() < 0.3 else heads, "dim": rng.choice([4, 10, 16, 32, 64]), "rot_dim": rot_dim, "vdim": vdim,
+             "q_rank": rng.choice([5, 16, 24, 40, 64]), "kv_rank": rng.choice([6, 8, 16, 40, 64, 136]), "scale": round(rng.uniform(0.05, 0.4), 3),
+             "rot": {"dims": rot_dim, "base": rng.choice([100.0, 10000.0, 300000.0])}}
+    if rng.random() < 0.8:
+        mixer["mask"] = {"size": rng.choice([1, 2, 7, 33, 64, 65, 100, 190])}
+    return mixer
+
+
+def draw(seed: int) -> dict:
+    rng = random.Random(5000 + seed)
+    layers = []
+    for _ in range(rng.randint(1, 6)):
+        kind = rng.choice(["gla", "mamba2", "latent_attention"])
+        mlp, roll = None, rng.random()
+        if roll < 0.35:
+            mlp = {"kind": "dense", "ff": rng.choice([8, 9, 20, 48, 100, 128])}
+        elif roll < 0.85:
+            count = rng.choice([1, 2, 3, 4])
+            size = rng.choice([1, 2, 3])
+            keep = rng.randint(1, count)
+            mlp = {"kind": "moe", "expert": {"ff": rng.choice([8, 9, 20, 48, 100]), "limit": rng.choice([0.5, 1.0, 4.0])},
+                   "router": {"experts": count * size, "top": rng.randint(1, min(keep * size, 4))}}
+            if count > 1 or rng.random() < 0.5:
+                mlp["router"]["groups"] = {"count": count, "keep": keep}
+        layers.append({"type": kind, "mixer": draw_mixer(rng, kind), "mlp": mlp})
+    raw = {"architecture": "Misudra", "vocab": rng.randint(30, 300), "width": rng.choice([36, 40, 64, 72, 96, 100, 128, 200]),
+           "norm": {"eps": rng.choice([1e-6, 1e-5, 1e-3])}, "layers": layers}
+    if rng.random() < 0.75:
+        start = rng.randrange(len(layers))
+        raw["loop"] = {"start": start, "stop": rng.randint(start + 1, len(layers)), "times": rng.randint(1, 3)}
+    return raw
+
+
+@pytest.mark.parametrize("dtype", ("fp32", "bf16"))
+@pytest.mark.parametrize("seed", range(12))
+def test_a_model_drawn_at_random(seed, dtype):
+    config = config_from_dict(draw(seed))
+    raw = config.to_hf_dict()
+    with tempfile.TemporaryDirectory() as holder:
+        folder = write_random_model(holder, config, seed=seed, dtype=STORE[dtype])
+        checkpoint = Checkpoint(folder)
+        tensors = {n: checkpoint.read(n) for n in checkpoint.names()}
+        for n in list(tensors):                    # sharper attention than the draw gives
+            if n.endswith(".dq.norm"):
+                tensors[n] = (tensors[n].float() * 3.0).to(tensors[n].dtype)
+        write_safetensors(Path(folder) / "model.safetensors", tensors)
+        weights = {n: t.float() for n, t in tensors.items()}
+        engine = Engine.from_pretrained(folder, dtype=dtype, max_tokens=2048, max_step_tokens=random.Random(seed).choice([96, 512, 4096]))
+    generator = torch.Generator().manual_seed(seed)
+    lengths = (200, 1, 70)
+    requests = [torch.randint(0, config.vocab_size, (n + 8,), generator=generator).tolist() for n in lengths]
+    wants, clear = [], []
+    for r in requests:
+        margins = []
+        wants.append(plain.forward(raw, weights, r, margins=margins).float())
+        clear.append(torch.stack(margins).min(dim=0).values >= CLOSE_CALL if margins and dtype == "bf16" else torch.ones(len(r), dtype=torch.bool))
+    what = f"seed {seed}: {raw}"
+
+    def close(actual, request, rows, text):
+        actual = actual.float().cpu()
+        assert bool(torch.isfinite(actual).all()), text
+        keep = clear[request][rows]
+        if bool(keep.any()):
+            close_all(actual[keep], wants[request][rows][keep], dtype, text, model_rows=True)
+
+    # whole, then the same request with its last 40 tokens one by one, then in portions of 19
+    slot = engine.new_sequence()
+    close(engine.step([StepEntry(slot, requests[0], list(range(len(requests[0]))))]), 0, slice(None), "whole, " + what)
+    engine.release(slot)
+    slot = engine.new_sequence()
+    head = len(requests[0]) - 40
+    rows = [engine.step([StepEntry(slot, requests[0][:head], [head - 1])])]
+    rows += [engine.step([StepEntry(slot, [t], [0])]) for t in requests[0][head:]]
+    engine.release(slot)
+    close(torch.cat(rows), 0, slice(head - 1, None), "token by token, " + what)
+    slot = engine.new_sequence()
+    rows = []
+    for begin in range(0, len(requests[0]), 19):
+        piece = requests[0][begin:begin + 19]
+        rows.append(engine.step([StepEntry(slot, piece, list(range(len(piece))))]))
+    engine.release(slot)
+    close(torch.cat(rows), 0, slice(None), "in portions, " + what)
+    # an unequal batch, then eight tokens each
+    slots = [engine.new_sequence() for _ in requests]
+    rows = [[] for _ in requests]
+    out = engine.step([StepEntry(s, r[:n], [n - 1]) for s, r, n in zip(slots, requests, lengths)])
+    for i in range(len(requests)):
+        rows[i].append(out[i:i + 1])
+    for t in range(8):
+        out = engine.step([StepEntry(s, [r[n + t]], [0]) for s, r, n in zip(slots, requests, lengths)])
+        for i in range(len(requests)):
+            rows[i].append(out[i:i + 1])
+    for i, n in enumerate(lengths):
+        close(torch.cat(rows[i]), i, slice(n - 1, None), f"batch row {i}, " + what)
+    for s in slots:
+        engine.release(s)
+    engine.cache.book.check()
+    engine.check_kernels()
