@@ -1,7 +1,7 @@
 """Decode and prefill throughput of the Qwen3-8B shape on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl b200|reference] [--temperature T]
-    python bench.py --workload 0.6b-unequal | 32b-long | lederax-layers | vunepel-layers | bisodra-layers | regupel-layers
+    python bench.py --workload 0.6b-unequal | 32b-long | lederax-layers | vunepel-layers | bisodra-layers | regupel-layers | misudra-layers
 
 Prints ONE JSON line.  ``value`` is decoded tokens per second at batch 8 from a 2,048-token cache,
 timed on the device over the decode steps (step function plus greedy sampling kernel, tokens given
@@ -27,7 +27,9 @@ a latent, attention with a short convolution on q and k under a window with kept
 first one's cache rows, a second convolution layer; the same three options), ``regupel-layers`` (four layers of the Regupel
 design: two parallel layers, windowed attention with kept first keys beside a linear attention with a decay per head, and two
 attention layers with a sink and a gate per head, each with routed experts and a shared expert, beside the Vunepel layers
-of equal size; the same three options).
+of equal size; the same three options), ``misudra-layers`` (four layers of the Misudra design: a gated linear attention with a
+dense feed-forward, a state-space layer, a windowed attention through a latent and a second gated linear attention with routed
+experts, the first two behind a map of the stream, beside Vunepel layers of equal size; the same three options).
 """
 from __future__ import annotations
 
@@ -61,9 +63,9 @@ def parse_args():
     parser.add_argument("--no-prefill", action="store_true")
     parser.add_argument("--min-seconds", type=float, default=2.0, help="a timed region lasts at least this long")
     parser.add_argument("--temperature", type=float, default=0.0, help="sampling temperature of the end-to-end run (0: greedy)")
-    parser.add_argument("--workload", default=None, choices=["0.6b-unequal", "32b-long", "lederax-layers", "vunepel-layers", "bisodra-layers", "regupel-layers"])
+    parser.add_argument("--workload", default=None, choices=["0.6b-unequal", "32b-long", "lederax-layers", "vunepel-layers", "bisodra-layers", "regupel-layers", "misudra-layers"])
     parser.add_argument("--size", default=None, help="vunepel-layers, bisodra-layers: only the size whose name starts with this")
-    parser.add_argument("--arm", default=None, choices=["vunepel", "bisodra", "regupel", "dense"], help="vunepel-layers, bisodra-layers, regupel-layers: only this model")
+    parser.add_argument("--arm", default=None, choices=["vunepel", "bisodra", "regupel", "misudra", "dense"], help="vunepel-layers, bisodra-layers, regupel-layers: only this model")
     parser.add_argument("--phase", default=None, choices=["prefill", "decode8", "decode64"], help="vunepel-layers, bisodra-layers: only this measurement")
     return parser.parse_args()
 
@@ -551,6 +553,107 @@ def run_regupel_layers(args) -> dict:
             "sizes": out}
 
 
+MISUDRA_SIZES = (
+    # name, width, recurrent heads, key size, value size, state-space heads, their value size, state rows, groups, attention heads, plain, rotated and
+    # value size, query rank, latent, window, experts, top, groups, kept groups, expert width, dense width
+    ("w2048-gla16x128-ssm32x64x128-latent16x512-window1024-e16x1024-top2", 2048, 16, 128, 128, 32, 64, 128, 4, 16, 128, 64, 128, 768, 512, 1024, 16, 2, 4, 2, 1024, 6144),
+    ("w4096-gla32x128-ssm64x64x128-latent32x512-window4096-e16x2048-top2", 4096, 32, 128, 128, 64, 64, 128, 8, 32, 128, 64, 128, 1536, 512, 4096, 16, 2, 4, 2, 2048, 12288),
+    ("w1024-gla8x64x128-ssm16x64x64-latent8x256-window512-e8x2048-top1", 1024, 8, 64, 128, 16, 64, 64, 2, 8, 64, 32, 64, 384, 256, 512, 8, 1, 2, 1, 2048, 3072),
+)
+
+
+def run_misudra_layers(args) -> dict:
+    """Prefill and one-token steps of four Misudra layers at sizes that resemble a real model's (a gated linear attention with a
+    dense feed-forward with biases and a state-space layer with routed experts, behind a map of the stream; an attention
+    through a latent under a window and a second gated linear attention with routed experts), and of the Vunepel layers that
+    come closest (the library's other design whose recurrence has a decay per key channel, a short convolution and experts
+    with the capped gate): same width and vocabulary, delta-rule layers with the same state size where the recurrent layers
+    stand, a differential attention layer under a chunk as long as the window, the same feed-forwards."""
+    import torch
+
+    from qwen_triton_b200 import QwenB200ForCausalLM, config_from_dict
+
+    peak, peak_source = peaks()
+    vocab, prompt_len = 32768, args.prompt_len
+    out = []
+    for size in MISUDRA_SIZES:
+        (name, width, heads, dim, vdim, s_heads, s_vdim, state, s_groups, a_heads, plain, rot, a_vdim, q_rank, latent, window, experts, top, groups,
+         keep, ff, dense) = size
+        if args.size and not name.startswith(args.size):
+            continue
+        rank = 16
+        moe = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}}}
+        gla = {"heads": heads, "dim": dim, "vdim": vdim, "tau": 16.0, "ranks": {"decay": rank}}
+        space = {"heads": s_heads, "vdim": s_vdim, "state": state, "groups": s_groups, "conv": 4, "norm_groups": s_groups}
+        attention = {"heads": a_heads, "dim": plain, "rot_dim": rot, "vdim": a_vdim, "q_rank": q_rank, "kv_rank": latent, "scale": (plain + rot) ** -0.5,
+                     "mask": {"size": window}, "rot": {"base": 500000.0, "dims": rot}}
+        misudra = {"architecture": "Misudra", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "loop": {"start": 0, "stop": 2, "times": 1},
+                   "layers": [{"type": "gla", "mixer": gla, "mlp": {"kind": "dense", "ff": dense}}, {"type": "mamba2", "mixer": space, "mlp": moe},
+                              {"type": "latent_attention", "mixer": attention, "mlp": moe}, {"type": "gla", "mixer": gla, "mlp": moe}]}
+        v_moe = {"kind": "moe", "router": {"experts": experts, "top": top, "scale": 2.0}, "expert": {"ff": ff, "limit": 7.0}}
+        v_heads, v_kv = max(1, a_heads // 2), max(1, a_heads // 8)
+        v_attention = {"heads": v_heads, "kv_heads": v_kv, "dim": plain, "vdim": plain, "scale": plain ** -0.5, "diff": 0.3,
+                       "rot": {"dims": plain, "base": 500000.0}, "mask": {"size": window}}
+        delta = {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": vdim, "conv": 4, "ranks": {"decay": 64, "gate": 64}}
+        vunepel = {"architecture": "Vunepel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+                   "layers": [{"type": "channel_delta", "mixer": delta, "mlp": {"kind": "dense", "ff": dense, "limit": 7.0}},
+                              {"type": "channel_delta", "mixer": delta, "mlp": v_moe}, {"type": "attention", "mixer": v_attention, "mlp": v_moe},
+                              {"type": "channel_delta", "mixer": delta, "mlp": v_moe}]}
+        # weights a token multiplies with (the experts: the chosen ones)
+        inner = s_heads * s_vdim
+        gla_w = width * (2 * heads * dim + 3 * heads * vdim + rank) + rank * heads * dim
+        space_w = width * (3 * inner + 2 * s_groups * state + s_heads)
+        latent_w = width * (q_rank + latent + rot + a_heads) + a_heads * ((plain + rot) * q_rank + plain * latent + a_vdim * latent + a_vdim * width)
+        mixers = 2 * gla_w + space_w + latent_w + 2 * width * width + 3 * width * dense
+        v_delta_w = width * (2 * heads * dim + 2 * heads * vdim + heads + 128) + 64 * heads * (dim + vdim)
+        v_attn_w = width * (2 * v_heads + 3 * v_kv) * plain + v_heads * plain * width
+        v_mixers = 3 * v_delta_w + v_attn_w + 3 * width * dense
+
+        def moe_weights(count):
+            return 3 * width * ff * count + width * experts
+
+        state_bytes = 2 * 4 * (2 * heads * dim * vdim + inner * state + 3 * (inner + 2 * s_groups * state))
+        arms = (("misudra", misudra, mixers, 2 * a_heads * (2 * latent + rot), 2 * (latent + rot), state_bytes),
+                ("vunepel", vunepel, v_mixers, 4 * 2 * v_heads * plain, 2 * 3 * v_kv * plain, 2 * 4 * 3 * (heads * dim * vdim + 3 * heads * (2 * dim + vdim))))
+        entry = {"size": name, "layers": 4}
+        for label, raw, mixer_weights, pair_flops, key_bytes, states in arms:
+            if args.arm and label != args.arm:
+                continue
+            model = QwenB200ForCausalLM.from_config(config_from_dict(raw), seed=1, dtype="bf16",
+                                                    max_tokens=64 * (prompt_len + 512), max_seq_len=prompt_len + 512,
+                                                    max_step_tokens=max(4096, prompt_len), chunk_tokens=prompt_len)
+            result = {}
+            if args.phase in (None, "prefill"):
+                ms = time_prefill(model, prompt_len, vocab, repeats=args.steps if args.phase else 5, warmup=args.warmup if args.phase else 3)
+                # a windowed query sees the last keys, a chunked one its chunk's earlier keys
+                keys = sum(min(i + 1, window) if label == "misudra" else i % window + 1 for i in range(prompt_len))
+                flops = 2 * prompt_len * (mixer_weights + 3 * moe_weights(top) + vocab * width / prompt_len) + pair_flops * keys
+                result["prefill"] = {"tokens": prompt_len, "ms": round(ms, 3), "tokens_per_s": round(prompt_len * 1e3 / ms),
+                                     "tensor_fraction": round(flops / (ms * 1e-3) / (peak["bf16_tflops"] * 1e12), 4)}
+            for batch in (8, 64):
+                if args.phase not in (None, f"decode{batch}"):
+                    continue
+                prompts = random_prompts(batch, prompt_len, vocab, 300 + batch)
+                ms, launches, clocks, context, steps = time_decode(model, prompts, args.steps, args.warmup, vocab,
+                                                                   args.min_seconds / 4, 256)
+                live = min(context, window) if label == "misudra" else context % window
+                read = 2 * (mixer_weights + 3 * moe_weights(min(experts, batch * top)) + vocab * width) + batch * (key_bytes * live + states)
+                result[f"decode_batch{batch}"] = {"ms_per_step": round(ms, 4), "tokens_per_s": round(batch * 1e3 / ms),
+                                                   "launches_per_step": round(launches / steps, 1), "steps": steps,
+                                                   "hbm_fraction": round(read / (ms * 1e-3) / (peak["hbm_gbs"] * 1e9), 4),
+                                                   "clocks": clocks}
+            entry[label] = result
+            print(f"[bench] {name} {label}: " + json.dumps({k: {a: b for a, b in v.items() if a != 'clocks'} for k, v in result.items()}),
+                  file=sys.stderr, flush=True)
+            del model
+            torch.cuda.empty_cache()
+        out.append(entry)
+    return {"workload": args.workload, "impl": "b200", "dtype": "bf16", "data": "synthetic", "n_gpus": 1,
+            "config": {"prompt_len": prompt_len, "layers": 4, "vocab": vocab, "peaks": peak_source,
+                       "l2": "weights, caches and states of a step exceed L2 at every size but the smallest"},
+            "sizes": out}
+
+
 def time_prefill(model, tokens: int, vocab: int, repeats: int = 5, warmup: int = 3):
     import torch
     from qwen_triton_b200 import StepEntry
@@ -745,6 +848,8 @@ def run_workload(args) -> dict:
         return run_bisodra_layers(args)
     if args.workload == "regupel-layers":
         return run_regupel_layers(args)
+    if args.workload == "misudra-layers":
+        return run_misudra_layers(args)
     import torch
 
     from qwen_triton_b200 import QwenB200ForCausalLM, StepEntry, load_preset

@@ -26,7 +26,7 @@ __global__ void embedding_kernel(float* __restrict__ residual, const T* __restri
 
 // The same with an RMS norm behind the gather: residual[t, :] = x / sqrt(mean(x^2) + eps) * norm_w for the scaled row x.
 // `start` (or null) takes a copy of the result in the table's type: the embedding's output, for a model whose layers
-// meet it again.  One block per token; a row is read twice (from L1 the second time).
+// meet it again.  One block per token.
 template <typename T>
 __global__ void embedding_norm_kernel(float* __restrict__ residual, const T* __restrict__ table, const int* __restrict__ ids, int hidden,
                                       int vocab, float scale, const float* __restrict__ norm_w, float eps, T* __restrict__ start) {
@@ -37,17 +37,25 @@ __global__ void embedding_norm_kernel(float* __restrict__ residual, const T* __r
     int id = ids[t];
     const bool valid = id >= 0 && id < vocab;
     const T* row = table + (size_t)(valid ? id : 0) * hidden;
-    float inv = scale;
-    if (norm_w) {
-        float sq = 0.f;
-        for (int i = threadIdx.x; i < hidden; i += blockDim.x) { const float x = to_float(row[i]) * scale; sq += x * x; }
-        inv = rsqrtf(block_sum(sq, scratch) / (float)hidden + eps) * scale;
+    constexpr int KEEP = 16;                                  // elements a thread keeps; wider rows are read again
+    float x[KEEP], sq = 0.f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        x[j] = i < hidden && valid ? to_float(row[i]) * scale : 0.f;
+        sq += x[j] * x[j];
     }
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
-        const float y = valid ? to_float(row[i]) * inv * (norm_w ? norm_w[i] : 1.f) : 0.f;
+    for (int i = threadIdx.x + KEEP * blockDim.x; i < hidden; i += blockDim.x) { const float v = valid ? to_float(row[i]) * scale : 0.f; sq += v * v; }
+    const float inv = norm_w ? rsqrtf(block_sum(sq, scratch) / (float)hidden + eps) : 1.f;
+    auto put = [&](int i, float v) {
+        const float y = v * inv * (norm_w ? __ldg(norm_w + i) : 1.f);
         residual[(size_t)t * hidden + i] = y;
         if (start) start[(size_t)t * hidden + i] = from_float<T>(y);
-    }
+    };
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j)
+        if (threadIdx.x + j * blockDim.x < hidden) put(threadIdx.x + j * blockDim.x, x[j]);
+    for (int i = threadIdx.x + KEEP * blockDim.x; i < hidden; i += blockDim.x) put(i, valid ? to_float(row[i]) * scale : 0.f);
 }
 
 extern "C" int qt_embedding(float* residual, const void* table, const int* ids, int n_tokens, int hidden, int vocab,
@@ -77,12 +85,28 @@ __global__ void stream_concat_kernel(float* __restrict__ residual, const TD* __r
     pdl_launch_dependents();
     pdl_wait();
     const size_t at = (size_t)blockIdx.x * hidden, to = 2 * at;
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
-        float x = residual[at + i];
-        if (delta) x += load_sum(delta, at + i, n_splits, split_stride);
-        residual[at + i] = 0.f;
-        out[to + i] = from_float<TO>(x);
-        out[to + hidden + i] = start[at + i];
+    constexpr int AHEAD = 8;                                  // elements a thread asks for before it stores the first
+    for (int i0 = threadIdx.x; i0 < hidden; i0 += AHEAD * blockDim.x) {
+        float x[AHEAD];
+        TO s[AHEAD];
+#pragma unroll
+        for (int j = 0; j < AHEAD; ++j) {
+            const int i = i0 + j * blockDim.x;
+            x[j] = 0.f;
+            if (i < hidden) {
+                x[j] = residual[at + i];
+                s[j] = start[at + i];
+                if (delta) x[j] += load_sum(delta, at + i, n_splits, split_stride);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < AHEAD; ++j) {
+            const int i = i0 + j * blockDim.x;
+            if (i >= hidden) break;
+            residual[at + i] = 0.f;
+            out[to + i] = from_float<TO>(x[j]);
+            out[to + hidden + i] = s[j];
+        }
     }
 }
 

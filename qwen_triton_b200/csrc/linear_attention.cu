@@ -467,15 +467,23 @@ struct GroupNormParams {
 
 __device__ __forceinline__ float gn_gate(const GroupNormParams& p, size_t t, int i) {
     const float* at = p.proj + t * p.proj_cols + p.at_gate + i;
-    float g = at[0];
-    for (int s = 1; s < p.n_splits; ++s) g += at[(size_t)s * p.split_stride];
+    float g = 0.f;
+    if (p.n_splits == 1) g = __ldg(at);
+    else {
+        for (int s0 = 0; s0 < p.n_splits; s0 += 8) {                    // eight loads of a split product's planes in flight
+            float v[8];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = s0 + j < p.n_splits ? __ldg(at + (size_t)(s0 + j) * p.split_stride) : 0.f;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) g += v[j];
+        }
+    }
     const float sig = 1.f / (1.f + expf(-g));
     return p.silu ? g * sig : sig;
 }
 __device__ __forceinline__ float gn_value(const GroupNormParams& p, size_t t, int i) {
-    float y = p.o[t * p.width + i];
-    if (p.x) y += p.skip[i / p.per_skip] * p.x[t * p.x_cols + p.at_x + i];
-    if (p.proj && p.gate_first) y *= gn_gate(p, t, i);
+    float y = __ldg(p.o + t * p.width + i);
+    if (p.x) y += __ldg(p.skip + i / p.per_skip) * __ldg(p.x + t * p.x_cols + p.at_x + i);
     return y;
 }
 
@@ -492,24 +500,28 @@ __global__ void group_gate_norm_kernel(const GroupNormParams p, TO* __restrict__
     const int part = WARP ? blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5) : blockIdx.y;
     if (WARP && part * p.part >= p.width) return;                       // whole warps leave; a block's threads stay together otherwise
     const int first = WARP ? threadIdx.x & 31 : threadIdx.x, step = WARP ? 32 : blockDim.x, base = part * p.part;
-    float y[GN_CACHE], sq = 0.f;
+    float y[GN_CACHE], gate[GN_CACHE], sq = 0.f;
 #pragma unroll
     for (int j = 0; j < GN_CACHE; ++j) {
         const int i = first + j * step;
         y[j] = i < p.part ? gn_value(p, t, base + i) : 0.f;
+        gate[j] = i < p.part && p.proj ? gn_gate(p, t, base + i) : 1.f;
+    }
+#pragma unroll
+    for (int j = 0; j < GN_CACHE; ++j) {
+        if (p.gate_first) { y[j] *= gate[j]; gate[j] = 1.f; }
         sq += y[j] * y[j];
     }
-    for (int i = first + GN_CACHE * step; i < p.part; i += step) { const float v = gn_value(p, t, base + i); sq += v * v; }
+    for (int i = first + GN_CACHE * step; i < p.part; i += step) {
+        const float v = gn_value(p, t, base + i) * (p.proj && p.gate_first ? gn_gate(p, t, base + i) : 1.f);
+        sq += v * v;
+    }
     const float inv = rsqrtf((WARP ? warp_sum(sq) : block_sum(sq, scratch)) / (float)p.part + p.eps) * p.scale;
-    auto finish = [&](float v, int i) {
-        v *= inv * p.weight[p.weight_len == p.part ? i : base + i];
-        if (p.proj && !p.gate_first) v *= gn_gate(p, t, base + i);
-        out[t * p.width + base + i] = from_float<TO>(v);
-    };
+    auto finish = [&](float v, int i) { out[t * p.width + base + i] = from_float<TO>(v * inv * __ldg(p.weight + (p.weight_len == p.part ? i : base + i))); };
 #pragma unroll
     for (int j = 0; j < GN_CACHE; ++j)
-        if (first + j * step < p.part) finish(y[j], first + j * step);
-    for (int i = first + GN_CACHE * step; i < p.part; i += step) finish(gn_value(p, t, base + i), i);
+        if (first + j * step < p.part) finish(y[j] * gate[j], first + j * step);
+    for (int i = first + GN_CACHE * step; i < p.part; i += step) finish(gn_value(p, t, base + i) * (p.proj ? gn_gate(p, t, base + i) : 1.f), i);
 }
 
 extern "C" int qt_group_gate_norm(const float* o, const float* x, int x_cols, int at_x, const float* skip, int skips, const float* proj, int n_splits,

@@ -24,6 +24,8 @@
 
 #include <math.h>
 
+#include <initializer_list>
+
 using namespace qt;
 
 namespace {
@@ -56,69 +58,118 @@ __device__ __forceinline__ Chunk chunk_of(const ChunkArgs& p, int seq, int c) {
     return {begin + c * CT, min(CT, end - begin - c * CT), begin / CT + seq + c};
 }
 
+// Four consecutive floats from p on, `left` of which exist (zeros beyond); one 16-byte load where `vec` says the address allows it.
+__device__ __forceinline__ float4 load4(const float* p, int left, bool vec) {
+    if (vec && left >= 4) return __ldg(reinterpret_cast<const float4*>(p));
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (left > 0) v.x = __ldg(p);
+    if (left > 1) v.y = __ldg(p + 1);
+    if (left > 2) v.z = __ldg(p + 2);
+    if (left > 3) v.w = __ldg(p + 3);
+    return v;
+}
+__device__ __forceinline__ void put4(float* p, const float4& v, int left, bool vec) {
+    if (vec && left >= 4) { *reinterpret_cast<float4*>(p) = v; return; }
+    if (left > 0) p[0] = v.x;
+    if (left > 1) p[1] = v.y;
+    if (left > 2) p[2] = v.z;
+    if (left > 3) p[3] = v.w;
+}
+__device__ __forceinline__ float4 times(const float4& v, float f) { return make_float4(v.x * f, v.y * f, v.z * f, v.w * f); }
+
 // ----------------------------------------------------------------------------- decays per key channel
-// grid (chunks of the longest sequence, heads, sequences), 256 threads; dynamic shared memory 3 CT (dim + 4) + CT (CT + 1) + 7 dim floats.
-__global__ void __launch_bounds__(256) chunk_prepare_channel_kernel(const ChunkArgs p) {
+// grid (chunks of the longest sequence, heads, sequences), PC_THREADS threads; dynamic shared memory (floats): 3 rows of CT x ld, then 15 dim4,
+// with dim4 = dim rounded up to a multiple of 4 and ld = dim4 + 4.
+constexpr int PC_THREADS = 512;
+
+__device__ __forceinline__ float dot4(const float4& a, const float4& b, float acc) {
+    return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, acc))));
+}
+__device__ __forceinline__ float4 mul4(const float4& a, const float4& b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+
+// Sixteen values per lane, summed over the lanes of the warp: lane l gets the sum of value l % 16.
+__device__ __forceinline__ float transpose_sum(float (&part)[SUB], int lane) {
+#pragma unroll
+    for (int half = SUB / 2; half >= 1; half >>= 1) {
+        const bool upper = (lane & half) != 0;
+#pragma unroll
+        for (int j = 0; j < half; ++j) {
+            const float give = upper ? part[j] : part[j + half], keep = upper ? part[j + half] : part[j];
+            part[j] = keep + __shfl_xor_sync(0xffffffffu, give, half);
+        }
+    }
+    return part[0] + __shfl_xor_sync(0xffffffffu, part[0], 16);
+}
+
+__global__ void __launch_bounds__(PC_THREADS, 2) chunk_prepare_channel_kernel(const ChunkArgs p, int vec) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ __align__(16) float sm[];
-    const int dim = p.dim, ld = dim + 4, head = blockIdx.y, key_head = head / p.heads_per_key;
+    const int dim = p.dim, quads = (dim + 3) / 4, dim4 = quads * 4, ld = dim4 + 4, head = blockIdx.y, key_head = head / p.heads_per_key;
     const Chunk ck = chunk_of(p, blockIdx.z, blockIdx.x);
     if (ck.count <= 0) return;
-    float* qs = sm;                        // [CT][ld] q, later e^{sum of its run up to t} q
-    float* ks = qs + CT * ld;              // [CT][ld] k, later e^{sum of its run behind s} k
+    float* qs = sm;                        // [CT][ld] q, later e^{sum of g in its run up to t} q
+    float* ks = qs + CT * ld;              // [CT][ld] k, later e^{sum of g in its run behind s} k
     float* as = ks + CT * ld;              // [CT][ld] e^{g}
-    float* tile = as + CT * ld;            // [CT][CT + 1] A, row t
-    float* run = tile + CT * (CT + 1);     // [RUNS][dim] sum of g over a run
-    float* over = run + RUNS * dim;        // [3][dim] e^{run 1}, e^{run 2}, e^{run 1 + run 2}
+    float* run = as + CT * ld;             // [RUNS][dim4] sum of g over a run
+    float* over = run + RUNS * dim4;       // [3][dim4] e^{run 1}, e^{run 2}, e^{run 1 + run 2}
+    float* before = over + 3 * dim4;       // [RUNS][dim4] e^{the runs before}
+    float* after = before + RUNS * dim4;   // [RUNS][dim4] e^{the runs behind}
     const float* g = p.log_decay + ((size_t)ck.first * p.heads + head) * dim;
     const size_t g_row = (size_t)p.heads * dim;
-    for (int i = threadIdx.x; i < CT * dim; i += 256) {
-        const int t = i / dim, n = i % dim;
-        const bool in = t < ck.count;
-        const size_t row = (size_t)(ck.first + t) * p.cols + (size_t)key_head * dim + n;
-        qs[t * ld + n] = in ? p.rows[row + p.at_q] * p.out_scale : 0.f;
-        ks[t * ld + n] = in ? p.rows[row + p.at_k] : 0.f;
-        as[t * ld + n] = in ? expf(g[t * g_row + n]) : 1.f;
-    }
-    for (int i = threadIdx.x; i < CT * (CT + 1); i += 256) tile[i] = 0.f;
-    __syncthreads();
-    // inside a run: one warp per s; its lanes hold k_s decayed so far, multiplied by e^{g_t} as t goes on
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int s = warp; s < ck.count; s += 8) {
-        const int r0 = s / SUB * SUB;
-        float part[SUB];
+    const float* rows = p.rows + (size_t)ck.first * p.cols + (size_t)key_head * dim;
+    constexpr int AHEAD = 4;
+    for (int i0 = threadIdx.x; i0 < CT * quads; i0 += AHEAD * PC_THREADS) {
+        float4 q[AHEAD], k[AHEAD], e[AHEAD];
 #pragma unroll
-        for (int j = 0; j < SUB; ++j) part[j] = 0.f;
+        for (int j = 0; j < AHEAD; ++j) {
+            const int i = i0 + j * PC_THREADS, t = i / quads, n = i % quads * 4;
+            const int left = i < CT * quads && t < ck.count ? dim - n : 0;
+            q[j] = load4(rows + (size_t)t * p.cols + p.at_q + n, left, vec);
+            k[j] = load4(rows + (size_t)t * p.cols + p.at_k + n, left, vec);
+            e[j] = load4(g + (size_t)t * g_row + n, left, vec);
+        }
+#pragma unroll
+        for (int j = 0; j < AHEAD; ++j) {
+            const int i = i0 + j * PC_THREADS, t = i / quads, n = i % quads * 4;
+            if (i >= CT * quads) break;
+            *reinterpret_cast<float4*>(qs + t * ld + n) = times(q[j], p.out_scale);
+            *reinterpret_cast<float4*>(ks + t * ld + n) = k[j];
+            *reinterpret_cast<float4*>(as + t * ld + n) = make_float4(expf(e[j].x), expf(e[j].y), expf(e[j].z), expf(e[j].w));
+        }
+    }
+    __syncthreads();
+    float* within = p.within + ((size_t)ck.index * p.heads + head) * CT * CT;      // [s][t]
+    // inside a run: a warp takes two neighbouring s; its lanes hold k_s decayed so far, multiplied by e^{g_t} as t goes on
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int s = 2 * warp; s < CT; s += 2 * (PC_THREADS / 32)) {
+        const int r0 = s / SUB * SUB;
+        float part0[SUB], part1[SUB];
+#pragma unroll
+        for (int j = 0; j < SUB; ++j) part0[j] = part1[j] = 0.f;
         for (int n = lane; n < dim; n += 32) {
-            float w = ks[s * ld + n];
+            float w0 = ks[s * ld + n], w1 = ks[(s + 1) * ld + n];
 #pragma unroll
             for (int j = 0; j < SUB; ++j) {
                 const int t = r0 + j;
-                if (t > s) w *= as[t * ld + n];
-                if (t >= s) part[j] += w * qs[t * ld + n];
+                if (t < s) continue;
+                const float q = qs[t * ld + n], a = as[t * ld + n];
+                if (t > s) w0 *= a;
+                part0[j] = fmaf(w0, q, part0[j]);
+                if (t > s + 1) w1 *= a;
+                if (t > s) part1[j] = fmaf(w1, q, part1[j]);
             }
         }
-        // sixteen sums over the lanes: halve the values a lane carries four times, then one more exchange
-#pragma unroll
-        for (int half = SUB / 2; half >= 1; half >>= 1) {
-            const bool upper = (lane & half) != 0;
-#pragma unroll
-            for (int j = 0; j < half; ++j) {
-                const float give = upper ? part[j] : part[j + half], keep = upper ? part[j + half] : part[j];
-                part[j] = keep + __shfl_xor_sync(0xffffffffu, give, half);
-            }
-        }
-        const float total = part[0] + __shfl_xor_sync(0xffffffffu, part[0], 16);
-        if (lane < SUB && r0 + lane >= s) tile[(r0 + lane) * (CT + 1) + s] = total;
+        const float sum0 = transpose_sum(part0, lane), sum1 = transpose_sum(part1, lane);
+        if (lane < SUB) { within[s * CT + r0 + lane] = sum0; within[(s + 1) * CT + r0 + lane] = sum1; }
     }
     __syncthreads();
     // running sums inside the runs, forwards on q and backwards on k
-    for (int i = threadIdx.x; i < RUNS * dim; i += 256) {
-        const int r = i / dim, n = i % dim;
+    for (int i = threadIdx.x; i < RUNS * dim4; i += PC_THREADS) {
+        const int r = i / dim4, n = i % dim4;
         float v[SUB];
 #pragma unroll
-        for (int j = 0; j < SUB; ++j) v[j] = r * SUB + j < ck.count ? g[(size_t)(r * SUB + j) * g_row + n] : 0.f;
+        for (int j = 0; j < SUB; ++j) v[j] = n < dim && r * SUB + j < ck.count ? __ldg(g + (size_t)(r * SUB + j) * g_row + n) : 0.f;
         float sum = 0.f;
 #pragma unroll
         for (int j = 0; j < SUB; ++j) { sum += v[j]; qs[(r * SUB + j) * ld + n] *= expf(sum); }
@@ -128,114 +179,149 @@ __global__ void __launch_bounds__(256) chunk_prepare_channel_kernel(const ChunkA
         for (int j = SUB - 1; j >= 0; --j) { ks[(r * SUB + j) * ld + n] *= expf(behind); behind += v[j]; }
     }
     __syncthreads();
-    for (int n = threadIdx.x; n < dim; n += 256) {
-        over[n] = expf(run[dim + n]);
-        over[dim + n] = expf(run[2 * dim + n]);
-        over[2 * dim + n] = expf(run[dim + n] + run[2 * dim + n]);
-        p.whole[((size_t)ck.index * p.heads + head) * dim + n] = expf(run[n] + run[dim + n] + run[2 * dim + n] + run[3 * dim + n]);
+    for (int n = threadIdx.x; n < dim4; n += PC_THREADS) {
+        const float g0 = run[n], g1 = run[dim4 + n], g2 = run[2 * dim4 + n], g3 = run[3 * dim4 + n];
+        over[n] = expf(g1); over[dim4 + n] = expf(g2); over[2 * dim4 + n] = expf(g1 + g2);
+        before[n] = 1.f; before[dim4 + n] = expf(g0); before[2 * dim4 + n] = expf(g0 + g1); before[3 * dim4 + n] = expf(g0 + g1 + g2);
+        after[n] = expf(g1 + g2 + g3); after[dim4 + n] = expf(g2 + g3); after[2 * dim4 + n] = expf(g3); after[3 * dim4 + n] = 1.f;
+        if (n < dim) p.whole[((size_t)ck.index * p.heads + head) * dim + n] = expf(g0 + g1 + g2 + g3);
     }
     __syncthreads();
-    // between runs: A of run i against run j < i, two t by two s per thread
-    for (int item = threadIdx.x; item < 6 * 64; item += 256) {
+    // between runs: A of run i against run j < i, two t by two s per thread; and zeros where t lies in an earlier run than s
+    for (int item = threadIdx.x; item < 6 * 64; item += PC_THREADS) {
         const int pair = item >> 6, local = item & 63;
         const int i = pair < 1 ? 1 : pair < 3 ? 2 : 3, j = pair < 1 ? 0 : pair < 3 ? pair - 1 : pair - 3;
-        const int t = i * SUB + (local >> 3) * 2, s = j * SUB + (local & 7) * 2;
-        const float* mid = i - j == 3 ? over + 2 * dim : i - j == 2 ? (j == 0 ? over : over + dim) : nullptr;
-        if (t >= ck.count) continue;
+        const int t = i * SUB + (local & 7) * 2, s = j * SUB + (local >> 3) * 2;
+        const float* mid = i - j == 3 ? over + 2 * dim4 : i - j == 2 ? (j == 0 ? over : over + dim4) : nullptr;
         float a00 = 0.f, a01 = 0.f, a10 = 0.f, a11 = 0.f;
-        const float *q0 = qs + t * ld, *q1 = q0 + ld, *k0 = ks + s * ld, *k1 = k0 + ld;
-        for (int n = 0; n < dim; ++n) {
-            float x0 = k0[n], x1 = k1[n];
-            if (mid) { x0 *= mid[n]; x1 *= mid[n]; }
-            a00 += q0[n] * x0; a01 += q0[n] * x1; a10 += q1[n] * x0; a11 += q1[n] * x1;
+        const float *q0 = qs + t * ld, *k0 = ks + s * ld;
+        for (int n = 0; n < dim4; n += 4) {
+            float4 x0 = *reinterpret_cast<const float4*>(k0 + n), x1 = *reinterpret_cast<const float4*>(k0 + ld + n);
+            const float4 y0 = *reinterpret_cast<const float4*>(q0 + n), y1 = *reinterpret_cast<const float4*>(q0 + ld + n);
+            if (mid) { const float4 m = *reinterpret_cast<const float4*>(mid + n); x0 = mul4(x0, m); x1 = mul4(x1, m); }
+            a00 = dot4(y0, x0, a00); a01 = dot4(y0, x1, a01); a10 = dot4(y1, x0, a10); a11 = dot4(y1, x1, a11);
         }
-        tile[t * (CT + 1) + s] = a00; tile[t * (CT + 1) + s + 1] = a01;
-        tile[(t + 1) * (CT + 1) + s] = a10; tile[(t + 1) * (CT + 1) + s + 1] = a11;
+        *reinterpret_cast<float2*>(within + s * CT + t) = make_float2(a00, a10);
+        *reinterpret_cast<float2*>(within + (s + 1) * CT + t) = make_float2(a01, a11);
+        const int late = i * SUB + (local >> 3) * 2, early = j * SUB + (local & 7) * 2;
+        *reinterpret_cast<float2*>(within + late * CT + early) = make_float2(0.f, 0.f);
+        *reinterpret_cast<float2*>(within + (late + 1) * CT + early) = make_float2(0.f, 0.f);
     }
     // the decayed q and k of the whole chunk
-    for (int i = threadIdx.x; i < ck.count * dim; i += 256) {
-        const int t = i / dim, n = i % dim, r = t / SUB;
-        float before = 0.f, after = 0.f;
-#pragma unroll
-        for (int o = 0; o < RUNS; ++o) { if (o < r) before += run[o * dim + n]; if (o > r) after += run[o * dim + n]; }
+    for (int i = threadIdx.x; i < ck.count * quads; i += PC_THREADS) {
+        const int t = i / quads, n = i % quads * 4, r = t / SUB;
         const size_t at = ((size_t)(ck.first + t) * p.heads + head) * dim + n;
-        p.q_from[at] = qs[t * ld + n] * expf(before);
-        p.k_to[at] = ks[t * ld + n] * expf(after);
+        put4(p.q_from + at, mul4(*reinterpret_cast<const float4*>(qs + t * ld + n), *reinterpret_cast<const float4*>(before + r * dim4 + n)), dim - n, vec);
+        put4(p.k_to + at, mul4(*reinterpret_cast<const float4*>(ks + t * ld + n), *reinterpret_cast<const float4*>(after + r * dim4 + n)), dim - n, vec);
     }
-    __syncthreads();
-    float* within = p.within + ((size_t)ck.index * p.heads + head) * CT * CT;
-    for (int i = threadIdx.x; i < CT * CT; i += 256) within[i] = tile[(i % CT) * (CT + 1) + i / CT];
 }
 
 // ----------------------------------------------------------------------------- tiles of products
-constexpr int TILE = 64, KS = 16, LD = TILE + 4;
+// A block of PT_THREADS threads forms 64 x TN results (TN 64 or 128); thread (ty, tx) of 8 x 16 owns rows 8 ty .. + 7 and the columns
+// 4 tx .. + 3 of every 64.  The two operands pass through shared memory in slices of KS rows along the sum.  Results are kept
+// as pairs of neighbouring columns: one instruction multiplies and adds both (fma.rn.f32x2, two ordinary float operations).
+constexpr int TILE = 64, KS = 16, PT_THREADS = 128;
 
-// acc[8][4] += X^T Y for X [KS][TILE], Y [KS][TILE] in shared memory (rows LD apart): thread ty owns rows 8 ty .., tx columns 4 tx ..
-__device__ __forceinline__ void tile_fma(const float* xs, const float* ys, float (&acc)[8][4], int ty, int tx) {
+__device__ __forceinline__ unsigned long long pair_of(float a, float b) {
+    unsigned long long r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float2 unpair(unsigned long long v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ void fma_pair(unsigned long long& d, unsigned long long a, unsigned long long b) {
+    asm("fma.rn.f32x2 %0, %1, %2, %0;" : "+l"(d) : "l"(a), "l"(b));
+}
+
+template <int TN> struct Acc {
+    unsigned long long v[8][TN / 32];      // column pairs: 2 (p % 2) + 64 (p / 2) + 4 tx for pair p
+    __device__ __forceinline__ void clear() {
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+#pragma unroll
+            for (int j = 0; j < TN / 32; ++j) v[i][j] = 0ull;
+    }
+    __device__ __forceinline__ float4 quad(int i, int group) const {
+        const float2 a = unpair(v[i][2 * group]), b = unpair(v[i][2 * group + 1]);
+        return make_float4(a.x, a.y, b.x, b.y);
+    }
+    __device__ __forceinline__ void scale_row(int i, float f) {
+#pragma unroll
+        for (int j = 0; j < TN / 32; ++j) { const float2 a = unpair(v[i][j]); v[i][j] = pair_of(a.x * f, a.y * f); }
+    }
+};
+
+template <int TN> __device__ __forceinline__ void tile_fma(const float* xs, const float* ys, Acc<TN>& acc, int ty, int tx) {
+    constexpr int LDX = TILE + 4, LDY = TN + 4;
 #pragma unroll
     for (int k = 0; k < KS; ++k) {
-        const float4 a0 = *reinterpret_cast<const float4*>(xs + k * LD + 8 * ty), a1 = *reinterpret_cast<const float4*>(xs + k * LD + 8 * ty + 4);
-        const float4 b = *reinterpret_cast<const float4*>(ys + k * LD + 4 * tx);
+        const float4 a0 = *reinterpret_cast<const float4*>(xs + k * LDX + 8 * ty), a1 = *reinterpret_cast<const float4*>(xs + k * LDX + 8 * ty + 4);
+        unsigned long long b[TN / 32];
+#pragma unroll
+        for (int j = 0; j < TN / 64; ++j) {
+            const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(ys + k * LDY + 64 * j + 4 * tx);
+            b[2 * j] = v.x; b[2 * j + 1] = v.y;
+        }
         const float a[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-            acc[i][0] = fmaf(a[i], b.x, acc[i][0]); acc[i][1] = fmaf(a[i], b.y, acc[i][1]);
-            acc[i][2] = fmaf(a[i], b.z, acc[i][2]); acc[i][3] = fmaf(a[i], b.w, acc[i][3]);
+            const unsigned long long aa = pair_of(a[i], a[i]);
+#pragma unroll
+            for (int j = 0; j < TN / 32; ++j) fma_pair(acc.v[i][j], aa, b[j]);
         }
     }
 }
 
-constexpr int PT_THREADS = 128, PT_LOADS = TILE * KS / PT_THREADS;      // elements of a slice per thread
-
-// One slice of KS rows of a 64 x 64 product: x(k, i) and y(k, i) give elements (0 outside), with i or k running fastest over
-// neighbouring threads as the operand lies in memory.  The slice after next is fetched into registers under the arithmetic.
-template <bool X_K_FAST, bool Y_K_FAST, typename FX, typename FY>
-__device__ __forceinline__ void tile_product(int depth, FX x, FY y, float (&acc)[8][4], float* xs, float* ys) {
+// acc += sum over k < depth of x(k, i) y(k, n).  x and y return four neighbouring elements as they lie in memory (zeros outside):
+// along k for a K_FAST operand (element (k .. k + 3, i)), else along i.  The next slice is fetched under the arithmetic.
+template <int TN, bool X_K_FAST, bool Y_K_FAST, typename FX, typename FY>
+__device__ __forceinline__ void tile_product(int depth, FX x, FY y, Acc<TN>& acc, float* xs, float* ys) {
+    constexpr int LDX = TILE + 4, LDY = TN + 4, NX = TILE * KS / 4 / PT_THREADS, NY = TN * KS / 4 / PT_THREADS;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-    float xr[PT_LOADS], yr[PT_LOADS];
-    auto place = [&](int j, bool k_fast, int& k, int& i) {
-        const int e = threadIdx.x + j * PT_THREADS;
-        if (k_fast) { k = e % KS; i = e / KS; } else { k = e / TILE; i = e % TILE; }
-    };
+    float4 xr[NX], yr[NY];
     auto fetch = [&](int k0) {
 #pragma unroll
-        for (int j = 0; j < PT_LOADS; ++j) {
-            int k, i;
-            place(j, X_K_FAST, k, i);
-            xr[j] = k0 + k < depth ? x(k0 + k, i) : 0.f;
-            place(j, Y_K_FAST, k, i);
-            yr[j] = k0 + k < depth ? y(k0 + k, i) : 0.f;
+        for (int j = 0; j < NX; ++j) {
+            const int e = threadIdx.x + j * PT_THREADS;
+            xr[j] = X_K_FAST ? x(k0 + 4 * (e % (KS / 4)), e / (KS / 4)) : x(k0 + e / (TILE / 4), 4 * (e % (TILE / 4)));
+        }
+#pragma unroll
+        for (int j = 0; j < NY; ++j) {
+            const int e = threadIdx.x + j * PT_THREADS;
+            yr[j] = Y_K_FAST ? y(k0 + 4 * (e % (KS / 4)), e / (KS / 4)) : y(k0 + e / (TN / 4), 4 * (e % (TN / 4)));
+        }
+    };
+    auto place = [&](float* dst, int ld, const float4& v, bool k_fast, int e, int width) {
+        if (k_fast) {
+            const int k = 4 * (e % (KS / 4)), i = e / (KS / 4);
+            dst[k * ld + i] = v.x; dst[(k + 1) * ld + i] = v.y; dst[(k + 2) * ld + i] = v.z; dst[(k + 3) * ld + i] = v.w;
+        } else {
+            *reinterpret_cast<float4*>(dst + (e / (width / 4)) * ld + 4 * (e % (width / 4))) = v;
         }
     };
     fetch(0);
     for (int k0 = 0; k0 < depth; k0 += KS) {
         __syncthreads();
 #pragma unroll
-        for (int j = 0; j < PT_LOADS; ++j) {
-            int k, i;
-            place(j, X_K_FAST, k, i);
-            xs[k * LD + i] = xr[j];
-            place(j, Y_K_FAST, k, i);
-            ys[k * LD + i] = yr[j];
-        }
+        for (int j = 0; j < NX; ++j) place(xs, LDX, xr[j], X_K_FAST, threadIdx.x + j * PT_THREADS, TILE);
+#pragma unroll
+        for (int j = 0; j < NY; ++j) place(ys, LDY, yr[j], Y_K_FAST, threadIdx.x + j * PT_THREADS, TN);
         __syncthreads();
         if (k0 + KS < depth) fetch(k0 + KS);
-        tile_fma(xs, ys, acc, ty, tx);
+        tile_fma<TN>(xs, ys, acc, ty, tx);
     }
-}
-
-__device__ __forceinline__ void clear(float (&acc)[8][4]) {
-#pragma unroll
-    for (int i = 0; i < 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 }
 
 // ----------------------------------------------------------------------------- decays per head
 // grid (chunks of the longest sequence, heads, sequences), 128 threads.
-__global__ void __launch_bounds__(PT_THREADS) chunk_prepare_head_kernel(const ChunkArgs p) {
+__global__ void __launch_bounds__(PT_THREADS) chunk_prepare_head_kernel(const ChunkArgs p, int vec) {
     pdl_launch_dependents();
     pdl_wait();
-    __shared__ __align__(16) float xs[KS * LD];
-    __shared__ __align__(16) float ys[KS * LD];
+    __shared__ __align__(16) float xs[KS * (TILE + 4)];
+    __shared__ __align__(16) float ys[KS * (TILE + 4)];
     __shared__ double upto[CT];             // sum of g from the chunk's first token up to t
     __shared__ float scale[CT];
     const int head = blockIdx.y, key_head = head / p.heads_per_key;
@@ -263,20 +349,21 @@ __global__ void __launch_bounds__(PT_THREADS) chunk_prepare_head_kernel(const Ch
     }
     const float* q = p.rows + (size_t)ck.first * p.cols + p.at_q + (size_t)key_head * p.dim;
     const float* k = p.rows + (size_t)ck.first * p.cols + p.at_k + (size_t)key_head * p.dim;
-    float acc[8][4];                        // rows s, columns t
-    clear(acc);
-    tile_product<true, true>(p.dim, [&](int n, int s) { return s < ck.count ? k[(size_t)s * p.cols + n] : 0.f; },
-                             [&](int n, int t) { return t < ck.count ? q[(size_t)t * p.cols + n] : 0.f; }, acc, xs, ys);
+    Acc<TILE> acc;                          // rows s, columns t
+    acc.clear();
+    tile_product<TILE, true, true>(p.dim, [&](int n, int s) { return load4(k + (size_t)s * p.cols + n, s < ck.count ? p.dim - n : 0, vec); },
+                                   [&](int n, int t) { return load4(q + (size_t)t * p.cols + n, t < ck.count ? p.dim - n : 0, vec); }, acc, xs, ys);
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     float* within = p.within + ((size_t)ck.index * p.heads + head) * CT * CT;
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
         const int s = 8 * ty + i;
-        float v[4];
+        const float4 x = acc.quad(i, 0);
+        float v[4] = {x.x, x.y, x.z, x.w};
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int t = 4 * tx + j;
-            v[j] = s <= t && t < ck.count ? acc[i][j] * expf((float)(upto[t] - upto[s])) * scale[s] * p.out_scale : 0.f;
+            v[j] = s <= t && t < ck.count ? v[j] * expf((float)(upto[t] - upto[s])) * scale[s] * p.out_scale : 0.f;
         }
         *reinterpret_cast<float4*>(within + s * CT + 4 * tx) = make_float4(v[0], v[1], v[2], v[3]);
     }
@@ -284,31 +371,30 @@ __global__ void __launch_bounds__(PT_THREADS) chunk_prepare_head_kernel(const Ch
 
 // ----------------------------------------------------------------------------- what a chunk writes
 // grid (chunks x tiles of the state, heads, sequences), 128 threads: states[m][n] = sum_s v_s[m] k_s[n].
-template <bool PER_CHANNEL>
-__global__ void __launch_bounds__(PT_THREADS) chunk_write_kernel(const ChunkArgs p, int tiles_n, int tiles) {
+template <bool PER_CHANNEL, int TN>
+__global__ void __launch_bounds__(PT_THREADS) chunk_write_kernel(const ChunkArgs p, int tiles_n, int tiles, int vec_v, int vec_k, int vec_s) {
     pdl_launch_dependents();
     pdl_wait();
-    __shared__ __align__(16) float xs[KS * LD];
-    __shared__ __align__(16) float ys[KS * LD];
+    __shared__ __align__(16) float xs[KS * (TILE + 4)];
+    __shared__ __align__(16) float ys[KS * (TN + 4)];
     const int head = blockIdx.y, key_head = head / p.heads_per_key;
-    const int which = blockIdx.x % tiles, m0 = which / tiles_n * TILE, n0 = which % tiles_n * TILE;
+    const int which = blockIdx.x % tiles, m0 = which / tiles_n * TILE, n0 = which % tiles_n * TN;
     const Chunk ck = chunk_of(p, blockIdx.z, blockIdx.x / tiles);
     if (ck.count <= 0) return;
     const float* v = p.rows + (size_t)ck.first * p.cols + p.at_v + (size_t)head * p.vdim + m0;
-    const float* factor = p.k_to + (size_t)ck.first * p.heads + head;                               // per head: one per token
+    const float* factor = PER_CHANNEL ? (p.v_scale ? p.v_scale + (size_t)ck.first * p.heads + head : nullptr)      // one number per token
+                                      : p.k_to + (size_t)ck.first * p.heads + head;
     const float* k = PER_CHANNEL ? p.k_to + ((size_t)ck.first * p.heads + head) * p.dim + n0
                                  : p.rows + (size_t)ck.first * p.cols + p.at_k + (size_t)key_head * p.dim + n0;
     const size_t k_row = PER_CHANNEL ? (size_t)p.heads * p.dim : (size_t)p.cols;
-    const float* scale = PER_CHANNEL && p.v_scale ? p.v_scale + (size_t)ck.first * p.heads + head : nullptr;
-    float acc[8][4];
-    clear(acc);
-    tile_product<false, false>(ck.count,
+    Acc<TN> acc;
+    acc.clear();
+    tile_product<TN, false, false>(ck.count,
         [&](int s, int i) {
-            if (m0 + i >= p.vdim) return 0.f;
-            const float x = v[(size_t)s * p.cols + i];
-            return PER_CHANNEL ? (scale ? x * scale[(size_t)s * p.heads] : x) : x * factor[(size_t)s * p.heads];
+            const float4 x = load4(v + (size_t)s * p.cols + i, s < ck.count ? p.vdim - m0 - i : 0, vec_v);
+            return factor && s < ck.count ? times(x, __ldg(factor + (size_t)s * p.heads)) : x;
         },
-        [&](int s, int i) { return n0 + i < p.dim ? k[(size_t)s * k_row + i] : 0.f; }, acc, xs, ys);
+        [&](int s, int i) { return load4(k + (size_t)s * k_row + i, s < ck.count ? p.dim - n0 - i : 0, vec_k); }, acc, xs, ys);
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     float* dst = p.states + ((size_t)ck.index * p.heads + head) * p.vdim * p.dim;
 #pragma unroll
@@ -316,8 +402,10 @@ __global__ void __launch_bounds__(PT_THREADS) chunk_write_kernel(const ChunkArgs
         const int m = m0 + 8 * ty + i;
         if (m >= p.vdim) continue;
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-            if (n0 + 4 * tx + j < p.dim) dst[(size_t)m * p.dim + n0 + 4 * tx + j] = acc[i][j];
+        for (int j = 0; j < TN / 64; ++j) {
+            const int n = n0 + 64 * j + 4 * tx;
+            put4(dst + (size_t)m * p.dim + n, acc.quad(i, j), p.dim - n, vec_s);
+        }
     }
 }
 
@@ -374,13 +462,13 @@ __global__ void __launch_bounds__(256) chunk_pass_kernel(const ChunkArgs p) {
 
 // ----------------------------------------------------------------------------- what a chunk reads
 // grid (chunks x tiles of value columns, heads, sequences), 128 threads: out[t][m].
-template <bool PER_CHANNEL>
-__global__ void __launch_bounds__(PT_THREADS) chunk_read_kernel(const ChunkArgs p, int tiles) {
+template <bool PER_CHANNEL, int TN>
+__global__ void __launch_bounds__(PT_THREADS) chunk_read_kernel(const ChunkArgs p, int tiles, int vec_q, int vec_v, int vec_s, int vec_o) {
     pdl_launch_dependents();
     pdl_wait();
-    __shared__ __align__(16) float xs[KS * LD];
-    __shared__ __align__(16) float ys[KS * LD];
-    const int head = blockIdx.y, key_head = head / p.heads_per_key, m0 = blockIdx.x % tiles * TILE;
+    __shared__ __align__(16) float xs[KS * (TILE + 4)];
+    __shared__ __align__(16) float ys[KS * (TN + 4)];
+    const int head = blockIdx.y, key_head = head / p.heads_per_key, m0 = blockIdx.x % tiles * TN;
     const Chunk ck = chunk_of(p, blockIdx.z, blockIdx.x / tiles);
     if (ck.count <= 0) return;
     const float* q = PER_CHANNEL ? p.q_from + ((size_t)ck.first * p.heads + head) * p.dim
@@ -389,41 +477,50 @@ __global__ void __launch_bounds__(PT_THREADS) chunk_read_kernel(const ChunkArgs 
     const float* states = p.states + (((size_t)ck.index * p.heads + head) * p.vdim + m0) * p.dim;
     const float* within = p.within + ((size_t)ck.index * p.heads + head) * CT * CT;
     const float* v = p.rows + (size_t)ck.first * p.cols + p.at_v + (size_t)head * p.vdim + m0;
-    const float* scale = PER_CHANNEL && p.v_scale ? p.v_scale + (size_t)ck.first * p.heads + head : nullptr;
+    const float* factor = PER_CHANNEL && p.v_scale ? p.v_scale + (size_t)ck.first * p.heads + head : nullptr;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-    float acc[8][4];
-    clear(acc);
-    tile_product<true, true>(p.dim, [&](int n, int t) { return t < ck.count ? q[(size_t)t * q_row + n] : 0.f; },
-                             [&](int n, int i) { return m0 + i < p.vdim ? states[(size_t)i * p.dim + n] : 0.f; }, acc, xs, ys);
+    Acc<TN> acc;
+    acc.clear();
+    tile_product<TN, true, true>(p.dim, [&](int n, int t) { return load4(q + (size_t)t * q_row + n, t < ck.count ? p.dim - n : 0, vec_q); },
+                                 [&](int n, int i) { return load4(states + (size_t)i * p.dim + n, m0 + i < p.vdim ? p.dim - n : 0, vec_s); }, acc, xs, ys);
     if (!PER_CHANNEL) {
-        const float* factor = p.q_from + (size_t)ck.first * p.heads + head;
+        const float* from = p.q_from + (size_t)ck.first * p.heads + head;
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const float f = 8 * ty + i < ck.count ? factor[(size_t)(8 * ty + i) * p.heads] : 0.f;
-            acc[i][0] *= f; acc[i][1] *= f; acc[i][2] *= f; acc[i][3] *= f;
-        }
+        for (int i = 0; i < 8; ++i) acc.scale_row(i, 8 * ty + i < ck.count ? from[(size_t)(8 * ty + i) * p.heads] : 0.f);
     }
-    tile_product<false, false>(ck.count, [&](int s, int t) { return within[s * CT + t]; },
+    tile_product<TN, false, false>(ck.count, [&](int s, int t) { return load4(within + s * CT + t, s < ck.count ? 4 : 0, true); },
         [&](int s, int i) {
-            if (m0 + i >= p.vdim) return 0.f;
-            const float x = v[(size_t)s * p.cols + i];
-            return scale ? x * scale[(size_t)s * p.heads] : x;
+            const float4 x = load4(v + (size_t)s * p.cols + i, s < ck.count ? p.vdim - m0 - i : 0, vec_v);
+            return factor && s < ck.count ? times(x, __ldg(factor + (size_t)s * p.heads)) : x;
         }, acc, xs, ys);
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
         const int t = 8 * ty + i;
         if (t >= ck.count) continue;
-        float* dst = p.out + ((size_t)(ck.first + t) * p.heads + head) * p.vdim + m0 + 4 * tx;
+        float* dst = p.out + ((size_t)(ck.first + t) * p.heads + head) * p.vdim;
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-            if (m0 + 4 * tx + j < p.vdim) dst[j] = acc[i][j];
+        for (int j = 0; j < TN / 64; ++j) {
+            const int m = m0 + 64 * j + 4 * tx;
+            put4(dst + m, acc.quad(i, j), p.vdim - m, vec_o);
+        }
     }
+}
+
+bool aligned4(const void* p, std::initializer_list<int> strides) {
+    bool ok = (uintptr_t)p % 16 == 0;
+    for (int s : strides) ok = ok && s % 4 == 0;
+    return ok;
 }
 
 template <bool PER_CHANNEL>
 int run_chunks(const ChunkArgs& p, int n_seqs, int chunks, cudaStream_t s) {
+    // 16-byte accesses where the operand's rows start on 16-byte boundaries
+    const int vec_v = aligned4(p.rows, {p.cols, p.at_v, p.vdim}), vec_s = aligned4(p.states, {p.dim}), vec_o = aligned4(p.out, {p.vdim});
+    const int raw_q = aligned4(p.rows, {p.cols, p.at_q, p.dim}), raw_k = aligned4(p.rows, {p.cols, p.at_k, p.dim});
+    const int vec_q = PER_CHANNEL ? aligned4(p.q_from, {p.dim}) : raw_q, vec_k = PER_CHANNEL ? aligned4(p.k_to, {p.dim}) : raw_k;
     if (PER_CHANNEL) {
-        const size_t smem = ((size_t)3 * CT * (p.dim + 4) + (size_t)CT * (CT + 1) + (size_t)7 * p.dim) * sizeof(float);
+        const int dim4 = (p.dim + 3) / 4 * 4;
+        const size_t smem = ((size_t)3 * CT * (dim4 + 4) + (size_t)(4 + 3 + 8) * dim4) * sizeof(float);
         static bool configured = false;
         if (!configured) {
             cudaError_t err = cudaFuncSetAttribute(chunk_prepare_channel_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
@@ -431,20 +528,32 @@ int run_chunks(const ChunkArgs& p, int n_seqs, int chunks, cudaStream_t s) {
             configured = true;
         }
         QT_REQUIRE(smem <= 227 * 1024, "decayed_attention_chunked: %d key channels need more shared memory than a block has", p.dim);
-        launch_kernel(chunk_prepare_channel_kernel, dim3(chunks, p.heads, n_seqs), dim3(256), smem, s, p);
+        const int vec = raw_q && raw_k && vec_q && vec_k && aligned4(p.log_decay, {p.dim});
+        launch_kernel(chunk_prepare_channel_kernel, dim3(chunks, p.heads, n_seqs), dim3(PC_THREADS), smem, s, p, vec);
     } else {
-        launch_kernel(chunk_prepare_head_kernel, dim3(chunks, p.heads, n_seqs), dim3(PT_THREADS), 0, s, p);
+        launch_kernel(chunk_prepare_head_kernel, dim3(chunks, p.heads, n_seqs), dim3(PT_THREADS), 0, s, p, (int)(raw_q && raw_k));
     }
     QT_CHECK_LAUNCH("chunk_prepare");
-    const int tiles_m = (p.vdim + TILE - 1) / TILE, tiles_n = (p.dim + TILE - 1) / TILE;
-    launch_kernel(chunk_write_kernel<PER_CHANNEL>, dim3(chunks * tiles_m * tiles_n, p.heads, n_seqs), dim3(PT_THREADS), 0, s, p, tiles_n, tiles_m * tiles_n);
+    const int tiles_m = (p.vdim + TILE - 1) / TILE;
+    if (p.dim > 64) {
+        const int tiles_n = (p.dim + 127) / 128;
+        launch_kernel(chunk_write_kernel<PER_CHANNEL, 128>, dim3(chunks * tiles_m * tiles_n, p.heads, n_seqs), dim3(PT_THREADS), 0, s, p, tiles_n, tiles_m * tiles_n,
+                      vec_v, vec_k, vec_s);
+    } else {
+        launch_kernel(chunk_write_kernel<PER_CHANNEL, 64>, dim3(chunks * tiles_m, p.heads, n_seqs), dim3(PT_THREADS), 0, s, p, 1, tiles_m, vec_v, vec_k, vec_s);
+    }
     QT_CHECK_LAUNCH("chunk_write");
     const int size = p.vdim * p.dim;
-    const bool wide = p.dim % 4 == 0 && (uintptr_t)p.state % 16 == 0 && (uintptr_t)p.states % 16 == 0 && (uintptr_t)p.whole % 16 == 0;
+    const bool wide = vec_s && aligned4(p.state, {}) && aligned4(p.whole, {});
     if (wide) launch_kernel(chunk_pass_kernel<PER_CHANNEL, 4>, dim3((size + 1023) / 1024, p.heads, n_seqs), dim3(256), 0, s, p);
     else launch_kernel(chunk_pass_kernel<PER_CHANNEL, 1>, dim3((size + 255) / 256, p.heads, n_seqs), dim3(256), 0, s, p);
     QT_CHECK_LAUNCH("chunk_pass");
-    launch_kernel(chunk_read_kernel<PER_CHANNEL>, dim3(chunks * tiles_m, p.heads, n_seqs), dim3(PT_THREADS), 0, s, p, tiles_m);
+    if (p.vdim > 64) {
+        const int tiles = (p.vdim + 127) / 128;
+        launch_kernel(chunk_read_kernel<PER_CHANNEL, 128>, dim3(chunks * tiles, p.heads, n_seqs), dim3(PT_THREADS), 0, s, p, tiles, vec_q, vec_v, vec_s, vec_o);
+    } else {
+        launch_kernel(chunk_read_kernel<PER_CHANNEL, 64>, dim3(chunks, p.heads, n_seqs), dim3(PT_THREADS), 0, s, p, 1, vec_q, vec_v, vec_s, vec_o);
+    }
     QT_CHECK_LAUNCH("chunk_read");
     return QT_OK;
 }

@@ -32,9 +32,17 @@ struct ConvParams {
     int n_tokens, nq, nkv, d, n_taps, page_tokens, ring_tokens, write_kv;
 };
 
+// The sum of split-K partial sums in their order, eight loads in flight at a time.
 __device__ __forceinline__ float sum_splits(const float* __restrict__ base, size_t index, int n_splits, size_t split_stride) {
-    float acc = base[index];
-    for (int s = 1; s < n_splits; ++s) acc += base[index + (size_t)s * split_stride];
+    if (n_splits == 1) return base[index];
+    float acc = 0.f;
+    for (int s0 = 0; s0 < n_splits; s0 += 8) {
+        float v[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = s0 + j < n_splits ? base[index + (size_t)(s0 + j) * split_stride] : 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc += v[j];
+    }
     return acc;
 }
 
@@ -129,21 +137,22 @@ struct ConvActParams {
     int at_step, heads;               // the columns of the heads' step sizes (heads 0: none)
     const float* step_bias; const float* rate_log;       // [heads]
     float* step; float* log_decay;    // [T, heads]
+    int run;                          // consecutive tokens a thread walks (at most CA_TOKENS)
     int n_tokens, n_taps, keep;       // keep: every sequence brings one token, and its kept inputs are shifted here
 };
 
-constexpr int CA_TOKENS = 8;          // consecutive tokens of a channel that one thread walks
+constexpr int CA_TOKENS = 8;          // consecutive tokens of a channel that one thread walks in a step of many
 
 __device__ __forceinline__ float conv_silu(float y) { return y / (1.f + expf(-y)); }
 
-// grid (blocks of 128 columns: the channels, then the heads; runs of CA_TOKENS tokens).  TAPS > 0: the inputs of the last TAPS
+// grid (blocks of 128 columns: the channels, then the heads; runs of `run` tokens).  TAPS > 0: the inputs of the last TAPS
 // tokens stay in registers from token to token; 0: any number of taps, read again for every token.
 template <int TAPS>
 __global__ void __launch_bounds__(128) conv_act_kernel(const ConvActParams p) {
     pdl_launch_dependents();
     pdl_wait();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
-    const int t0 = blockIdx.y * CA_TOKENS, t1 = min(p.n_tokens, t0 + CA_TOKENS);
+    const int t0 = blockIdx.y * p.run, t1 = min(p.n_tokens, t0 + p.run);
     if (c >= p.channels) {
         const int h = c - p.channels;
         if (h >= p.heads) return;
@@ -167,6 +176,22 @@ __global__ void __launch_bounds__(128) conv_act_kernel(const ConvActParams p) {
         float w[N], u[N];
 #pragma unroll
         for (int j = 0; j < N; ++j) w[j] = p.taps[(size_t)c * N + j];
+        const int first = p.token_seq[t0];
+        if (t1 - t0 == CA_TOKENS && p.n_splits == 1 && p.token_seq[t1 - 1] == first && !p.keep) {
+            // the usual run of a long step, all tokens of one sequence: every input is asked for before the first is used
+            const int row0 = p.seq_start[first];
+            float x[CA_TOKENS + N - 1];
+#pragma unroll
+            for (int j = 0; j < CA_TOKENS + N - 1; ++j) x[j] = input(first, row0, t0 - row0 - (N - 1) + j);
+#pragma unroll
+            for (int i = 0; i < CA_TOKENS; ++i) {
+                float y = 0.f;
+#pragma unroll
+                for (int j = 0; j < N; ++j) y += w[j] * x[i + j];
+                p.out[(size_t)(t0 + i) * p.channels + c] = conv_silu(y + b);
+            }
+            return;
+        }
         int before = -1;
         for (int t = t0; t < t1; ++t) {
             const int seq = p.token_seq[t], row0 = p.seq_start[seq], local = t - row0;
@@ -211,10 +236,11 @@ extern "C" int qt_conv_act(const float* proj, int n_splits, long long split_stri
     QT_REQUIRE(n_seqs <= 65535 && (n_tokens + CA_TOKENS - 1) / CA_TOKENS <= 65535, "conv_act: too many tokens or sequences for one launch");
     if (n_tokens == 0) return QT_OK;
     cudaStream_t s = (cudaStream_t)stream;
+    const int run = n_tokens >= 256 ? CA_TOKENS : 1;                 // few tokens: a thread each, so that the launch fills the machine
     const int keep = one_token && n_taps <= 4 && n_tokens == n_seqs ? 1 : 0;
     ConvActParams p{proj, n_splits, (size_t)split_stride, proj_cols, at, channels, taps, bias, kept, token_seq, seq_start, slots, out,
-                    at_step, heads, step_bias, rate_log, step, log_decay, n_tokens, n_taps, keep};
-    const dim3 grid((channels + heads + 127) / 128, (n_tokens + CA_TOKENS - 1) / CA_TOKENS);
+                    at_step, heads, step_bias, rate_log, step, log_decay, run, n_tokens, n_taps, keep};
+    const dim3 grid((channels + heads + 127) / 128, (n_tokens + run - 1) / run);
     switch (n_taps) {
         case 1: launch_kernel(conv_act_kernel<1>, grid, dim3(128), 0, s, p); break;
         case 2: launch_kernel(conv_act_kernel<2>, grid, dim3(128), 0, s, p); break;

@@ -62,7 +62,8 @@ class LatentAttention:
         self.at_gate = self.q_rank + (self.row if self.own_kv else 0)
         used = self.at_gate + (self.heads * (1 if self.head_gate else self.dv) if self.gated else 0)
         self.proj_rows = -(-used // 8) * 8
-        self.proj = Linear("latent.proj" + ("" if self.own_kv else ".reader"), self.proj_rows, self.hidden, runtime, float_out=True)
+        self.proj = Linear("latent.proj" + ("" if self.own_kv else ".reader"), self.proj_rows, self.hidden, runtime, float_out=True, role="qkv")
+        self.takes_scaled_rows = self.proj.fused_capable
         self.uq = Linear("latent.uq", self.heads * (self.d + self.rot), self.q_rank, runtime)
         float_out = bool(params.get("float_out", False))
         self.o = Linear("latent.o" + (".float" if float_out else ""), self.hidden, self.heads * self.dv, runtime, float_out=float_out, role="attn_out")
@@ -156,7 +157,7 @@ class LatentAttention:
         if cache.k is None or cache.k.shape[-1] != self.row:
             raise ValueError(f"{self.prefix}: the cache rows it reads are not {self.rank} + {self.rot} elements long")
         table = ctx.block_table(cache.group)
-        proj = self.proj(x)
+        proj = self.proj.finished(x)
         cq = ws.view("latent.cq", tokens, self.q_rank)
         kernels.latent_prepare(proj, self.q_norm, self.kv_norm, self.eps, self.cos_sin, cq, cache.k if write else None, ctx.token_seq,
                                ctx.token_pos, table if write else None, self.rank, self.rot, cache.page_tokens, cache.ring_tokens, write_kv=write)

@@ -220,6 +220,16 @@ class Linear:
         kernels.gemm(x, self.weight, result, self._loaded_bias())
         return result
 
+    def finished(self, x) -> GemmOut:
+        """The product as one plane: for few rows the fused product, whose blocks add their K ranges on the chip (and apply the
+        factor of ``ScaledRows``), where the plain one would hand partial sums to every reader."""
+        rows = x.shape[0]
+        if isinstance(x, ScaledRows) or not (self.float_out and self.fusable(rows)):
+            return self(x)
+        out = self.runtime.workspace.view(f"{self.key}.out", rows, self.out_features)
+        kernels.gemm_fused_store(x, self.weight, out, splits=self._fused_splits(rows), stages=self._fused_stages(rows), bias=self._loaded_bias())
+        return GemmOut(out.view(1, rows, self.out_features))
+
     def _loaded_bias(self) -> torch.Tensor | None:
         if self.has_bias and self.bias is None:
             raise ValueError(f"{self.key}: the bias was not loaded")

@@ -337,7 +337,8 @@ class GatedLinearAttention(_DecayedMixer):
         self.at_gate = self.at_v + self.heads * self.vdim
         self.at_decay = self.at_gate + self.heads * self.vdim
         self.proj_rows = -(-(self.at_decay + self.rank) // 8) * 8
-        self.proj = Linear("gla.proj", self.proj_rows, self.hidden, runtime, float_out=True)
+        self.proj = Linear("gla.proj", self.proj_rows, self.hidden, runtime, float_out=True, role="qkv")
+        self.takes_scaled_rows = self.proj.fused_capable
         float_out = bool(params.get("float_out", False))
         self.o = Linear("gla.o" + (".float" if float_out else ""), self.hidden, self.heads * self.vdim, runtime, float_out=float_out, role="attn_out")
         ws = runtime.workspace
@@ -387,7 +388,7 @@ class GatedLinearAttention(_DecayedMixer):
         self._check(cache)
         tokens, width = x.shape[0], self.heads * self.vdim
         ws = self.runtime.workspace
-        proj = self.proj(x)
+        proj = self.proj.finished(x)
         decay = ws.view("gla.decay", tokens, self.heads, self.dim)
         kernels.lowrank(proj, self.at_decay, self.decay_out, decay.view(tokens, self.heads * self.dim), self.decay_bias, power=1.0 / self.tau)
         # split sums are added once, not by every block of the recurrence that reads them
@@ -436,7 +437,8 @@ class StateSpace(_DecayedMixer):
         self.at_step = self.inner + self.channels
         self.rows = self.at_step + self.heads
         self.proj_rows = -(-self.rows // 8) * 8
-        self.proj = Linear("ssm.proj", self.proj_rows, self.hidden, runtime, float_out=True)
+        self.proj = Linear("ssm.proj", self.proj_rows, self.hidden, runtime, float_out=True, role="qkv")
+        self.takes_scaled_rows = self.proj.fused_capable
         float_out = bool(params.get("float_out", False))
         self.o = Linear("ssm.o" + (".float" if float_out else ""), self.hidden, self.inner, runtime, float_out=float_out, role="attn_out")
         ws, tokens = runtime.workspace, runtime.max_step_tokens
@@ -489,7 +491,7 @@ class StateSpace(_DecayedMixer):
         self._check(states)
         tokens = x.shape[0]
         ws = self.runtime.workspace
-        proj = self.proj(x)
+        proj = self.proj.finished(x)
         mixed = ws.view("ssm.mixed", tokens, self.channels)
         step, decay = ws.view("ssm.step", tokens, self.heads), ws.view("ssm.decay", tokens, self.heads)
         kernels.conv_act(proj, self.inner, self.conv, self.conv_bias, kept.state, ctx, mixed, self.at_step, self.step_bias, self.rate_log, step, decay)
