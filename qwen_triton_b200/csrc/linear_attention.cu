@@ -465,22 +465,23 @@ struct GroupNormParams {
     int width, part, silu, gate_first;
 };
 
-__device__ __forceinline__ float gn_gate(const GroupNormParams& p, size_t t, int i) {
+__device__ __forceinline__ float gn_gate_sum(const GroupNormParams& p, size_t t, int i) {
     const float* at = p.proj + t * p.proj_cols + p.at_gate + i;
     float g = 0.f;
-    if (p.n_splits == 1) g = __ldg(at);
-    else {
-        for (int s0 = 0; s0 < p.n_splits; s0 += 8) {                    // eight loads of a split product's planes in flight
-            float v[8];
+    for (int s0 = 0; s0 < p.n_splits; s0 += 8) {                        // eight loads of a split product's planes in flight
+        float v[8];
 #pragma unroll
-            for (int j = 0; j < 8; ++j) v[j] = s0 + j < p.n_splits ? __ldg(at + (size_t)(s0 + j) * p.split_stride) : 0.f;
+        for (int j = 0; j < 8; ++j) v[j] = s0 + j < p.n_splits ? __ldg(at + (size_t)(s0 + j) * p.split_stride) : 0.f;
 #pragma unroll
-            for (int j = 0; j < 8; ++j) g += v[j];
-        }
+        for (int j = 0; j < 8; ++j) g += v[j];
     }
+    return g;
+}
+__device__ __forceinline__ float gn_gate_value(const GroupNormParams& p, float g) {
     const float sig = 1.f / (1.f + expf(-g));
     return p.silu ? g * sig : sig;
 }
+__device__ __forceinline__ float gn_gate(const GroupNormParams& p, size_t t, int i) { return gn_gate_value(p, gn_gate_sum(p, t, i)); }
 __device__ __forceinline__ float gn_value(const GroupNormParams& p, size_t t, int i) {
     float y = __ldg(p.o + t * p.width + i);
     if (p.x) y += __ldg(p.skip + i / p.per_skip) * __ldg(p.x + t * p.x_cols + p.at_x + i);
@@ -491,7 +492,8 @@ __device__ __forceinline__ float gn_value(const GroupNormParams& p, size_t t, in
 // beyond what the registers hold are formed again in the second pass.  grid (tokens, blocks of parts).
 constexpr int GN_CACHE = 8;
 
-template <typename TO, bool WARP>
+// ONE_PLANE: the gate's sums are finished, so a thread asks for everything it needs before it uses the first value.
+template <typename TO, bool WARP, bool ONE_PLANE>
 __global__ void group_gate_norm_kernel(const GroupNormParams p, TO* __restrict__ out) {
     pdl_launch_dependents();
     pdl_wait();
@@ -501,14 +503,27 @@ __global__ void group_gate_norm_kernel(const GroupNormParams p, TO* __restrict__
     if (WARP && part * p.part >= p.width) return;                       // whole warps leave; a block's threads stay together otherwise
     const int first = WARP ? threadIdx.x & 31 : threadIdx.x, step = WARP ? 32 : blockDim.x, base = part * p.part;
     float y[GN_CACHE], gate[GN_CACHE], sq = 0.f;
+    const float* o = p.o + t * p.width + base;
+    const float* x = p.x ? p.x + t * p.x_cols + p.at_x + base : nullptr;
+    const float* g = p.proj ? p.proj + t * p.proj_cols + p.at_gate + base : nullptr;
 #pragma unroll
     for (int j = 0; j < GN_CACHE; ++j) {
         const int i = first + j * step;
-        y[j] = i < p.part ? gn_value(p, t, base + i) : 0.f;
-        gate[j] = i < p.part && p.proj ? gn_gate(p, t, base + i) : 1.f;
+        const bool in = i < p.part;
+        y[j] = in ? __ldg(o + i) : 0.f;
+        if (ONE_PLANE) gate[j] = in && g ? __ldg(g + i) : 0.f;
+        else gate[j] = in && g ? gn_gate_sum(p, t, base + i) : 0.f;
+    }
+    if (x) {
+#pragma unroll
+        for (int j = 0; j < GN_CACHE; ++j) {
+            const int i = first + j * step;
+            if (i < p.part) y[j] = fmaf(__ldg(p.skip + (base + i) / p.per_skip), __ldg(x + i), y[j]);
+        }
     }
 #pragma unroll
     for (int j = 0; j < GN_CACHE; ++j) {
+        gate[j] = g ? gn_gate_value(p, gate[j]) : 1.f;
         if (p.gate_first) { y[j] *= gate[j]; gate[j] = 1.f; }
         sq += y[j] * y[j];
     }
@@ -537,13 +552,17 @@ extern "C" int qt_group_gate_norm(const float* o, const float* x, int x_cols, in
     GroupNormParams p{o, x, x_cols, at_x, skip, x ? width / skips : 1, proj, n_splits, (size_t)split_stride, proj_cols, at_gate, weight, weight_len, eps, scale,
                       width, part, silu, gate_first};
     return QT_DISPATCH_DTYPE(out_dtype, "group_gate_norm", {
+        const bool one = n_splits == 1;
         if (groups > 1 && part <= 32 * GN_CACHE) {
-            launch_kernel(group_gate_norm_kernel<T, true>, dim3(n_tokens, (groups + 3) / 4), dim3(128), 0, s, p, (T*)out);
+            const dim3 grid(n_tokens, (groups + 3) / 4);
+            if (one) launch_kernel(group_gate_norm_kernel<T, true, true>, grid, dim3(128), 0, s, p, (T*)out);
+            else launch_kernel(group_gate_norm_kernel<T, true, false>, grid, dim3(128), 0, s, p, (T*)out);
         } else {
             int threads = ((part + GN_CACHE * 32 - 1) / (GN_CACHE * 32)) * 32;      // 8 elements a thread; few tokens: fewer each
             if (n_tokens < 256) threads = ((part + 63) / 64) * 32;
-            threads = threads < 128 ? 128 : threads > 1024 ? 1024 : threads;
-            launch_kernel(group_gate_norm_kernel<T, false>, dim3(n_tokens, groups), dim3(threads), 0, s, p, (T*)out);
+            threads = threads < 64 ? 64 : threads > 1024 ? 1024 : threads;
+            if (one) launch_kernel(group_gate_norm_kernel<T, false, true>, dim3(n_tokens, groups), dim3(threads), 0, s, p, (T*)out);
+            else launch_kernel(group_gate_norm_kernel<T, false, false>, dim3(n_tokens, groups), dim3(threads), 0, s, p, (T*)out);
         }
         QT_CHECK_LAUNCH("group_gate_norm");
         return QT_OK;

@@ -13,10 +13,10 @@
 //                                e^{G(start, end)} of a (chunk, head).
 // chunk_prepare_head_kernel      g per head: A = (q_t . k_s) e^{G(s, t)} times the factor on v_s, and per token e^{G(start, t)} and
 //                                e^{G(s, end)} times that factor; q and k themselves (which several heads may share) stay as they are.
-// chunk_write_kernel             sum_s (e^{G(s, end)} k_s) v_s^T of a (chunk, head): a 64 x 64 x 64 product per tile.
+// chunk_write_kernel             sum_s (e^{G(s, end)} k_s) v_s^T of a (chunk, head): a product over its tokens per tile of 64 x 64 or 64 x 128.
 // chunk_pass_kernel              walks a sequence's chunks elementwise: puts S_c in the place of what chunk c writes, and the last
 //                                state back into the sequence's row.
-// chunk_read_kernel              o of a (chunk, head): two products per 64 x 64 tile, over the state's rows and over the chunk's tokens.
+// chunk_read_kernel              o of a (chunk, head): two products per tile, over the state's rows and over the chunk's tokens.
 //
 // The chunk c of sequence i has the scratch index seq_start[i] / CT + i + c, which is below T / CT + (sequences) and distinct
 // for distinct chunks.  States (and their scratch) are stored transposed, [heads, vdim, dim], as in linear_attention.cu.
