@@ -200,7 +200,8 @@ __global__ void __launch_bounds__(32 * LA_LANES) linear_attention_step_kernel(co
     const int key_head = MODE == LA_CONSTANT ? head : head / p.heads_per_key;
     const bool live = col < p.vdim;
     float* state = p.state + (((size_t)p.slots[seq] * p.heads + head) * p.vdim + (live ? col : 0)) * p.dim;
-    const int row0 = lane * RPL;
+    const int row0 = 4 * lane;                              // this lane holds rows 4 lane + at(i): its 16-byte pieces lie beside its neighbours'
+    auto at = [](int i) { return i / 4 * 4 * LA_LANES + i % 4; };
     const bool vec = p.dim % 4 == 0 && ((uintptr_t)p.state & 15) == 0;
     float S[RPL];
 #pragma unroll
@@ -209,14 +210,14 @@ __global__ void __launch_bounds__(32 * LA_LANES) linear_attention_step_kernel(co
         if (vec) {
 #pragma unroll
             for (int i = 0; i < RPL; i += 4)
-                if (row0 + i < p.dim) {
-                    const float4 v = *reinterpret_cast<const float4*>(state + row0 + i);
+                if (row0 + at(i) < p.dim) {
+                    const float4 v = *reinterpret_cast<const float4*>(state + row0 + at(i));
                     S[i] = v.x; S[i + 1] = v.y; S[i + 2] = v.z; S[i + 3] = v.w;
                 }
         } else {
 #pragma unroll
             for (int i = 0; i < RPL; ++i)
-                if (row0 + i < p.dim) S[i] = state[row0 + i];
+                if (row0 + at(i) < p.dim) S[i] = state[row0 + at(i)];
         }
     }
     const bool quads = p.n_splits == 1 && p.dim % 4 == 0 && p.at_q % 4 == 0 && p.at_k % 4 == 0 && p.proj_cols % 4 == 0 && ((uintptr_t)p.proj & 15) == 0;
@@ -229,9 +230,17 @@ __global__ void __launch_bounds__(32 * LA_LANES) linear_attention_step_kernel(co
             const size_t th = (size_t)t * p.heads + head;
             if (p.v_scale) v *= __ldg(p.v_scale + th);
             if (MODE == LA_PER_HEAD) decay[0] = expf(__ldg(p.log_decay + th));
-            else {
+            else if (vec && ((uintptr_t)p.log_decay & 15) == 0) {
 #pragma unroll
-                for (int i = 0; i < (MODE == LA_PER_CHANNEL ? RPL : 1); ++i) decay[i] = row0 + i < p.dim ? expf(__ldg(p.log_decay + th * p.dim + row0 + i)) : 0.f;
+                for (int i = 0; i < (MODE == LA_PER_CHANNEL ? RPL : 1); i += 4) {
+                    const float4 g = row0 + at(i) < p.dim ? __ldg(reinterpret_cast<const float4*>(p.log_decay + th * p.dim + row0 + at(i))) : make_float4(0.f, 0.f, 0.f, 0.f);
+                    const float e[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) if (MODE == LA_PER_CHANNEL) decay[(i + j) % (MODE == LA_PER_CHANNEL ? RPL : 1)] = e[j];
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < (MODE == LA_PER_CHANNEL ? RPL : 1); ++i) decay[i] = row0 + at(i) < p.dim ? __ldg(p.log_decay + th * p.dim + row0 + at(i)) : 0.f;
             }
         }
         float q[RPL], k[RPL];
@@ -239,19 +248,23 @@ __global__ void __launch_bounds__(32 * LA_LANES) linear_attention_step_kernel(co
         if (quads) {                                        // 16-byte loads of a row that is finished and aligned
 #pragma unroll
             for (int i = 0; i < RPL; i += 4) {
-                const bool has = row0 + i < p.dim;
-                const float4 q4 = has ? __ldg(reinterpret_cast<const float4*>(p.proj + q_at + i)) : make_float4(0.f, 0.f, 0.f, 0.f);
-                const float4 k4 = has ? __ldg(reinterpret_cast<const float4*>(p.proj + k_at + i)) : make_float4(0.f, 0.f, 0.f, 0.f);
+                const bool has = row0 + at(i) < p.dim;
+                const float4 q4 = has ? __ldg(reinterpret_cast<const float4*>(p.proj + q_at + at(i))) : make_float4(0.f, 0.f, 0.f, 0.f);
+                const float4 k4 = has ? __ldg(reinterpret_cast<const float4*>(p.proj + k_at + at(i))) : make_float4(0.f, 0.f, 0.f, 0.f);
                 q[i] = q4.x; q[i + 1] = q4.y; q[i + 2] = q4.z; q[i + 3] = q4.w;
                 k[i] = k4.x; k[i + 1] = k4.y; k[i + 2] = k4.z; k[i + 3] = k4.w;
             }
         } else {
 #pragma unroll
             for (int i = 0; i < RPL; ++i) {                 // every load of the token ahead of its arithmetic
-                const bool has = row0 + i < p.dim;
-                q[i] = has ? la_raw(p, q_at + i) : 0.f;
-                k[i] = has ? la_raw(p, k_at + i) : 0.f;
+                const bool has = row0 + at(i) < p.dim;
+                q[i] = has ? la_raw(p, q_at + at(i)) : 0.f;
+                k[i] = has ? la_raw(p, k_at + at(i)) : 0.f;
             }
+        }
+        if (MODE == LA_PER_CHANNEL) {                           // the logarithms are turned once everything has been asked for
+#pragma unroll
+            for (int i = 0; i < (MODE == LA_PER_CHANNEL ? RPL : 1); ++i) decay[i] = expf(decay[i]);
         }
         float a0 = 0.f, a1 = 0.f;
 #pragma unroll
@@ -269,11 +282,11 @@ __global__ void __launch_bounds__(32 * LA_LANES) linear_attention_step_kernel(co
         if (vec) {
 #pragma unroll
             for (int i = 0; i < RPL; i += 4)
-                if (row0 + i < p.dim) *reinterpret_cast<float4*>(state + row0 + i) = make_float4(S[i], S[i + 1], S[i + 2], S[i + 3]);
+                if (row0 + at(i) < p.dim) *reinterpret_cast<float4*>(state + row0 + at(i)) = make_float4(S[i], S[i + 1], S[i + 2], S[i + 3]);
         } else {
 #pragma unroll
             for (int i = 0; i < RPL; ++i)
-                if (row0 + i < p.dim) state[row0 + i] = S[i];
+                if (row0 + at(i) < p.dim) state[row0 + at(i)] = S[i];
         }
     }
 }
