@@ -124,7 +124,8 @@ __global__ void __launch_bounds__(LT_THREADS, 1) latent_attention_kernel(const L
     const int last_row = q0 + rows - 1;
     const int qpos[2] = {past + min(q0 + rg * 16 + g, last_row) / heads, past + min(q0 + rg * 16 + g + 8, last_row) / heads};
     const int warp_pos_min = past + min(q0 + rg * 16, last_row) / heads, warp_pos_max = past + min(q0 + rg * 16 + 15, last_row) / heads;
-    // of the keys at and above a warp's first position, those below `low_min` are hidden from its first row, and a page wholly below from all
+    // under a window: the first key that the warp's first row sees (a page wholly before it is skipped) and that its last row sees (a page
+    // that starts before it is masked element by element, by the rows' own first keys in `low`)
     const int low_min = p.window > 0 ? warp_pos_min - p.window + 1 : -1, low_max = p.window > 0 ? warp_pos_max - p.window + 1 : -1;
     const int low[2] = {p.window > 0 ? qpos[0] - p.window + 1 : -1, p.window > 0 ? qpos[1] - p.window + 1 : -1};
     const uint32_t q_frag = q_s + (uint32_t)((rg * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * lds + (lane >> 4) * 8) * 2u;
