@@ -5,6 +5,7 @@ from .vunepel import VunepelConfig
 from .bisodra import BisodraConfig
 from .regupel import RegupelConfig
 from .misudra import MisudraConfig
+from .bizurax import BizuraxConfig
 from .registry import (
     config_from_dict,
     load_config,
@@ -21,9 +22,10 @@ register_architecture("Vunepel", VunepelConfig)
 register_architecture("Bisodra", BisodraConfig)
 register_architecture("Regupel", RegupelConfig)
 register_architecture("Misudra", MisudraConfig)
+register_architecture("Bizurax", BizuraxConfig)
 
 __all__ = [
-    "BisodraConfig", "ConfigError", "LayerCall", "LayerSpec", "LederaxConfig", "MisudraConfig", "ModelSpec", "PartSpec", "Qwen3Config", "RegupelConfig", "VunepelConfig",
+    "BisodraConfig", "BizuraxConfig", "ConfigError", "LayerCall", "LayerSpec", "LederaxConfig", "MisudraConfig", "ModelSpec", "PartSpec", "Qwen3Config", "RegupelConfig", "VunepelConfig",
     "config_from_dict", "load_config", "load_config_dict", "load_preset", "preset_names",
     "register_architecture", "registered_architectures",
 ]

@@ -88,11 +88,14 @@ class ModelSpec:
     head: PartSpec
     max_positions: int
     eos_token_ids: tuple[int, ...] = ()
+    streams: int | None = None             # parallel copies of the residual stream (None: the plain one, which most blocks and norms expect)
     entries: Sequence[PartSpec] = ()       # stream maps that calls of the schedule name (``LayerCall.entry``)
 
     def validate(self) -> None:
         if self.vocab_size <= 0 or self.hidden_size <= 0:
             raise ValueError("vocab_size and hidden_size must be positive")
+        if self.streams is not None and self.streams < 1:
+            raise ValueError(f"streams={self.streams} must be positive")
         if not self.layers:
             raise ValueError("a model needs at least one layer")
         for pos, call in enumerate(self.schedule):

@@ -12,7 +12,8 @@
 // query also sees the keys at positions below `keep_first`, at their true distances.  With `sink` the softmax has one
 // more term of score 0 that carries no value: p_j = exp(s_j) / (1 + sum exp(s_j)); with `sinks` (one float per query head) the
 // term's score is the head's number, taken as it is (not scaled).  `v_row` is the length of a value
-// row in the value cache where it is longer than `dv` (values that are the leading elements of the cached keys).
+// row in the value cache where it is longer than `dv` (values that are the leading elements of the cached keys).  With `softcap`
+// > 0 a score s becomes softcap tanh(s / softcap) before everything else (the sink's score does not).
 //
 // Counterparts in luozoupi/Qwen-Triton: kernels/flash_attention.py:54-152 (one kernel for both
 // cases, no split, no window) and the masked SDPA branch of modules/attention.py:110-123 with
@@ -42,6 +43,7 @@ struct AttnParams {
     int sink;             // 1: one more softmax term of score 0 without a value
     int v_row;            // elements between the value rows of neighbouring tokens (dv unless the rows are longer)
     const float* sinks;   // [nq] the sink term's score per query head (null: 0)
+    float softcap;        // > 0: scores pass softcap tanh(s / softcap)
 };
 
 // r2 < 0 marks the linear form r1 * distance
@@ -132,6 +134,7 @@ __global__ void __launch_bounds__(PF_WARPS * 32) attention_prefill_kernel(const 
             const int pos = past + q0 + r;
             float s = 0.f;
             for (int c = 0; c < d; ++c) s += qs[r * d + c] * ks[lane * kstride + c];
+            if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
             const bool visible = r < rows && key < range_hi && key <= pos &&
                                  (p.window <= 0 || key > pos - p.window || key < p.keep_first) &&
                                  (p.chunk <= 0 || key >= pos / p.chunk * p.chunk);
@@ -211,7 +214,7 @@ extern "C" int qt_attention_prefill(const void* q, const void* k_cache, const vo
                                     const int* block_table, int max_blocks, const int* seq_start, const int* seq_past,
                                     int n_seqs, int max_q_len, int nq, int nkv, int d, int page_tokens, int ring_tokens,
                                     int window, float scale, int dv, const float* r1, const float* r2, int chunk, int nv,
-                                    int keep_first, int sink, int v_row, const float* sinks, void* stream) {
+                                    int keep_first, int sink, int v_row, const float* sinks, float softcap, void* stream) {
     if (n_seqs == 0 || max_q_len == 0) return QT_OK;
     if (nv <= 0) nv = nkv;
     if (v_row <= 0) v_row = dv;
@@ -219,7 +222,7 @@ extern "C" int qt_attention_prefill(const void* q, const void* k_cache, const vo
     if (rc) return rc;
     QT_REQUIRE(nq <= 65535 && n_seqs <= 65535, "attention_prefill: too many heads or sequences for one launch");
     AttnParams p{q, k_cache, v_cache, out, block_table, max_blocks, seq_start, seq_past, n_seqs, nq, nkv, d, page_tokens, ring_tokens, window, scale,
-                 dv, r1, r2, chunk, nv, keep_first, sink, v_row, sinks};
+                 dv, r1, r2, chunk, nv, keep_first, sink, v_row, sinks, softcap};
     cudaStream_t s = (cudaStream_t)stream;
     return QT_DISPATCH_DTYPE(dtype, "attention_prefill", {
         if (dv <= 64) return launch_prefill<T, 64>(p, max_q_len, s);
@@ -314,6 +317,10 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) attention_decode_kernel(const 
                 const float kv = to_float(krow[c]);
 #pragma unroll
                 for (int h = 0; h < DEC_HEADS; ++h) s[h] += qs[h * d + c] * kv;
+            }
+            if (p.softcap > 0.f) {
+#pragma unroll
+                for (int h = 0; h < DEC_HEADS; ++h) s[h] = p.softcap * tanhf(s[h] / p.softcap);
             }
             if (penalised) {
 #pragma unroll
@@ -447,7 +454,7 @@ extern "C" int qt_attention_decode(const void* q, const void* k_cache, const voi
                                    const int* block_table, int max_blocks, const int* seq_len, int n_seqs, int nq,
                                    int nkv, int d, int page_tokens, int ring_tokens, int window, float scale,
                                    int n_splits, float* part_acc, float* part_ml, int dv, const float* r1, const float* r2,
-                                   int chunk, int nv, int keep_first, int sink, int v_row, const float* sinks, void* stream) {
+                                   int chunk, int nv, int keep_first, int sink, int v_row, const float* sinks, float softcap, void* stream) {
     if (n_seqs == 0) return QT_OK;
     if (nv <= 0) nv = nkv;
     if (v_row <= 0) v_row = dv;
@@ -457,7 +464,7 @@ extern "C" int qt_attention_decode(const void* q, const void* k_cache, const voi
     QT_REQUIRE(n_splits == 1 || (part_acc && part_ml), "attention_decode: split results need scratch memory");
     QT_REQUIRE(n_seqs <= 65535, "attention_decode: too many sequences for one launch");
     DecodeParams dp{{q, k_cache, v_cache, out, block_table, max_blocks, nullptr, nullptr, n_seqs, nq, nkv, d, page_tokens, ring_tokens, window, scale,
-                     dv, r1, r2, chunk, nv, keep_first, sink, v_row, sinks},
+                     dv, r1, r2, chunk, nv, keep_first, sink, v_row, sinks, softcap},
                     seq_len, n_splits, part_acc, part_ml};
     cudaStream_t s = (cudaStream_t)stream;
     return QT_DISPATCH_DTYPE(dtype, "attention_decode", {

@@ -98,7 +98,8 @@ extern "C" int qt_attention_decode_ws(const void* q, const void* k_cache, const 
                                       const int* block_table, int max_blocks, const int* seq_len, int n_seqs, int nq,
                                       int nkv, int d, int page_tokens, int ring_tokens, int window, float scale,
                                       int n_splits, int warps, float* part_acc, float* part_ml, const float* r1, const float* r2,
-                                      int chunk, int nv, int keep_first, int sink, const float* sinks, void* stream) {
+                                      int chunk, int nv, int keep_first, int sink, const float* sinks, float softcap, int cap_small,
+                                      void* stream) {
     QT_REQUIRE(chunk >= 0 && nv >= 0 && (nv == 0 || nkv % nv == 0), "attention_decode_ws: chunk=%d, %d value heads for %d key heads", chunk, nv, nkv);
     if (n_seqs == 0) return QT_OK;
     int rc = check("attention_decode_ws", n_seqs, nq, nkv, d, page_tokens, ring_tokens, window);
@@ -108,6 +109,7 @@ extern "C" int qt_attention_decode_ws(const void* q, const void* k_cache, const 
                "attention_decode_ws: kept first keys (%d) go with no ring and no chunks", keep_first);
     QT_REQUIRE(n_splits >= 1 && n_splits <= 65535, "attention_decode_ws: n_splits=%d", n_splits);
     QT_REQUIRE(warps >= 1 && warps <= WS_MAX_WARPS, "attention_decode_ws: %d warps per block (1 to %d)", warps, WS_MAX_WARPS);
+    QT_REQUIRE(softcap >= 0.f && (softcap == 0.f || !r1), "attention_decode_ws: a score cap of %g goes with no distance penalty", (double)softcap);
     QT_REQUIRE(scale > 0.f, "attention_decode_ws: the score scale must be positive (the row maximum is taken before scaling)");
     // Up to eight blocks per (sequence, kv head) run as one cluster and merge through the first block's shared memory;
     // more than that (or QT_B200_DECODE_CLUSTER=0) go through scratch and the combine kernel.
@@ -121,26 +123,29 @@ extern "C" int qt_attention_decode_ws(const void* q, const void* k_cache, const 
     QT_REQUIRE(n_splits == 1 || cluster || (part_acc && part_ml), "attention_decode_ws: split results need scratch memory");
     MmaParams p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, (__nv_bfloat16*)out,
                 block_table, max_blocks, nullptr, nullptr, seq_len, n_seqs, nq, nkv, d, ring_tokens, window, scale,
-                n_splits, part_acc, part_ml, 2, cluster ? 1 : 0, r1, r2, chunk, nv, keep_first, sink, sinks};
+                n_splits, part_acc, part_ml, 2, cluster ? 1 : 0, r1, r2, chunk, nv, keep_first, sink, sinks, softcap};
     const size_t smem = rings + (cluster ? inboxes : 0);
     dim3 grid(n_splits, nkv * ((group + 15) / 16), n_seqs), block(32 * warps);
     cudaStream_t s = (cudaStream_t)stream;
-#define QT_LAUNCH_WS(DMAX, EXACT, PEN)                                                                                   \
+#define QT_LAUNCH_WS(DMAX, EXACT, PEN, CAP)                                                                              \
     do {                                                                                                                 \
         static bool ok = false;                                                                                          \
-        if (!ok) { rc = raise_smem(attention_decode_ws_kernel<DMAX, EXACT, PEN>, 227 * 1024, "attention_decode_ws"); if (rc) return rc; ok = true; } \
-        if (cluster) launch_kernel_cluster(attention_decode_ws_kernel<DMAX, EXACT, PEN>, grid, block, smem, s, (unsigned)n_splits, p); \
-        else launch_kernel(attention_decode_ws_kernel<DMAX, EXACT, PEN>, grid, block, smem, s, p);                        \
+        if (!ok) { rc = raise_smem(attention_decode_ws_kernel<DMAX, EXACT, PEN, CAP>, 227 * 1024, "attention_decode_ws"); if (rc) return rc; ok = true; } \
+        if (cluster) launch_kernel_cluster(attention_decode_ws_kernel<DMAX, EXACT, PEN, CAP>, grid, block, smem, s, (unsigned)n_splits, p); \
+        else launch_kernel(attention_decode_ws_kernel<DMAX, EXACT, PEN, CAP>, grid, block, smem, s, p);                        \
     } while (0)
-    if (r1) {
-        if (d == 128) QT_LAUNCH_WS(128, true, true);
-        else if (d == 64) QT_LAUNCH_WS(64, true, true);
-        else if (d < 64) QT_LAUNCH_WS(64, false, true);
-        else QT_LAUNCH_WS(128, false, true);
-    } else if (d == 128) QT_LAUNCH_WS(128, true, false);
-    else if (d == 64) QT_LAUNCH_WS(64, true, false);
-    else if (d < 64) QT_LAUNCH_WS(64, false, false);
-    else QT_LAUNCH_WS(128, false, false);
+#define QT_LAUNCH_WS_SIZE(PEN, CAP)                        \
+    do {                                                   \
+        if (d == 128) QT_LAUNCH_WS(128, true, PEN, CAP);   \
+        else if (d == 64) QT_LAUNCH_WS(64, true, PEN, CAP); \
+        else if (d < 64) QT_LAUNCH_WS(64, false, PEN, CAP); \
+        else QT_LAUNCH_WS(128, false, PEN, CAP);           \
+    } while (0)
+    if (r1) QT_LAUNCH_WS_SIZE(true, CAP_NONE);
+    else if (softcap > 0.f && cap_small) QT_LAUNCH_WS_SIZE(false, CAP_SMALL);
+    else if (softcap > 0.f) QT_LAUNCH_WS_SIZE(false, CAP_ANY);
+    else QT_LAUNCH_WS_SIZE(false, CAP_NONE);
+#undef QT_LAUNCH_WS_SIZE
 #undef QT_LAUNCH_WS
     QT_CHECK_LAUNCH("attention_decode_ws");
     if (n_splits > 1 && !cluster) {
@@ -154,7 +159,7 @@ extern "C" int qt_attention_prefill_mma(const void* q, const void* k_cache, cons
                                         const int* block_table, int max_blocks, const int* seq_start, const int* seq_past,
                                         int n_seqs, int max_q_len, int nq, int nkv, int d, int page_tokens, int ring_tokens,
                                         int window, float scale, const float* r1, const float* r2, int chunk, int nv, int keep_first,
-                                        int sink, const float* sinks, void* stream) {
+                                        int sink, const float* sinks, float softcap, int cap_small, void* stream) {
     QT_REQUIRE(chunk >= 0 && nv >= 0 && (nv == 0 || nkv % nv == 0), "attention_prefill_mma: chunk=%d, %d value heads for %d key heads", chunk, nv, nkv);
     if (n_seqs == 0 || max_q_len == 0) return QT_OK;
     int rc = check("attention_prefill_mma", n_seqs, nq, nkv, d, page_tokens, ring_tokens, window);
@@ -162,31 +167,32 @@ extern "C" int qt_attention_prefill_mma(const void* q, const void* k_cache, cons
     QT_REQUIRE(r1 != nullptr || r2 == nullptr, "attention_prefill_mma: the distance penalty needs its first factor");
     QT_REQUIRE(keep_first >= 0 && (keep_first == 0 || (ring_tokens == 0 && chunk == 0)),
                "attention_prefill_mma: kept first keys (%d) go with no ring and no chunks", keep_first);
-    QT_REQUIRE(r1 == nullptr || scale > 0.f, "attention_prefill_mma: with a distance penalty the score scale must be positive");
+    QT_REQUIRE((r1 == nullptr && softcap == 0.f) || scale > 0.f, "attention_prefill_mma: with a distance penalty or a score cap the score scale must be positive");
+    QT_REQUIRE(softcap >= 0.f && (softcap == 0.f || !r1), "attention_prefill_mma: a score cap of %g goes with no distance penalty", (double)softcap);
     MmaParams p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, (__nv_bfloat16*)out,
                 block_table, max_blocks, seq_start, seq_past, nullptr, n_seqs, nq, nkv, d, ring_tokens, window, scale,
-                1, nullptr, nullptr, 2, 0, r1, r2, chunk, nv, keep_first, sink, sinks};
+                1, nullptr, nullptr, 2, 0, r1, r2, chunk, nv, keep_first, sink, sinks, softcap};
     const int lds = d + PAD;
     const size_t smem = (size_t)4 * PAGE * lds * 2;
     dim3 grid((max_q_len + PF_BQ - 1) / PF_BQ, nq, n_seqs);
     cudaStream_t s = (cudaStream_t)stream;
-    if (r1 && d <= 64) {
-        static bool ok = false;
-        if (!ok) { rc = raise_smem(attention_prefill_mma_kernel<64, true>, 100 * 1024, "attention_prefill_mma"); if (rc) return rc; ok = true; }
-        launch_kernel(attention_prefill_mma_kernel<64, true>, dim3(grid), dim3(128), smem, s, p);
-    } else if (r1) {
-        static bool ok = false;
-        if (!ok) { rc = raise_smem(attention_prefill_mma_kernel<128, true>, 100 * 1024, "attention_prefill_mma"); if (rc) return rc; ok = true; }
-        launch_kernel(attention_prefill_mma_kernel<128, true>, dim3(grid), dim3(128), smem, s, p);
-    } else if (d <= 64) {
-        static bool ok = false;
-        if (!ok) { rc = raise_smem(attention_prefill_mma_kernel<64>, 100 * 1024, "attention_prefill_mma"); if (rc) return rc; ok = true; }
-        launch_kernel(attention_prefill_mma_kernel<64>, dim3(grid), dim3(128), smem, s, p);
-    } else {
-        static bool ok = false;
-        if (!ok) { rc = raise_smem(attention_prefill_mma_kernel<128>, 100 * 1024, "attention_prefill_mma"); if (rc) return rc; ok = true; }
-        launch_kernel(attention_prefill_mma_kernel<128>, dim3(grid), dim3(128), smem, s, p);
-    }
+#define QT_LAUNCH_PF(DMAX, PEN, CAP)                                                                                     \
+    do {                                                                                                                 \
+        static bool ok = false;                                                                                          \
+        if (!ok) { rc = raise_smem(attention_prefill_mma_kernel<DMAX, PEN, CAP>, 100 * 1024, "attention_prefill_mma"); if (rc) return rc; ok = true; } \
+        launch_kernel(attention_prefill_mma_kernel<DMAX, PEN, CAP>, dim3(grid), dim3(128), smem, s, p);                  \
+    } while (0)
+#define QT_LAUNCH_PF_SIZE(PEN, CAP)                  \
+    do {                                             \
+        if (d <= 64) QT_LAUNCH_PF(64, PEN, CAP);     \
+        else QT_LAUNCH_PF(128, PEN, CAP);            \
+    } while (0)
+    if (r1) QT_LAUNCH_PF_SIZE(true, CAP_NONE);
+    else if (softcap > 0.f && cap_small) QT_LAUNCH_PF_SIZE(false, CAP_SMALL);
+    else if (softcap > 0.f) QT_LAUNCH_PF_SIZE(false, CAP_ANY);
+    else QT_LAUNCH_PF_SIZE(false, CAP_NONE);
+#undef QT_LAUNCH_PF_SIZE
+#undef QT_LAUNCH_PF
     QT_CHECK_LAUNCH("attention_prefill_mma");
     return QT_OK;
 }

@@ -19,6 +19,7 @@
 #pragma once
 
 #include "common.cuh"
+#include "score_cap.cuh"
 
 #include <math.h>
 
@@ -61,6 +62,8 @@ struct MmaParams {
     int sink = 0;
     // sinks: the sink term's score per query head, taken as it is (not scaled); null: 0.
     const float* sinks = nullptr;
+    // softcap (kernels instantiated with a CAP): scores pass softcap tanh(s / softcap) first; the sink's does not.
+    float softcap = 0.f;
 };
 
 // The factor on a row's accumulator and its new denominator when the sink term joins a softmax whose running maximum
@@ -389,7 +392,7 @@ struct WarpTileCopy {
     }
 };
 
-template <int DMAX, bool EXACT, bool PEN = false>
+template <int DMAX, bool EXACT, bool PEN = false, int CAP = CAP_NONE>
 __global__ void __launch_bounds__(32 * WS_MAX_WARPS) attention_decode_ws_kernel(const MmaParams p) {
     pdl_launch_dependents();
     const bool merges_in_cluster = p.cluster_merge && gridDim.x > 1;
@@ -472,6 +475,7 @@ __global__ void __launch_bounds__(32 * WS_MAX_WARPS) attention_decode_ws_kernel(
     for (int i = 0; i < DMAX / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     const float scale2 = p.scale * LOG2E;                            // positive (checked by the host)
     float pen_c[2] = {0.f, 0.f}, pen_r2[2] = {0.f, 0.f};             // of this thread's two rows (query heads g and g + 8)
+    const ScoreCap cap = CAP != CAP_NONE ? ScoreCap::make<CAP>(p.softcap, p.scale) : ScoreCap{};
     const bool pen_linear = PEN && p.r2 == nullptr;
     if (PEN) {
 #pragma unroll
@@ -504,6 +508,12 @@ __global__ void __launch_bounds__(32 * WS_MAX_WARPS) attention_decode_ws_kernel(
                 mma_bf16(s[2], qf[ks], b1[0], b1[1]);
                 mma_bf16(s[3], qf[ks], b1[2], b1[3]);
             }
+        }
+        if (CAP != CAP_NONE) {
+#pragma unroll
+            for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[nt][e] = capped<CAP>(s[nt][e], cap);
         }
         if (PEN && pen_linear) {                                     // entries beyond the sequence are overwritten below
 #pragma unroll
@@ -698,7 +708,7 @@ __global__ void attention_combine_mma_kernel(const float* __restrict__ part_acc,
 // ----------------------------------------------------------------------------- prefill
 constexpr int PF_BQ = 64;
 
-template <int DMAX, bool PEN = false>
+template <int DMAX, bool PEN = false, int CAP = CAP_NONE>
 __global__ void __launch_bounds__(128, 3) attention_prefill_mma_kernel(const MmaParams p) {
     pdl_launch_dependents();
     pdl_wait();
@@ -759,6 +769,7 @@ __global__ void __launch_bounds__(128, 3) attention_prefill_mma_kernel(const Mma
 #pragma unroll
     for (int i = 0; i < DMAX / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     const float scale2 = p.scale * LOG2E;
+    const ScoreCap cap = CAP != CAP_NONE ? ScoreCap::make<CAP>(p.softcap, p.scale) : ScoreCap{};
     const bool pen_linear = PEN && p.r2 == nullptr;
     const float pen_c = PEN ? p.r1[head] / (pen_linear ? p.scale : scale2) : 0.f, pen_r2 = PEN && !pen_linear ? p.r2[head] : 0.f;
     // absolute positions of this thread's two query rows; rows beyond the sequence act as its last row
@@ -800,6 +811,12 @@ __global__ void __launch_bounds__(128, 3) attention_prefill_mma_kernel(const Mma
             // of the warp and need no mask.
             const bool all_visible = pos0 + PAGE - 1 <= warp_pos_min &&
                                      (p.window <= 0 || pos0 > warp_pos_max - p.window || pos0 + PAGE - 1 < keep_first) && pos0 >= warp_lo_max;
+            if (CAP != CAP_NONE) {
+#pragma unroll
+                for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) s[nt][e] = capped<CAP>(s[nt][e], cap);
+            }
             if (PEN && pen_linear) {                                 // keys ahead of a row's query are overwritten by the mask below
 #pragma unroll
                 for (int nt = 0; nt < 8; ++nt)

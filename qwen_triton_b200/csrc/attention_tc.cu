@@ -32,9 +32,14 @@
 // s - (r1 / (scale log2 e)) log2(1 + r2 (i - j)), one FMA for the argument (the key's place in the tile is a constant
 // of the unrolled loop), lg2.approx, one FMA; keys ahead of the query give arguments that the mask then overwrites.
 //
+// CAP: scores pass softcap tanh(s / softcap) before the maximum (score_cap.cuh), in the same place; no score of a masked key is
+// used.  `sinks` (or `sink` alone: 0): the softmax's denominator has one more term, exp of the head's number, which is neither
+// scaled nor capped and has no value; it joins a row's sum once, at the end.
+//
 // Counterpart in luozoupi/Qwen-Triton: kernels/flash_attention.py:54-152 (32 x 32 tl.dot tiles) and the masked
 // SDPA branch of modules/attention.py:110-123.
 #include "tc_common.cuh"
+#include "score_cap.cuh"
 
 #include <math.h>
 
@@ -63,6 +68,9 @@ struct TcAttnParams {
     int* status;
     const float* r1;               // [nq] factors of the distance penalty (PEN), else null
     const float* r2;
+    int sink;                      // 1: the softmax has one more term without a value, of score sinks[head] (null: 0)
+    const float* sinks;
+    float softcap;                 // of the score cap (CAP)
 };
 
 __device__ __forceinline__ float fast_log2(float x) {
@@ -143,7 +151,7 @@ __device__ __forceinline__ int cache_page(const int* table, int max_blocks, int 
 
 // BKEY: keys per tile, one page or two.  One page: half the shared memory and tensor memory, so that two blocks share
 // an SM and one's softmax runs under the other's MMAs.
-template <int HD, int BKEY, bool PEN>
+template <int HD, int BKEY, bool PEN, int CAP>
 __global__ void __launch_bounds__(THREADS, BKEY == 64 ? 2 : 1) attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                        const __grid_constant__ CUtensorMap map_k,
                                                                        const __grid_constant__ CUtensorMap map_v,
@@ -300,6 +308,7 @@ __global__ void __launch_bounds__(THREADS, BKEY == 64 ? 2 : 1) attention_prefill
         const int last_lo = p.chunk > 0 ? p_last / p.chunk * p.chunk : 0;
         const float scale2 = p.scale * LOG2E;
         const float pen_c = PEN ? -p.r1[head] / scale2 : 0.f, pen_r2 = PEN ? -p.r2[head] : 0.f;     // negated once, for the FMAs
+        const ScoreCap cap = CAP != CAP_NONE ? ScoreCap::make<CAP>(p.softcap, p.scale) : ScoreCap{};
         float m_run = -INFINITY, l_run = 0.f;              // the maximum this row scales by (scaled base-2 domain) and its sum
         pdl_wait();                                        // the output may still be read by an earlier kernel
         bool ok = true;
@@ -322,6 +331,22 @@ __global__ void __launch_bounds__(THREADS, BKEY == 64 ? 2 : 1) attention_prefill
 #pragma unroll
                     for (int c = 0; c < 32; ++c)
                         v[q][c] = __float_as_uint(fmaf(pen_c, fast_log2(fmaf(pen_r2, (float)(q * 32 + c), first)), __uint_as_float(v[q][c])));
+            }
+            if (CAP == CAP_SMALL) {
+                const uint64_t in2 = pair_f32(cap.in, cap.in);
+#pragma unroll
+                for (int q = 0; q < QUARTERS; ++q)
+#pragma unroll
+                    for (int c = 0; c < 32; c += 2) {
+                        float x0, x1;
+                        unpair_f32(capped_small2(pair_u32(v[q][c], v[q][c + 1]), in2), x0, x1);
+                        v[q][c] = __float_as_uint(x0); v[q][c + 1] = __float_as_uint(x1);
+                    }
+            } else if (CAP == CAP_ANY) {
+#pragma unroll
+                for (int q = 0; q < QUARTERS; ++q)
+#pragma unroll
+                    for (int c = 0; c < 32; ++c) v[q][c] = __float_as_uint(capped<CAP>(__uint_as_float(v[q][c]), cap));
             }
             // mask only where some row of the block cannot see the whole tile
             const bool masked = pos0 + BKEY - 1 > p_first || (p.window > 0 && pos0 <= p_last - p.window) || pos0 < last_lo;
@@ -395,7 +420,13 @@ __global__ void __launch_bounds__(THREADS, BKEY == 64 ? 2 : 1) attention_prefill
         }
         if (ok && mbar_wait(pv_full + 8 * ((n_tiles - 1) & 1), (uint32_t)((n_tiles - 1) >> 1) & 1u, status, 3)) {
             tc_fence_after();
-            const float inv = 1.f / l_run;
+            float factor = 1.f;
+            if (p.sink) {                                  // formed around the larger of the two, so that no exponential overflows
+                const float s2 = p.sinks ? p.sinks[head] * LOG2E : 0.f, top = fmaxf(m_run, s2);
+                factor = fast_exp2(m_run - top);
+                l_run = l_run * factor + fast_exp2(s2 - top);
+            }
+            const float inv = factor / l_run;
             __nv_bfloat16* dst = p.out + ((size_t)(q_begin + q0 + r) * p.nq + head) * HD;
 #pragma unroll 1
             for (int c0 = 0; c0 < HD; c0 += 32) {
@@ -426,7 +457,7 @@ __global__ void __launch_bounds__(THREADS, BKEY == 64 ? 2 : 1) attention_prefill
     }
 }
 
-template <int HD, int BKEY, bool PEN>
+template <int HD, int BKEY, bool PEN, int CAP>
 int launch(const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap& map_v, const TcAttnParams& p, int n_seqs,
            int max_q_len, cudaStream_t stream) {
     constexpr uint32_t HALVES = HD / 64;
@@ -434,12 +465,12 @@ int launch(const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap
     const size_t smem = (size_t)HALVES * HALF_BYTES + 4 * (size_t)HALVES * BKEY * 128 + ALIGN_SLACK + 128 + 64;
     static bool configured = false;
     if (!configured) {
-        cudaError_t err = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, BKEY, PEN>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        cudaError_t err = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, BKEY, PEN, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
         if (err != cudaSuccess) QT_FAIL(QT_ERR_LAUNCH, "attention_prefill_tc: cannot raise shared memory: %s", cudaGetErrorString(err));
         configured = true;
     }
     dim3 grid(p.nq, (max_q_len + BQ - 1) / BQ, n_seqs);
-    launch_kernel(attention_prefill_tc_kernel<HD, BKEY, PEN>, grid, dim3(THREADS), smem, stream, map_q, map_k, map_v, p);
+    launch_kernel(attention_prefill_tc_kernel<HD, BKEY, PEN, CAP>, grid, dim3(THREADS), smem, stream, map_q, map_k, map_v, p);
     QT_CHECK_LAUNCH("attention_prefill_tc");
     return QT_OK;
 }
@@ -452,7 +483,7 @@ extern "C" int qt_attention_prefill_tc(const void* q, const void* k_cache, const
                                        int n_pages, const int* block_table, int max_blocks, const int* seq_start,
                                        const int* seq_past, int n_seqs, int max_q_len, int nq, int nkv, int d,
                                        int page_tokens, int ring_tokens, int window, float scale, const float* r1, const float* r2,
-                                       int chunk, int nv,
+                                       int chunk, int nv, int sink, const float* sinks, float softcap, int cap_small,
                                        int* status, void* stream) {
     if (n_seqs == 0 || max_q_len == 0) return QT_OK;
     QT_REQUIRE(n_seqs > 0 && nq > 0 && nkv > 0 && nq % nkv == 0, "attention_prefill_tc: bad head counts nq=%d nkv=%d (B=%d)", nq, nkv, n_seqs);
@@ -464,6 +495,8 @@ extern "C" int qt_attention_prefill_tc(const void* q, const void* k_cache, const
     QT_REQUIRE(status != nullptr, "attention_prefill_tc: a status word is required");
     QT_REQUIRE((r1 == nullptr) == (r2 == nullptr) && (r1 == nullptr || scale > 0.f),
                "attention_prefill_tc: the distance penalty needs both of its factors and a positive score scale");
+    QT_REQUIRE(softcap >= 0.f && (softcap == 0.f || (!r1 && scale > 0.f)), "attention_prefill_tc: a score cap of %g goes with a positive scale and no distance penalty",
+               (double)softcap);
     QT_REQUIRE(((uintptr_t)q % 16 == 0) && ((uintptr_t)k_cache % 16 == 0) && ((uintptr_t)v_cache % 16 == 0) && ((uintptr_t)out % 16 == 0),
                "attention_prefill_tc: operands must be 16-byte aligned");
     CUtensorMap map_q, map_k, map_v;
@@ -475,15 +508,20 @@ extern "C" int qt_attention_prefill_tc(const void* q, const void* k_cache, const
     QT_REQUIRE(chunk >= 0 && nkv % nv == 0, "attention_prefill_tc: chunk=%d, %d value heads for %d key heads", chunk, nv, nkv);
     rc = tensor_map(&map_v, v_cache, (uint64_t)n_pages * nv * PAGE, (uint64_t)d, PAGE);
     if (rc) return rc;
-    TcAttnParams p{(__nv_bfloat16*)out, block_table, max_blocks, seq_start, seq_past, nq, nkv, ring_tokens, window, chunk, nv, scale, status, r1, r2};
+    TcAttnParams p{(__nv_bfloat16*)out, block_table, max_blocks, seq_start, seq_past, nq, nkv, ring_tokens, window, chunk, nv, scale, status, r1, r2,
+                   sink, sinks, softcap};
     cudaStream_t s = (cudaStream_t)stream;
     // key tiles of one page, two blocks per SM: measured 12-22 % faster than tiles of two pages with one block per SM
-    if (r1) {
-        if (d == 64) return launch<64, 64, true>(map_q, map_k, map_v, p, n_seqs, max_q_len, s);
-        return launch<128, 64, true>(map_q, map_k, map_v, p, n_seqs, max_q_len, s);
-    }
-    if (d == 64) return launch<64, 64, false>(map_q, map_k, map_v, p, n_seqs, max_q_len, s);
-    return launch<128, 64, false>(map_q, map_k, map_v, p, n_seqs, max_q_len, s);
+#define QT_LAUNCH_TC(PEN, CAP)                                                                      \
+    do {                                                                                            \
+        if (d == 64) return launch<64, 64, PEN, CAP>(map_q, map_k, map_v, p, n_seqs, max_q_len, s); \
+        return launch<128, 64, PEN, CAP>(map_q, map_k, map_v, p, n_seqs, max_q_len, s);             \
+    } while (0)
+    if (r1) QT_LAUNCH_TC(true, CAP_NONE);
+    if (softcap > 0.f && cap_small) QT_LAUNCH_TC(false, CAP_SMALL);
+    if (softcap > 0.f) QT_LAUNCH_TC(false, CAP_ANY);
+    QT_LAUNCH_TC(false, CAP_NONE);
+#undef QT_LAUNCH_TC
 }
 
 QT_DEFINE_LAST_ERROR(attention_tc)

@@ -146,7 +146,8 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(f
 #define QT_ACT_GELU_TANH 1
 #define QT_ACT_GELU 2
 #define QT_ACT_RELU 3
-#define QT_ACT_COUNT 4
+#define QT_ACT_RELU2 4      // the square of ReLU
+#define QT_ACT_COUNT 5
 
 // act(g) in float.  FAST takes the hardware approximations of exp and division for SiLU (2 ulp of float, for results
 // that are rounded to bfloat16 anyway); the other activations are the library's forms.
@@ -156,13 +157,14 @@ __device__ __forceinline__ float gate_activation(float g, int act) {
         case QT_ACT_GELU_TANH: return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
         case QT_ACT_GELU: return 0.5f * g * (1.f + erff(g * 0.7071067811865476f));
         case QT_ACT_RELU: return fmaxf(g, 0.f);
+        case QT_ACT_RELU2: { const float r = fmaxf(g, 0.f); return r * r; }
         default: return FAST ? __fdividef(g, 1.f + __expf(-g)) : g / (1.f + expf(-g));
     }
 }
 
 // A gate that also treats the up value, with a parameter: g' = min(g, limit), u' = clamp(u, -limit, limit),
 // y = g' sigmoid(1.702 g') (u' + 1).  Its code follows the activations above; the kernels that take `limit` accept it.
-#define QT_ACT_CAPPED 4
+#define QT_ACT_CAPPED 5
 
 // act(g) * u, or the capped gate.
 template <bool FAST>

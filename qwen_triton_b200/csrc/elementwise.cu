@@ -10,18 +10,22 @@
 using namespace qt;
 
 // ----------------------------------------------------------------------------- embedding
-// residual[t, :] = table[ids[t], :] widened to float, times `scale` (1 for a plain gather).  One block per token.
+// residual[t, c, :] = table[ids[t], :] widened to float, times `scale` (1 for a plain gather), for every c of `copies` (a residual
+// of several parallel streams starts with all of them alike; 1: the plain stream).  One block per token.
 template <typename T>
 __global__ void embedding_kernel(float* __restrict__ residual, const T* __restrict__ table,
-                                 const int* __restrict__ ids, int hidden, int vocab, float scale) {
+                                 const int* __restrict__ ids, int hidden, int vocab, float scale, int copies) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
     int id = ids[t];
     const bool valid = id >= 0 && id < vocab;   // ids are range-checked on the host; never read outside the table
     const T* row = table + (size_t)(valid ? id : 0) * hidden;
-    float* out = residual + (size_t)t * hidden;
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) out[i] = valid ? to_float(row[i]) * scale : 0.f;
+    float* out = residual + (size_t)t * copies * hidden;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        const float x = valid ? to_float(row[i]) * scale : 0.f;
+        for (int c = 0; c < copies; ++c) out[(size_t)c * hidden + i] = x;
+    }
 }
 
 // The same with an RMS norm behind the gather: residual[t, :] = x / sqrt(mean(x^2) + eps) * norm_w for the scaled row x.
@@ -59,7 +63,8 @@ __global__ void embedding_norm_kernel(float* __restrict__ residual, const T* __r
 }
 
 extern "C" int qt_embedding(float* residual, const void* table, const int* ids, int n_tokens, int hidden, int vocab,
-                            int table_dtype, float scale, const float* norm_w, float eps, void* start, void* stream) {
+                            int table_dtype, float scale, const float* norm_w, float eps, void* start, int copies, void* stream) {
+    QT_REQUIRE(copies >= 1 && (copies == 1 || (!norm_w && !start)), "embedding: %d copies of a row that is normed or kept", copies);
     QT_REQUIRE(n_tokens >= 0 && hidden > 0 && vocab > 0, "embedding: bad sizes T=%d H=%d V=%d", n_tokens, hidden, vocab);
     QT_REQUIRE(!norm_w || eps > 0.f, "embedding: eps must be positive");
     if (n_tokens == 0) return QT_OK;
@@ -70,7 +75,7 @@ extern "C" int qt_embedding(float* residual, const void* table, const int* ids, 
             QT_CHECK_LAUNCH("embedding_norm");
             return QT_OK;
         }
-        launch_kernel(embedding_kernel<T>, dim3(n_tokens), dim3(256), 0, (cudaStream_t)stream, residual, (const T*)table, ids, hidden, vocab, scale);
+        launch_kernel(embedding_kernel<T>, dim3(n_tokens), dim3(256), 0, (cudaStream_t)stream, residual, (const T*)table, ids, hidden, vocab, scale, copies);
         QT_CHECK_LAUNCH("embedding");
         return QT_OK;
     });

@@ -29,13 +29,14 @@ __device__ __forceinline__ float sum_splits(const float* __restrict__ base, size
 }
 
 struct PrepareParams {
-    const float* proj; int n_splits; size_t split_stride; int proj_cols;   // columns: query latent | key/value latent | rotated part | ...
+    const float* proj; int n_splits; size_t split_stride; int proj_cols;   // columns: query latent (or queries) | key/value latent | rotated part | ...
     const float* q_norm; const float* kv_norm; float eps;
     const float* cos_sin; int rotary_dim, max_pos;
     void* cq_out;                     // [T, q_rank]
     void* cache;                      // [pages, 1, page_tokens, rank + rot]
     const int* token_seq; const int* token_pos; const int* block_table; int max_blocks;
-    int q_rank, rank, rot, page_tokens, ring_tokens, write_kv;
+    int q_rank, rank, rot, page_tokens, ring_tokens, write_kv;      // q_rank 0: no query latent
+    int at_kv;                        // first column of the key/value latent
 };
 
 // one block per token
@@ -46,7 +47,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const PrepareParams
     __shared__ float scratch[32];
     const int t = blockIdx.x;
     const size_t base = (size_t)t * p.proj_cols;
-    {
+    if (p.q_rank > 0) {
         float sq = 0.f;
         for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) {
             const float x = sum_splits(p.proj, base + i, p.n_splits, p.split_stride);
@@ -61,7 +62,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const PrepareParams
     const int pos = p.token_pos[t];
     const int* table = p.block_table + (size_t)p.token_seq[t] * p.max_blocks;
     TO* row = (TO*)p.cache + cache_offset(table, pos, p.ring_tokens, p.page_tokens, 1, 0, p.rank + p.rot);
-    const size_t at = base + p.q_rank;
+    const size_t at = base + p.at_kv;
     float sq = 0.f;
     for (int i = threadIdx.x; i < p.rank; i += blockDim.x) {
         const float x = sum_splits(p.proj, at + i, p.n_splits, p.split_stride);
@@ -88,17 +89,18 @@ extern "C" int qt_latent_prepare(const float* proj, int n_splits, long long spli
                                  const float* kv_norm, float eps, const float* cos_sin, int rotary_dim, int max_pos, void* cq_out,
                                  void* cache, int out_dtype, const int* token_seq, const int* token_pos, const int* block_table,
                                  int max_blocks, int n_tokens, int q_rank, int rank, int rot, int page_tokens, int ring_tokens,
-                                 int write_kv, void* stream) {
-    QT_REQUIRE(n_tokens >= 0 && q_rank > 0 && rank > 0 && rot >= 0 && n_splits >= 1 && eps > 0.f, "latent_prepare: bad sizes");
-    QT_REQUIRE(q_rank + (write_kv ? rank + rot : 0) <= proj_cols, "latent_prepare: the latents need %d columns of %d",
-               q_rank + (write_kv ? rank + rot : 0), proj_cols);
+                                 int write_kv, int at_kv, void* stream) {
+    QT_REQUIRE(n_tokens >= 0 && q_rank >= 0 && at_kv >= q_rank && rank > 0 && rot >= 0 && n_splits >= 1 && eps > 0.f, "latent_prepare: bad sizes");
+    QT_REQUIRE(at_kv + (write_kv ? rank + rot : 0) <= proj_cols, "latent_prepare: the latents need %d columns of %d",
+               at_kv + (write_kv ? rank + rot : 0), proj_cols);
+    QT_REQUIRE(q_rank == 0 || (q_norm && cq_out), "latent_prepare: a query latent needs its weight and a place");
     QT_REQUIRE(rotary_dim >= 0 && rotary_dim % 2 == 0 && rotary_dim <= rot && (rotary_dim == 0 || cos_sin),
                "latent_prepare: %d of %d elements rotate", rotary_dim, rot);
     QT_REQUIRE(!write_kv || (cache && block_table && kv_norm), "latent_prepare: no cache to write to");
     if (n_tokens == 0) return QT_OK;
     cudaStream_t s = (cudaStream_t)stream;
     PrepareParams p{proj, n_splits, (size_t)split_stride, proj_cols, q_norm, kv_norm, eps, rotary_dim ? cos_sin : nullptr, rotary_dim, max_pos,
-                    cq_out, cache, token_seq, token_pos, block_table, max_blocks, q_rank, rank, rot, page_tokens, ring_tokens, write_kv};
+                    cq_out, cache, token_seq, token_pos, block_table, max_blocks, q_rank, rank, rot, page_tokens, ring_tokens, write_kv, at_kv};
     return QT_DISPATCH_DTYPE(out_dtype, "latent_prepare", {
         launch_kernel(latent_prepare_kernel<T>, dim3(n_tokens), dim3(256), 0, s, p);
         QT_CHECK_LAUNCH("latent_prepare");
@@ -107,11 +109,11 @@ extern "C" int qt_latent_prepare(const float* proj, int n_splits, long long spli
 }
 
 // ----------------------------------------------------------------------------- the rotated part of the queries
-// q [splits, T, heads * (dim + rot)] -> out[t, h, out_offset + i] for i < rot.  One thread per (token, head, element).
+// q [splits, T, q_cols >= heads * (dim + rot)] -> out[t, h, out_offset + i] for i < rot.  One thread per (token, head, element).
 template <typename TI, typename TO>
 __global__ void latent_query_rot_kernel(const TI* __restrict__ q, int n_splits, size_t split_stride, const float* __restrict__ cos_sin,
                                         int rotary_dim, const int* __restrict__ token_pos, TO* __restrict__ out, long long total,
-                                        int heads, int dim, int rot, int out_row, int out_offset) {
+                                        int heads, int dim, int rot, int q_cols, int out_row, int out_offset) {
     pdl_launch_dependents();
     pdl_wait();
     const int half = rotary_dim / 2;
@@ -120,7 +122,7 @@ __global__ void latent_query_rot_kernel(const TI* __restrict__ q, int n_splits, 
         const long long th = idx / rot;
         const int h = (int)(th % heads);
         const long long t = th / heads;
-        const size_t at = ((size_t)t * heads + h) * (dim + rot) + dim;
+        const size_t at = (size_t)t * q_cols + (size_t)h * (dim + rot) + dim;
         const float x = load_sum(q, at + i, n_splits, split_stride);
         float y = x;
         if (i < rotary_dim) {
@@ -134,8 +136,9 @@ __global__ void latent_query_rot_kernel(const TI* __restrict__ q, int n_splits, 
 }
 
 extern "C" int qt_latent_query_rot(const void* q, int in_dtype, int n_splits, long long split_stride, const float* cos_sin, int rotary_dim,
-                                   const int* token_pos, void* out, int out_dtype, int n_tokens, int heads, int dim, int rot, int out_row,
-                                   int out_offset, void* stream) {
+                                   const int* token_pos, void* out, int out_dtype, int n_tokens, int heads, int dim, int rot, int q_cols,
+                                   int out_row, int out_offset, void* stream) {
+    QT_REQUIRE(q_cols >= heads * (dim + rot), "latent_query_rot: %d heads of %d + %d in %d columns", heads, dim, rot, q_cols);
     QT_REQUIRE(n_tokens >= 0 && heads > 0 && dim >= 0 && rot >= 0 && out_offset >= 0 && out_offset + rot <= out_row, "latent_query_rot: bad sizes");
     QT_REQUIRE(rotary_dim >= 0 && rotary_dim % 2 == 0 && rotary_dim <= rot && (rotary_dim == 0 || cos_sin), "latent_query_rot: %d of %d elements rotate",
                rotary_dim, rot);
@@ -146,7 +149,7 @@ extern "C" int qt_latent_query_rot(const void* q, int in_dtype, int n_splits, lo
     if (blocks > (long long)sm_count() * 16) blocks = (long long)sm_count() * 16;
 #define QT_LAUNCH_ROT(TI, TO)                                                                                                      \
     launch_kernel(latent_query_rot_kernel<TI, TO>, dim3((unsigned)blocks), dim3(256), 0, s, (const TI*)q, n_splits, (size_t)split_stride, \
-                  cos_sin, rotary_dim, token_pos, (TO*)out, total, heads, dim, rot, out_row, out_offset)
+                  cos_sin, rotary_dim, token_pos, (TO*)out, total, heads, dim, rot, q_cols, out_row, out_offset)
     if (in_dtype == QT_F32 && out_dtype == QT_F32) QT_LAUNCH_ROT(float, float);
     else if (in_dtype == QT_F32 && out_dtype == QT_BF16) QT_LAUNCH_ROT(float, __nv_bfloat16);
     else if (in_dtype == QT_BF16 && out_dtype == QT_BF16) QT_LAUNCH_ROT(__nv_bfloat16, __nv_bfloat16);

@@ -76,6 +76,85 @@ extern "C" int qt_linear_attention_prepare(const float* proj, int n_splits, long
     return QT_OK;
 }
 
+// The same sums for rows whose first `heads` runs of `dim` columns (q heads, then k heads) are rotated by the token's position: in
+// each, element i < rd / 2 turns together with element i + rd / 2 by the angle whose cos and sin the table row of the position
+// holds (cos | sin, rd columns); the other columns pass.  A thread takes V neighbouring pairs, or V neighbouring columns that
+// do not turn; grid (blocks of a row's items, tokens).
+template <int V> struct RotPack { float v[V]; };
+template <int V> __device__ __forceinline__ RotPack<V> rot_sum(const float* p, int n_splits, size_t stride) {
+    RotPack<V> r;
+    if constexpr (V == 4) {
+        float4 x = __ldg(reinterpret_cast<const float4*>(p));
+        for (int s = 1; s < n_splits; ++s) {
+            const float4 y = __ldg(reinterpret_cast<const float4*>(p + (size_t)s * stride));
+            x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
+        }
+        r.v[0] = x.x; r.v[1] = x.y; r.v[2] = x.z; r.v[3] = x.w;
+    } else {
+        r.v[0] = __ldg(p);
+        for (int s = 1; s < n_splits; ++s) r.v[0] += __ldg(p + (size_t)s * stride);
+    }
+    return r;
+}
+template <int V> __device__ __forceinline__ void rot_put(float* p, const RotPack<V>& r) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+    else *p = r.v[0];
+}
+
+template <int V>
+__global__ void __launch_bounds__(256) linear_attention_rotate_kernel(const float* __restrict__ proj, int n_splits, size_t split_stride, int proj_cols, int cols,
+                                                                      float* __restrict__ out, int heads, int dim, int rd, const float* __restrict__ cos_sin,
+                                                                      int max_pos, const int* __restrict__ token_pos) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int item = blockIdx.x * 256 + threadIdx.x, half = rd / 2;
+    const int turning = half / V, still = (dim - rd) / V, per_head = turning + still, rotated = heads * per_head;
+    if (item >= rotated + (cols - heads * dim) / V) return;
+    const size_t t = blockIdx.y;
+    const float* row = proj + t * proj_cols;
+    float* dst = out + t * cols;
+    const int head = item / max(per_head, 1), within = item - head * per_head;
+    if (item < rotated && within < turning) {
+        const int at = head * dim + within * V;
+        const int pos = min(token_pos[t], max_pos - 1);
+        const float* table = cos_sin + (size_t)pos * rd + within * V;
+        const RotPack<V> c = rot_sum<V>(table, 1, 0), s = rot_sum<V>(table + half, 1, 0);
+        const RotPack<V> u = rot_sum<V>(row + at, n_splits, split_stride), w = rot_sum<V>(row + at + half, n_splits, split_stride);
+        RotPack<V> a, b;
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+            a.v[i] = u.v[i] * c.v[i] - w.v[i] * s.v[i];
+            b.v[i] = w.v[i] * c.v[i] + u.v[i] * s.v[i];
+        }
+        rot_put<V>(dst + at, a);
+        rot_put<V>(dst + at + half, b);
+    } else {
+        const int at = item < rotated ? head * dim + rd + (within - turning) * V : heads * dim + (item - rotated) * V;
+        rot_put<V>(dst + at, rot_sum<V>(row + at, n_splits, split_stride));
+    }
+}
+
+extern "C" int qt_linear_attention_rotate(const float* proj, int n_splits, long long split_stride, int proj_cols, int cols, float* out, int n_tokens, int heads,
+                                          int dim, int rotary_dim, const float* cos_sin, int max_pos, const int* token_pos, void* stream) {
+    QT_REQUIRE(n_tokens >= 0 && cols > 0 && cols <= proj_cols && n_splits >= 1 && heads > 0 && dim > 0 && (long long)heads * dim <= cols,
+               "linear_attention_rotate: %d heads of %d in %d of %d columns", heads, dim, cols, proj_cols);
+    QT_REQUIRE(rotary_dim > 0 && rotary_dim % 2 == 0 && rotary_dim <= dim && cos_sin && max_pos > 0 && token_pos, "linear_attention_rotate: %d of %d elements turn", rotary_dim, dim);
+    if (n_tokens == 0) return QT_OK;
+    QT_REQUIRE(n_tokens <= 65535, "linear_attention_rotate: %d tokens are too many for one launch", n_tokens);
+    const bool wide = rotary_dim % 8 == 0 && dim % 4 == 0 && cols % 4 == 0 && proj_cols % 4 == 0 && split_stride % 4 == 0 && (uintptr_t)proj % 16 == 0 &&
+                      (uintptr_t)out % 16 == 0 && (uintptr_t)cos_sin % 16 == 0;
+    const int v = wide ? 4 : 1;
+    const int items = heads * (dim - rotary_dim / 2) / v + (cols - heads * dim) / v;
+    const dim3 grid((items + 255) / 256, n_tokens);
+    cudaStream_t s = (cudaStream_t)stream;
+    if (wide) launch_kernel(linear_attention_rotate_kernel<4>, grid, dim3(256), 0, s, proj, n_splits, (size_t)split_stride, proj_cols, cols, out, heads, dim, rotary_dim,
+                            cos_sin, max_pos, token_pos);
+    else launch_kernel(linear_attention_rotate_kernel<1>, grid, dim3(256), 0, s, proj, n_splits, (size_t)split_stride, proj_cols, cols, out, heads, dim, rotary_dim,
+                       cos_sin, max_pos, token_pos);
+    QT_CHECK_LAUNCH("linear_attention_rotate");
+    return QT_OK;
+}
+
 // COLS columns of a head's state per block (COLS * 8 threads).  A chunk's q, k and v are fetched into registers while the
 // chunk before is worked on (every load of a chunk is issued before the first is used), pass SiLU where asked and go to
 // shared memory behind a barrier.

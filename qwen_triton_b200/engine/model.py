@@ -39,7 +39,7 @@ class CausalLM:
         self.entries = [part_class("stream_map", entry)(entry.params, runtime) for entry in spec.entries]
         self.final_norm = part_class("norm", spec.final_norm)(spec.final_norm.params, spec.final_norm["name"], runtime)
         self.head = part_class("head", spec.head)(spec.head.params, spec.vocab_size, spec.hidden_size, runtime)
-        runtime.workspace.declare("residual", runtime.max_step_tokens * spec.hidden_size, torch.float32)
+        runtime.workspace.declare("residual", runtime.max_step_tokens * (spec.streams or 1) * spec.hidden_size, torch.float32)
         if self.entries:
             runtime.workspace.declare("stream_start", runtime.max_step_tokens * spec.hidden_size, runtime.dtype)
 
@@ -86,7 +86,8 @@ class CausalLM:
         """Run the tokens of ``ctx`` through every scheduled layer; write the logits of ``ctx.want_rows``."""
         hidden = self.spec.hidden_size
         ws = self.runtime.workspace
-        stream = ResidualStream(ws.view("residual", ctx.n_tokens, hidden), ws.view("stream_start", ctx.n_tokens, hidden) if self.entries else None)
+        shape = (ctx.n_tokens, hidden) if self.spec.streams is None else (ctx.n_tokens, self.spec.streams, hidden)
+        stream = ResidualStream(ws.view("residual", *shape), ws.view("stream_start", ctx.n_tokens, hidden) if self.entries else None)
         if stream.start is not None:
             self.embedding.forward(ctx.token_ids, stream.residual, stream.start)
         else:

@@ -22,7 +22,7 @@ _c_int, _c_ll, _c_float, _c_ptr = ctypes.c_int, ctypes.c_longlong, ctypes.c_floa
 
 _SIGNATURES = {
     "elementwise": {
-        "qt_embedding": [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_float, _c_ptr, _c_ptr],
+        "qt_embedding": [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_float, _c_ptr, _c_int, _c_ptr],
         "qt_stream_concat": [_c_ptr, _c_ptr, _c_int, _c_int, _c_ll, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr],
         "qt_add_bias": [_c_ptr, _c_ptr, _c_int, _c_int, _c_ptr],
         "qt_add_rmsnorm": [_c_ptr, _c_ptr, _c_int, _c_int, _c_ll, _c_ptr, _c_float, _c_ptr, _c_int, _c_ptr, _c_int,
@@ -38,6 +38,10 @@ _SIGNATURES = {
                        _c_int, _c_ptr],
         "qt_map_difference": [_c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_ptr],
     },
+    "streams": {
+        # streams, delta, n_splits, split_stride, mix, out_weight, read, weight, eps, out, out_dtype, rows, n_rows, hidden, streams_count, stream
+        "qt_streams_norm": [_c_ptr, _c_ptr, _c_int, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr],
+    },
     "delta_rule": {
         "qt_delta_prepare": [_c_ptr, _c_int, _c_ll, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
                              _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr],
@@ -51,6 +55,8 @@ _SIGNATURES = {
         "qt_linear_attention_scan": [_c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int,
                                      _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
         "qt_linear_attention_prepare": [_c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr],
+        # proj, n_splits, split_stride, proj_cols, cols, out, n_tokens, heads, dim, rotary_dim, cos_sin, max_pos, token_pos, stream
+        "qt_linear_attention_rotate": [_c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr],
         "qt_decayed_attention_steps": [_c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_float, _c_ptr, _c_ptr, _c_ptr,
                                        _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
         # o, x, x_cols, at_x, skip, skips, proj, n_splits, split_stride, proj_cols, at_gate, weight, weight_len, eps, scale, groups, silu,
@@ -67,10 +73,10 @@ _SIGNATURES = {
     "attention": {
         "qt_attention_prefill": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int,
                                  _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_int,
-                                 _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
+                                 _c_int, _c_int, _c_int, _c_ptr, _c_float, _c_ptr],
         "qt_attention_decode": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int,
                                 _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int,
-                                _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
+                                _c_int, _c_int, _c_int, _c_ptr, _c_float, _c_ptr],
     },
     "layernorm": {
         "qt_add_layernorm": [_c_ptr, _c_ptr, _c_int, _c_int, _c_ll, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_ptr],
@@ -86,9 +92,9 @@ _SIGNATURES = {
     },
     "latent": {
         "qt_latent_prepare": [_c_ptr, _c_int, _c_ll, _c_int, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr,
-                              _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
+                              _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
         "qt_latent_query_rot": [_c_ptr, _c_int, _c_int, _c_ll, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                                _c_int, _c_ptr],
+                                _c_int, _c_int, _c_ptr],
         "qt_head_product": [_c_ptr, _c_int, _c_int, _c_ll, _c_ll, _c_ll, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_ll, _c_ll, _c_int,
                             _c_ptr, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr],
     },
@@ -115,13 +121,13 @@ _SIGNATURES = {
                                     _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_ptr],
         "qt_attention_decode_ws": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int,
                                    _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
-                                   _c_int, _c_int, _c_ptr, _c_ptr],
+                                   _c_int, _c_int, _c_ptr, _c_float, _c_int, _c_ptr],
         "qt_attention_prefill_mma": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int,
-                                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
+                                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_float, _c_int, _c_ptr],
     },
     "attention_tc": {
         "qt_attention_prefill_tc": [_c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int,
-                                    _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr],
+                                    _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_float, _c_int, _c_ptr, _c_ptr],
     },
     "gemm_simt": {
         "qt_gemm_simt": [_c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr],
@@ -260,8 +266,9 @@ class GemmOut:
 def embedding(residual: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, scale: float = 1.0, norm_weight: torch.Tensor | None = None,
               eps: float = 0.0, start: torch.Tensor | None = None) -> None:
     """residual[t] = table[ids[t]] * scale in float, RMS-normed with ``norm_weight`` [H] where given.  ids: int32 [T].
-    ``start`` [T, H] (the table's type) receives a copy of the result."""
-    tokens, hidden = residual.shape
+    ``start`` [T, H] (the table's type) receives a copy of the result.  A residual of several streams [T, S, H] gets the row S
+    times (then without norm and ``start``)."""
+    tokens, hidden, copies = residual.shape[0], residual.shape[-1], residual.shape[1] if residual.dim() == 3 else 1
     _need(residual, "residual", torch.float32)
     _need(table, "table")
     _need(ids, "ids", torch.int32, (tokens,))
@@ -272,7 +279,7 @@ def embedding(residual: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, sc
     if start is not None:
         _need(start, "start", table.dtype, (tokens, hidden))
     _call("elementwise", "qt_embedding", _ptr(residual), _ptr(table), _ptr(ids), tokens, hidden, table.shape[0],
-          _code(table, "table"), float(scale), _ptr(norm_weight), float(eps), _ptr(start), _stream())
+          _code(table, "table"), float(scale), _ptr(norm_weight), float(eps), _ptr(start), copies, _stream())
 
 
 def stream_concat(residual: torch.Tensor, delta: GemmOut | None, start: torch.Tensor, out: torch.Tensor) -> None:
@@ -362,6 +369,29 @@ def qkv_treat_write(qkv: GemmOut, bias: torch.Tensor | None, q_out: torch.Tensor
           _ptr(block_table), max_blocks, 0 if v_norm_eps is None else 1, float(v_norm_eps or 0.0), _ptr(blend_from),
           _ptr(blend_weight), _ptr(keep_to), tokens, num_heads, num_kv_heads, head_dim, v_head_dim, page_tokens, ring_tokens,
           1 if write_kv else 0, _stream())
+
+
+def streams_norm(streams: torch.Tensor, delta: GemmOut | None, mix: torch.Tensor | None, out_weight: torch.Tensor | None,
+                 read: torch.Tensor | None, weight: torch.Tensor, eps: float, out: torch.Tensor, rows: torch.Tensor | None = None) -> None:
+    """A residual of S parallel streams [T, S, H] (float) between two sublayers: with ``delta`` (what the sublayer before returned,
+    float sums) the streams become x_t = sum_s mix[s, t] x_s + out_weight[t] delta; ``out`` = rmsnorm(sum_s read[s] x_s) * weight.
+    ``read`` None: the plain sum.  With ``rows`` (int32 [K]) only those rows are formed and the streams stay as they are."""
+    tokens, count, hidden = streams.shape
+    _need(streams, "streams", torch.float32)
+    _need(weight, "weight", torch.float32, (hidden,))
+    _need(out, "out", shape=(tokens if rows is None else rows.shape[0], hidden))
+    if read is not None:
+        _need(read, "read", torch.float32, (count,))
+    if rows is not None:
+        _need(rows, "rows", torch.int32)
+    if delta is not None:
+        _need(mix, "mix", torch.float32, (count, count))
+        _need(out_weight, "out_weight", torch.float32, (count,))
+        if not delta.tensor.is_cuda or delta.tensor.dtype != torch.float32 or (delta.rows, delta.cols) != (tokens, hidden):
+            raise KernelError(f"streams_norm: delta {tuple(delta.tensor.shape)} {delta.tensor.dtype} does not match streams {tuple(streams.shape)} of float sums")
+    _call("streams", "qt_streams_norm", _ptr(streams), _ptr(delta.tensor) if delta else None, delta.n_splits if delta else 1,
+          delta.split_stride if delta else 0, _ptr(mix), _ptr(out_weight), _ptr(read), _ptr(weight), float(eps), _ptr(out), _code(out, "out"),
+          _ptr(rows), out.shape[0], hidden, count, _stream())
 
 
 def qk_norm_rope_write(qkv: GemmOut, q_out: torch.Tensor, k_cache: torch.Tensor | None, v_cache: torch.Tensor | None,
@@ -567,18 +597,24 @@ def gate_mul(x: torch.Tensor, gate: GemmOut, offset: int, group: int = 1) -> Non
           x.shape[0], x.shape[1], int(group), _stream())
 
 
-def latent_prepare(proj: GemmOut, q_norm: torch.Tensor, kv_norm: torch.Tensor | None, eps: float, cos_sin: torch.Tensor | None,
-                   cq_out: torch.Tensor, cache: torch.Tensor | None, token_seq: torch.Tensor, token_pos: torch.Tensor,
-                   block_table: torch.Tensor | None, rank: int, rot: int, page_tokens: int, ring_tokens: int, write_kv: bool = True) -> None:
+def latent_prepare(proj: GemmOut, q_norm: torch.Tensor | None, kv_norm: torch.Tensor | None, eps: float, cos_sin: torch.Tensor | None,
+                   cq_out: torch.Tensor | None, cache: torch.Tensor | None, token_seq: torch.Tensor, token_pos: torch.Tensor,
+                   block_table: torch.Tensor | None, rank: int, rot: int, page_tokens: int, ring_tokens: int, write_kv: bool = True,
+                   at_kv: int | None = None) -> None:
     """From the float sums ``proj`` [*, T, >= q_rank (+ rank + rot)] of a latent-attention mixer's first projection: the
     query latent's RMS norm (``q_norm`` [q_rank]) into ``cq_out`` [T, q_rank] and, with ``write_kv``, the cache row of every
     token: the key/value latent's RMS norm (``kv_norm`` [rank]) followed by the shared key part of ``rot`` elements, of
-    which the first ``cos_sin.shape[1]`` are rotated by the token's position.  ``cache`` is [pages, 1, page_tokens, rank + rot]."""
+    which the first ``cos_sin.shape[1]`` are rotated by the token's position.  ``cache`` is [pages, 1, page_tokens, rank + rot].
+    Without ``q_norm`` and ``cq_out`` there is no query latent; ``at_kv`` is the key/value latent's first column (default: q_rank)."""
     tokens = proj.rows
-    q_rank = q_norm.shape[0]
+    q_rank = q_norm.shape[0] if q_norm is not None else 0
     _need(proj.tensor, "proj", torch.float32)
-    _need(q_norm, "q_norm", torch.float32)
-    _need(cq_out, "cq_out", shape=(tokens, q_rank))
+    if q_norm is not None:
+        _need(q_norm, "q_norm", torch.float32)
+        _need(cq_out, "cq_out", shape=(tokens, q_rank))
+    elif not write_kv:
+        raise KernelError("latent_prepare: neither a query latent nor a cache row is wanted")
+    like = cq_out if cq_out is not None else cache
     _need(token_seq, "token_seq", torch.int32, (tokens,))
     _need(token_pos, "token_pos", torch.int32, (tokens,))
     rotary_dim, max_pos, max_blocks = 0, 0, 0
@@ -589,21 +625,21 @@ def latent_prepare(proj: GemmOut, q_norm: torch.Tensor, kv_norm: torch.Tensor | 
         _need(kv_norm, "kv_norm", torch.float32, (rank,))
         _need(block_table, "block_table", torch.int32)
         max_blocks = block_table.shape[1]
-        _need(cache, "cache", cq_out.dtype)
+        _need(cache, "cache", like.dtype)
         if tuple(cache.shape[1:]) != (1, page_tokens, rank + rot):
             raise KernelError(f"cache: shape {tuple(cache.shape)} is not [pages, 1, {page_tokens}, {rank + rot}]")
     _call("latent", "qt_latent_prepare", _ptr(proj.tensor), proj.n_splits, proj.split_stride, proj.cols, _ptr(q_norm), _ptr(kv_norm),
-          float(eps), _ptr(cos_sin), rotary_dim, max_pos, _ptr(cq_out), _ptr(cache), _code(cq_out, "cq_out"), _ptr(token_seq),
+          float(eps), _ptr(cos_sin), rotary_dim, max_pos, _ptr(cq_out), _ptr(cache), _code(like, "cq_out"), _ptr(token_seq),
           _ptr(token_pos), _ptr(block_table), max_blocks, tokens, q_rank, int(rank), int(rot), page_tokens, ring_tokens,
-          1 if write_kv else 0, _stream())
+          1 if write_kv else 0, q_rank if at_kv is None else int(at_kv), _stream())
 
 
 def latent_query_rot(q: GemmOut, cos_sin: torch.Tensor | None, token_pos: torch.Tensor, out: torch.Tensor, heads: int, dim: int, rot: int,
                      out_offset: int) -> None:
-    """The last ``rot`` elements of every head of ``q`` [*, T, heads (dim + rot)], the first ``cos_sin.shape[1]`` of them
+    """The last ``rot`` elements of every head of ``q`` [*, T, heads (dim + rot)] (further columns behind are left alone), the first ``cos_sin.shape[1]`` of them
     rotated by the token's position, into ``out`` [T, heads, row] at ``out_offset`` of every head's row."""
     tokens = q.rows
-    if q.cols != heads * (dim + rot) or out.dim() != 3 or tuple(out.shape[:2]) != (tokens, heads):
+    if q.cols < heads * (dim + rot) or out.dim() != 3 or tuple(out.shape[:2]) != (tokens, heads):
         raise KernelError(f"latent_query_rot: q {tuple(q.tensor.shape)}, out {tuple(out.shape)} for {heads} heads of {dim} + {rot}")
     _need(out, "out")
     _need(token_pos, "token_pos", torch.int32, (tokens,))
@@ -612,7 +648,7 @@ def latent_query_rot(q: GemmOut, cos_sin: torch.Tensor | None, token_pos: torch.
         _need(cos_sin, "cos_sin", torch.float32)
         rotary_dim = cos_sin.shape[1]
     _call("latent", "qt_latent_query_rot", _ptr(q.tensor), _code(q.tensor, "q"), q.n_splits, q.split_stride, _ptr(cos_sin), rotary_dim,
-          _ptr(token_pos), _ptr(out), _code(out, "out"), tokens, heads, dim, rot, out.shape[2], int(out_offset), _stream())
+          _ptr(token_pos), _ptr(out), _code(out, "out"), tokens, heads, dim, rot, q.cols, out.shape[2], int(out_offset), _stream())
 
 
 def head_product(x, weight: torch.Tensor, out: torch.Tensor, *, x_row: int, x_head: int, x_offset: int = 0, out_offset: int = 0,
@@ -775,6 +811,18 @@ def linear_attention_prepare(proj: GemmOut, cols: int, out: torch.Tensor, act: b
     return GemmOut(out.view(1, proj.rows, int(cols)))
 
 
+def linear_attention_rotate(proj: GemmOut, cols: int, out: torch.Tensor, heads: int, dim: int, cos_sin: torch.Tensor, token_pos: torch.Tensor) -> GemmOut:
+    """out [T, cols] (float) = the first ``cols`` columns of ``proj`` (float sums [*, T, all]), of which the first ``heads`` runs of ``dim``
+    (q heads, then k heads) are rotated by the token's position: the first ``cos_sin.shape[1]`` elements of each, in pairs (i, i + half)."""
+    _need(proj.tensor, "proj", torch.float32)
+    _need(out, "out", torch.float32, (proj.rows, int(cols)))
+    _need(cos_sin, "cos_sin", torch.float32)
+    _need(token_pos, "token_pos", torch.int32, (proj.rows,))
+    _call("linear_attention", "qt_linear_attention_rotate", _ptr(proj.tensor), proj.n_splits, proj.split_stride, proj.cols, int(cols), _ptr(out), proj.rows,
+          int(heads), int(dim), cos_sin.shape[1], _ptr(cos_sin), cos_sin.shape[0], _ptr(token_pos), _stream())
+    return GemmOut(out.view(1, proj.rows, int(cols)))
+
+
 DECAY_CHUNK = 64            # tokens per chunk of the chunked recurrence
 _DECAY_FEW_TOKENS = 16      # steps in which no sequence brings more run token by token
 
@@ -862,11 +910,11 @@ def group_gate_norm(o: torch.Tensor, weight: torch.Tensor, eps: float, out: torc
 
 SWIGLU_GROUP = 16      # rows of gate and of up that alternate in a weight laid out for the GEMM's gated epilogue
 # gate activations of a gated feed-forward, act(gate) * up: names a configuration may use -> the kernels' codes
-ACTIVATIONS = {"silu": 0, "swish": 0, "gelu_pytorch_tanh": 1, "gelu_tanh": 1, "gelu": 2, "relu": 3}
+ACTIVATIONS = {"silu": 0, "swish": 0, "gelu_pytorch_tanh": 1, "gelu_tanh": 1, "gelu": 2, "relu": 3, "relu2": 4}
 # a gate that also treats the up value and has a parameter ``limit``: g' = min(g, limit), u' = clamp(u, -limit, limit),
 # y = g' sigmoid(1.702 g') (u' + 1).  Taken, with ``limit``, by ``swiglu``, the experts' kernels and the products' gated epilogues.
 CAPPED_GATE = "capped_sigmoid"
-_CAPPED_CODE = 4
+_CAPPED_CODE = 5
 
 
 def activation_code(name: str, capped_ok: bool = False) -> int:
@@ -928,20 +976,32 @@ def _check_attention(q, k_cache, v_cache, out, block_table, num_kv_heads, page_t
 
 
 def _extended_choice(q, k_cache, v_cache, page_tokens: int, ring_tokens: int, scale: float, penalty, keep_first: int, sink: bool, v_dim,
-                     chunk, impl: str | None, mma: str) -> str | None:
+                     chunk, impl: str | None, mma: str, softcap: float | None = None) -> str | None:
     """The kernel for a call that asks for a linear distance penalty (``penalty`` = (slopes, None)), kept first keys, a
-    softmax sink, or values that are the head of the cached key rows; None for a call that asks for none of these.  The
-    mma.sync kernels (``mma`` names the caller's) compute the first three for values as wide as the keys; the generic
-    kernels compute all four."""
-    if not ((penalty is not None and penalty[1] is None) or keep_first > 0 or sink or v_dim is not None):
+    softmax sink, a cap on the scores, or values that are the head of the cached key rows; None for a call that asks for none of
+    these.  The mma.sync kernels (``mma`` names the caller's) compute the first four for values as wide as the keys (a cap goes
+    with no penalty), the tcgen05 prefill kernel a sink and a cap; the generic kernels compute everything."""
+    if not ((penalty is not None and penalty[1] is None) or keep_first > 0 or sink or v_dim is not None or softcap is not None):
         return None
     fits = (v_dim is None and v_cache.shape[-1] == q.shape[2] and attention_mma_supported(q, page_tokens) and scale > 0
-            and not (keep_first > 0 and (ring_tokens or chunk)))
+            and not (keep_first > 0 and (ring_tokens or chunk)) and not (softcap is not None and penalty is not None))
+    if mma == "mma" and impl in (None, "tc") and fits and penalty is None and not keep_first and attention_tc_supported(q, page_tokens):
+        return "tc"
     if impl in (None, mma) and fits:
         return mma
     if impl in (None, "generic"):
         return "generic"
-    raise KernelError(f"attention kernel {impl!r} does not take this call (linear penalty, kept first keys, sink or values inside the key rows)")
+    raise KernelError(f"attention kernel {impl!r} does not take this call (linear penalty, kept first keys, sink, score cap or values inside the key rows)")
+
+
+def _cap_args(softcap: float | None, score_bound: float | None) -> tuple[float, int]:
+    """The cap for a kernel (0: none), and whether every score is known to stay within it: |score| <= softcap, with room for the
+    rounding of queries and keys to bfloat16."""
+    if softcap is None:
+        return 0.0, 0
+    if softcap <= 0:
+        raise KernelError(f"attention: a score cap of {softcap}")
+    return float(softcap), 1 if score_bound is not None and 1.02 * score_bound <= softcap else 0
 
 
 def _plain_attention(q: torch.Tensor, v_cache: torch.Tensor, penalty) -> bool:
@@ -997,12 +1057,13 @@ def _pick_attention(q: torch.Tensor, page_tokens: int, impl: str | None, prefill
 
 
 def attention_latent_supported(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, num_kv_heads: int, page_tokens: int,
-                               ring_tokens: int, window, scale: float, penalty, chunk, keep_first: int, sink: bool, v_dim) -> bool:
+                               ring_tokens: int, window, scale: float, penalty, chunk, keep_first: int, sink: bool, v_dim, softcap=None) -> bool:
     """The tensor-core kernel for cached latent rows takes bfloat16, one key head whose rows are the values' source
     too, rows and value sizes that are multiples of 8 (values up to 512, a row within shared memory), a positive
     scale, pages of 64 tokens and a plain causal softmax, over all earlier keys or a window of them."""
     return (v_dim is not None and v_cache is k_cache and num_kv_heads == 1 and ring_tokens % 64 == 0 and (not ring_tokens or bool(window))
-            and penalty is None and not chunk and not keep_first and not sink and scale > 0 and attention_latent_shape(q.dtype, q.shape[2], v_dim, page_tokens))
+            and penalty is None and not chunk and not keep_first and not sink and softcap is None and scale > 0
+            and attention_latent_shape(q.dtype, q.shape[2], v_dim, page_tokens))
 
 
 def attention_latent_shape(dtype: torch.dtype, row: int, rank: int, page_tokens: int) -> bool:
@@ -1024,7 +1085,7 @@ def attention_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
                       num_kv_heads: int, page_tokens: int, ring_tokens: int, window: int | None, scale: float,
                       impl: str | None = None, penalty: tuple[torch.Tensor, torch.Tensor] | None = None,
                       chunk: int | None = None, keep_first: int = 0, sink: bool = False, v_dim: int | None = None,
-                      sinks: torch.Tensor | None = None) -> None:
+                      sinks: torch.Tensor | None = None, softcap: float | None = None, score_bound: float | None = None) -> None:
     """Causal attention of packed sequences over the cache (which already holds this step's keys).
     ``chunk``: a query at position i sees key j only if i // chunk == j // chunk as well.  A value cache with fewer
     heads than the key cache serves key head g with value head g % (value heads).
@@ -1033,13 +1094,14 @@ def attention_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     r1_h * ln(1 + r2_h * (i - j)); ``penalty`` = (slopes, None): it loses slope_h * (i - j).
     ``keep_first``: a windowed query also sees the keys at positions below it.  ``sink``: the softmax has one more term
     of score 0 without a value, or, with ``sinks`` (float [heads]), of the head's own score, taken as it is (not scaled).  ``v_dim``: the values are the first ``v_dim`` elements of the rows of ``v_cache`` (which
-    may be the key cache itself)."""
+    may be the key cache itself).  ``softcap``: scores pass softcap * tanh(score / softcap), the sink's does not; ``score_bound``: what the
+    caller knows no score's size to exceed (a cheaper form of the cap where that is within the cap)."""
     _, num_heads, head_dim = _check_attention(q, k_cache, v_cache, out, block_table, num_kv_heads, page_tokens, penalty, v_dim)
     if sinks is not None:
         _need(sinks, "sinks", torch.float32, (num_heads,))
         sink = True
     if impl in (None, "latent") and attention_latent_supported(q, k_cache, v_cache, num_kv_heads, page_tokens, ring_tokens, window, scale, penalty,
-                                                               chunk, keep_first, sink, v_dim):
+                                                               chunk, keep_first, sink, v_dim, softcap):
         n_seqs = seq_past.shape[0]
         _need(seq_start, "seq_start", torch.int32, (n_seqs + 1,))
         _need(seq_past, "seq_past", torch.int32)
@@ -1050,7 +1112,7 @@ def attention_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         return
     if impl == "latent":
         raise KernelError("the tensor-core kernel for cached latent rows does not take this call")
-    extended = _extended_choice(q, k_cache, v_cache, page_tokens, ring_tokens, scale, penalty, keep_first, sink, v_dim, chunk, impl, "mma")
+    extended = _extended_choice(q, k_cache, v_cache, page_tokens, ring_tokens, scale, penalty, keep_first, sink, v_dim, chunk, impl, "mma", softcap)
     if extended is not None:
         impl = extended
     elif not _plain_attention(q, v_cache, penalty):
@@ -1061,25 +1123,26 @@ def attention_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     if block_table.shape[0] < n_seqs:
         raise KernelError("attention_prefill: block table has fewer rows than sequences")
     choice = _pick_attention(q, page_tokens, impl, prefill=True)
+    cap, cap_small = _cap_args(softcap, score_bound)
     if choice == "tc":
         _call("attention_tc", "qt_attention_prefill_tc", _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), q.shape[0],
               k_cache.shape[0], _ptr(block_table), block_table.shape[1], _ptr(seq_start), _ptr(seq_past), n_seqs,
               int(max_q_len), num_heads, num_kv_heads, head_dim, page_tokens, ring_tokens, int(window or 0), float(scale),
               _ptr(penalty[0]) if penalty else None, _ptr(penalty[1]) if penalty else None, int(chunk or 0), v_cache.shape[1],
-              _ptr(_status_word(q.device)), _stream())
+              1 if sink else 0, _ptr(sinks), cap, cap_small, _ptr(_status_word(q.device)), _stream())
         return
     if choice == "mma":
         _call("attention_mma", "qt_attention_prefill_mma", _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out),
               _ptr(block_table), block_table.shape[1], _ptr(seq_start), _ptr(seq_past), n_seqs, int(max_q_len), num_heads,
               num_kv_heads, head_dim, page_tokens, ring_tokens, int(window or 0), float(scale),
               _ptr(penalty[0]) if penalty else None, _ptr(penalty[1]) if penalty else None, int(chunk or 0), v_cache.shape[1],
-              int(keep_first), 1 if sink else 0, _ptr(sinks), _stream())
+              int(keep_first), 1 if sink else 0, _ptr(sinks), cap, cap_small, _stream())
         return
     _call("attention", "qt_attention_prefill", _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _code(q, "q"),
           _ptr(block_table), block_table.shape[1], _ptr(seq_start), _ptr(seq_past), n_seqs, int(max_q_len), num_heads,
           num_kv_heads, head_dim, page_tokens, ring_tokens, int(window or 0), float(scale), int(v_dim or v_cache.shape[-1]),
           _ptr(penalty[0]) if penalty else None, _ptr(penalty[1]) if penalty else None, int(chunk or 0), v_cache.shape[1],
-          int(keep_first), 1 if sink else 0, v_cache.shape[-1], _ptr(sinks), _stream())
+          int(keep_first), 1 if sink else 0, v_cache.shape[-1], _ptr(sinks), cap, _stream())
 
 
 def _ws_merges_in_cluster(n_splits: int, warps: int, group: int, head_dim: int) -> bool:
@@ -1099,7 +1162,8 @@ def attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      ring_tokens: int, window: int | None, scale: float, n_splits: int,
                      part_acc: torch.Tensor | None, part_ml: torch.Tensor | None, impl: str | None = None,
                      warps: int = 1, penalty: tuple[torch.Tensor, torch.Tensor] | None = None, chunk: int | None = None,
-                     keep_first: int = 0, sink: bool = False, v_dim: int | None = None, sinks: torch.Tensor | None = None) -> None:
+                     keep_first: int = 0, sink: bool = False, v_dim: int | None = None, sinks: torch.Tensor | None = None,
+                     softcap: float | None = None, score_bound: float | None = None) -> None:
     """One query token per sequence; ``seq_len`` counts the keys it sees (its own included).
 
     With ``n_splits`` > 1 the keys of each sequence are cut into that many ranges whose partial
@@ -1114,7 +1178,7 @@ def attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         _need(sinks, "sinks", torch.float32, (num_heads,))
         sink = True
     if impl in (None, "latent") and attention_latent_supported(q, k_cache, v_cache, num_kv_heads, page_tokens, ring_tokens, window, scale, penalty,
-                                                               chunk, keep_first, sink, v_dim):
+                                                               chunk, keep_first, sink, v_dim, softcap):
         if n_splits > 1:
             _need(part_acc, "part_acc", torch.float32)
             _need(part_ml, "part_ml", torch.float32)
@@ -1127,7 +1191,7 @@ def attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         raise KernelError("the tensor-core kernel for cached latent rows does not take this call")
     if impl == "mma" and _special_mask(k_cache, v_cache, chunk):
         raise KernelError("the block-tile decode kernel takes no mask in chunks and no value heads shared by several key heads")
-    extended = _extended_choice(q, k_cache, v_cache, page_tokens, ring_tokens, scale, penalty, keep_first, sink, v_dim, chunk, impl, "ws")
+    extended = _extended_choice(q, k_cache, v_cache, page_tokens, ring_tokens, scale, penalty, keep_first, sink, v_dim, chunk, impl, "ws", softcap)
     if extended is not None:
         impl = extended
     elif not _plain_attention(q, v_cache, penalty):
@@ -1145,18 +1209,19 @@ def attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     common = (_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), block_table.shape[1], _ptr(seq_len),
               n_seqs, num_heads, num_kv_heads, head_dim, page_tokens, ring_tokens, int(window or 0), float(scale), int(n_splits))
     launches = 2 if n_splits > 1 else 1
+    cap, cap_small = _cap_args(softcap, score_bound)
     if picked == "ws" and _ws_merges_in_cluster(n_splits, warps, num_heads // num_kv_heads, head_dim):
         launches = 1
     if picked == "ws":
         _call("attention_mma", "qt_attention_decode_ws", *common, int(warps), _ptr(part_acc), _ptr(part_ml),
               _ptr(penalty[0]) if penalty else None, _ptr(penalty[1]) if penalty else None, int(chunk or 0), v_cache.shape[1],
-              int(keep_first), 1 if sink else 0, _ptr(sinks), _stream(), launches=launches)
+              int(keep_first), 1 if sink else 0, _ptr(sinks), cap, cap_small, _stream(), launches=launches)
     elif picked == "mma":
         _call("attention_mma", "qt_attention_decode_mma", *common, _ptr(part_acc), _ptr(part_ml), _stream(), launches=launches)
     else:
         _call("attention", "qt_attention_decode", *common[:4], _code(q, "q"), *common[4:], _ptr(part_acc), _ptr(part_ml),
               int(v_dim or v_cache.shape[-1]), _ptr(penalty[0]) if penalty else None, _ptr(penalty[1]) if penalty else None,
-              int(chunk or 0), v_cache.shape[1], int(keep_first), 1 if sink else 0, v_cache.shape[-1], _ptr(sinks), _stream(), launches=launches)
+              int(chunk or 0), v_cache.shape[1], int(keep_first), 1 if sink else 0, v_cache.shape[-1], _ptr(sinks), cap, _stream(), launches=launches)
 
 
 # ----------------------------------------------------------------------------- experts chosen by a table

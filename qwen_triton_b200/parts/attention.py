@@ -34,6 +34,9 @@ Further parameters, each off unless given, for designs that treat scores or valu
   positions; the cache then keeps every key (no ring) and the kernels mask;
 * ``sink`` = "learned": the softmax's denominator also holds exp(s_h), one stored number per query head
   (tensor ``names["sink"]``) that is not scaled and has no value; ``sink`` = True: the same with s_h = 0;
+* ``softcap``: scores pass softcap * tanh(score / softcap) ahead of the softmax (the sink's does not); unit-norm queries and keys bound
+  every score by head_dim * scale, which the kernels use where it is within the cap;
+* ``bias`` with ``float_proj``: the q, k and v biases are added to the projection's float sums, ahead of norm and rotation;
 * ``head_gate``: every head's output is multiplied by sigmoid(w_h . x), one number per head; the rows W_g [heads, hidden]
   (tensor ``names["g"]``) ride at the end of the q/k/v projection, whose sums are then float (``float_proj`` asks for
   float sums by itself).
@@ -89,6 +92,9 @@ class Attention:
         self.sink = params.get("sink", False)
         if self.sink not in (False, True, "learned"):
             raise ValueError(f"{prefix}: sink={self.sink!r} is none of False, True, 'learned'")
+        self.softcap = float(params["softcap"]) if params.get("softcap") is not None else None
+        if self.softcap is not None and self.softcap <= 0:
+            raise ValueError(f"{prefix}: a score cap of {self.softcap}")
         self.head_gate = bool(params.get("head_gate", False))
         self.float_proj = bool(params.get("float_proj", False)) or self.head_gate
         self.sinks = None
@@ -115,7 +121,9 @@ class Attention:
         # values that are treated before they are cached: bias, treatment and cache write are one kernel of their own
         self.treated = self.v_norm_eps is not None or self.v_blend is not None or self.dv != self.d
         # values of their own shape that are otherwise untouched go with q/k norm and rotation (one kernel writes all)
-        self.own_values = self.treated and self.v_norm_eps is None and self.v_blend is None and not self.bias
+        self.own_values = self.treated and self.v_norm_eps is None and self.v_blend is None and (not self.bias or self.float_proj)
+        # no score can be larger than this (unit-norm queries and keys)
+        self.score_bound = self.d * abs(self.scale) if self.norm_mode == "unit" else None
         if self.maps > 1 or self.norm_mode in ("unit", "whole") or self.float_proj:
             self.own_values = True            # the general kernel behind the projection
         if self.own_values:
@@ -124,9 +132,12 @@ class Attention:
             raise ValueError(f"{prefix}: treated values (v_norm, v_blend) go with no rotation, no q/k norm and keys of the layer's own")
         if self.maps > 1 and (self.bias or self.window or self.penalised or self.sink or self.head_gate or self.norm_mode in ("unit", "whole")):
             raise ValueError(f"{prefix}: differential attention goes with no bias, window, distance penalty, sink, gate or norm of another kind")
-        if (self.keep_first or self.sink or self.head_gate or self.norm_mode in ("unit", "whole")) and (self.treated or self.bias or not self.own_kv or self.chunk):
+        if (self.keep_first or self.sink or self.head_gate or self.norm_mode in ("unit", "whole")) \
+                and (self.treated or (self.bias and (not self.float_proj or self.head_gate)) or not self.own_kv or self.chunk):
             raise ValueError(f"{prefix}: kept first keys, a sink, a gate per head and the unit and whole-row norms go with untreated values, "
-                             "no bias, no chunks and keys of the layer's own")
+                             "no bias (but on float sums without a gate), no chunks and keys of the layer's own")
+        if self.softcap is not None and self.penalised:
+            raise ValueError(f"{prefix}: a score cap goes with no distance penalty")
         self.gate_cols = -(-self.heads_out // 8) * 8 if self.head_gate else 0       # the gate's rows, padded so that rows of sums stay aligned
         # the mma.sync attention kernels take values as wide as the keys (and compute the distance penalty, given a
         # positive scale); everything else goes to the generic kernels
@@ -134,7 +145,8 @@ class Attention:
         proj_rows = self.nq * self.d + ((self.nkv * self.d + self.v_heads * self.dv) if self.own_kv else 0) + self.gate_cols
         self.at_gate = proj_rows - self.gate_cols
         if self.own_values:
-            self.qkv = Linear("attn.qkv.own_values" + (".float" if self.float_proj else ""), proj_rows, self.hidden, runtime, float_out=self.float_proj)
+            self.qkv = Linear("attn.qkv.own_values" + (".float" if self.float_proj else "") + (".biased" if self.bias else ""), proj_rows, self.hidden,
+                              runtime, float_out=self.float_proj, bias=self.bias)
         elif self.treated:
             self.qkv = Linear("attn.qkv.sums", proj_rows, self.hidden, runtime, float_out=True)      # float sums: the bias is added behind it
         else:
@@ -363,11 +375,13 @@ class Attention:
                                      cache.ring_tokens, self.window, self.scale, n_splits,
                                      ws.view("attn.part_acc", _MAX_SPLIT_PAIRS * self.nq * self.dv),
                                      ws.view("attn.part_ml", _MAX_SPLIT_PAIRS * self.nq * 2), warps=warps, penalty=penalty,
-                                     chunk=self.chunk, keep_first=self.keep_first, sink=bool(self.sink), sinks=self.sinks)
+                                     chunk=self.chunk, keep_first=self.keep_first, sink=bool(self.sink), sinks=self.sinks, softcap=self.softcap,
+                                     score_bound=self.score_bound)
         else:
             kernels.attention_prefill(q, cache.k, cache.v, out, table, ctx.seq_start, ctx.seq_past, ctx.max_q_len,
                                       self.nkv, cache.page_tokens, cache.ring_tokens, self.window, self.scale, penalty=penalty,
-                                      chunk=self.chunk, keep_first=self.keep_first, sink=bool(self.sink), sinks=self.sinks)
+                                      chunk=self.chunk, keep_first=self.keep_first, sink=bool(self.sink), sinks=self.sinks, softcap=self.softcap,
+                                      score_bound=self.score_bound)
         if self.head_gate:
             kernels.gate_mul(out.view(tokens, self.nq * self.dv), proj, self.at_gate, group=self.dv)
         if self.maps > 1:

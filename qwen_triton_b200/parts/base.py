@@ -189,6 +189,9 @@ class ResidualStream:
     kernel, which reads the stream anyway.  The addition may also be a product that is still to be
     launched (``DeferredProduct``): ``take_deferred`` hands it to a norm that fuses with it, reading
     ``pending`` launches it and gives its result.
+
+    A residual of several parallel streams is [T, S, H]; ``write`` then says how the pending addition enters them (a
+    ``HyperConnection``), and the norm that folds it also says what the next sublayer reads of them.
     """
 
     def __init__(self, residual: torch.Tensor, start: torch.Tensor | None = None) -> None:
@@ -196,6 +199,7 @@ class ResidualStream:
         self.start = start                 # the stream as the embedding left it [T, H] (activation dtype), for models whose stream maps read it
         self._pending: GemmOut | DeferredProduct | None = None
         self.more: list[GemmOut] = []      # further additions beside ``pending`` (a block whose parts run side by side)
+        self.write = None                  # how the pending addition enters a residual of several streams (``add(..., write=)``)
         self.post = None                   # a norm that the pending addition passes before it is added (``add(..., post=)``)
 
     @property
@@ -208,13 +212,14 @@ class ResidualStream:
     def pending(self, value: GemmOut | None) -> None:
         self._pending = value
 
-    def add(self, delta: "GemmOut | DeferredProduct", post=None) -> None:
+    def add(self, delta: "GemmOut | DeferredProduct", post=None, write=None) -> None:
         """Leave ``delta`` pending.  With ``post`` (a norm part) the addition is to be normed by it first: only a norm
         that says ``folds_post_norm`` takes such a stream (it reads ``stream.post`` and clears it); the others refuse it."""
         if self._pending is not None:
             raise RuntimeError("the residual stream already has a pending addition; apply a norm first")
         self._pending = delta
         self.post = post
+        self.write = write
 
     def add_beside(self, delta: GemmOut) -> None:
         """One more addition beside the pending one, for arrangements whose parts all read the same normed rows.  Only a
@@ -223,6 +228,11 @@ class ResidualStream:
             self._pending = delta
         else:
             self.more.append(delta)
+
+    @property
+    def several(self) -> bool:
+        """Whether the residual is several parallel streams."""
+        return self.residual.dim() == 3
 
     def take_all(self) -> list[GemmOut]:
         """Every pending addition, launched if need be; none is pending afterwards."""

@@ -11,6 +11,7 @@ from dataclasses import replace
 from ..config.spec import LayerSpec
 from ..weights.tensors import TensorSpec
 from .base import DeferredProduct, ResidualStream, Runtime, part_class, register_block
+from .hyper_connection import HyperConnection
 
 
 @register_block("pre_norm")
@@ -138,6 +139,48 @@ class SandwichBlock(PreNormBlock):
         x = self.feed_forward_norm.apply(stream)
         result = self.feed_forward.forward(x, ctx)
         stream.add(result.run() if isinstance(result, DeferredProduct) else result, post=self.feed_forward_post_norm)
+
+
+@register_block("hyper_connections")
+class HyperConnectionBlock(PreNormBlock):
+    """A pre-norm layer on a residual of several parallel streams: a sublayer reads norm(sum_s in[s] x_s), and its result y enters
+    as x_t <- sum_s mix[s, t] x_s + mult out[t] y, with an ``in``, a ``mix`` and an ``out`` of its own (see ``HyperConnection``).
+
+    The addition is left pending together with its connection (``stream.add(..., write=)``); the next norm updates the streams
+    and forms what it norms in one pass over them.  Block parameters: ``connection`` (the parameters of ``HyperConnection``) and
+    the name pieces ``mixer_connection`` and ``feed_forward_connection``."""
+
+    def __init__(self, layer: LayerSpec, runtime: Runtime) -> None:
+        super().__init__(layer, runtime)
+        params, names = layer.block["connection"], self._connection_names(layer)
+        self.mixer_connection = HyperConnection(params, names[0], runtime)
+        self.feed_forward_connection = HyperConnection(params, names[1], runtime) if layer.feed_forward is not None else None
+
+    @staticmethod
+    def _connection_names(layer: LayerSpec) -> tuple[str, str]:
+        p = layer.block.params
+        return tuple(f"{layer.prefix}.{p.get(key, key)}" for key in ("mixer_connection", "feed_forward_connection"))
+
+    @classmethod
+    def expected_tensors(cls, layer: LayerSpec) -> dict[str, TensorSpec]:
+        out = super().expected_tensors(layer)
+        first, second = (HyperConnection.expected_tensors(layer.block["connection"], name) for name in cls._connection_names(layer))
+        if layer.feed_forward is None:
+            second = {name: replace(spec, optional=True) for name, spec in second.items()}
+        out.update(first)
+        out.update(second)
+        return out
+
+    def parts(self) -> tuple:
+        return super().parts() + tuple(part for part in (self.mixer_connection, self.feed_forward_connection) if part is not None)
+
+    def forward(self, stream: ResidualStream, ctx, cache) -> None:
+        x = self.mixer_norm.apply(stream, read=self.mixer_connection.read)
+        stream.add(self.mixer.forward(x, ctx, cache), write=self.mixer_connection)
+        if self.feed_forward is None:
+            return
+        x = self.feed_forward_norm.apply(stream, read=self.feed_forward_connection.read)
+        stream.add(self.feed_forward.forward(x, ctx), write=self.feed_forward_connection)
 
 
 @register_block("parallel")

@@ -266,7 +266,8 @@ class RoutedExperts:
     ``normalize`` = False: the weights are the chosen scores themselves (times ``route_scale``), not divided by their sum.
     ``weight_on`` = "input": a pair's weight multiplies what its expert reads, not what it returns: the output is the sum of
     expert_e(w_e h), which for a gated expert is another function of w_e.  ``shared_gated`` = False: the shared expert is
-    added as it is, without a gate (and without the router's extra row).
+    added as it is, without a gate (and without the router's extra row).  ``router_bias``: the logits have a bias (tensor: the router's
+    name plus ``bias_suffix``, default ".bias"), added in float.
 
     The routing is computed on the device by a kernel behind the router's product, so a step launches the same
     kernels whatever the tokens are.  Few (token, expert) pairs run as matrix-vector passes per pair, many are
@@ -316,7 +317,11 @@ class RoutedExperts:
                                     "weight_suffix": params.get("weight_suffix", ".weight"), "float_out": True, "buffers": "experts.shared",
                                     "init_std": float(params.get("init_std", 0.02))},
                                    f"{prefix}.{params.get('shared_name', 'shared')}", runtime)
-        self.router = Linear("experts.router", self.experts + (1 if self.shared and self.shared_gated else 0), self.hidden, runtime, float_out=True)
+        self.router_bias = bool(params.get("router_bias", False))
+        if self.router_bias and self.shared is not None and self.shared_gated:
+            raise ValueError(f"{prefix}: a router with a bias goes with a shared expert that has no gate")
+        self.router = Linear("experts.router" + (".biased" if self.router_bias else ""), self.experts + (1 if self.shared and self.shared_gated else 0),
+                             self.hidden, runtime, float_out=True, bias=self.router_bias)
         self.up = self.down = None
         ws = runtime.workspace
         tokens = runtime.max_step_tokens
@@ -345,12 +350,18 @@ class RoutedExperts:
         shared_gate = f"{prefix}.{params.get('shared_name', 'shared')}.{params.get('shared_gate', 'gate_weight')}"
         return f"{prefix}.{params.get('router', 'router')}{suffix}", names, shared_gate
 
+    @staticmethod
+    def _router_bias_name(params, prefix: str) -> str:
+        return f"{prefix}.{params.get('router', 'router')}{params.get('bias_suffix', '.bias')}"
+
     @classmethod
     def expected_tensors(cls, params, prefix: str) -> dict[str, TensorSpec]:
         hidden, inter, experts = int(params["hidden_size"]), int(params["expert_size"]), int(params["experts"])
         router, names, shared_gate = cls._tensor_names(params, prefix)
         std = float(params.get("init_std", 0.02))
         out = {router: TensorSpec((experts, hidden), init_std=float(params.get("router_init_std", 0.1)))}
+        if params.get("router_bias", False):
+            out[cls._router_bias_name(params, prefix)] = TensorSpec((experts,), role="vector", init_std=0.3)
         for gate, up, down in names:
             out[gate] = TensorSpec((inter, hidden), init_std=std)
             out[up] = TensorSpec((inter, hidden), init_std=std)
@@ -376,6 +387,8 @@ class RoutedExperts:
             if self.shared_gated:
                 rows.append(source(shared_gate).to(dtype).reshape(1, self.hidden))
         self.router.set_weight(torch.cat(rows, dim=0))
+        if self.router_bias:
+            self.router.set_bias(source(self._router_bias_name(self.params, self.prefix)))
 
     def forward(self, x, ctx) -> GemmOut:
         tokens = x.shape[0]

@@ -2,7 +2,8 @@
 all heads share, and every head expands its keys and values from the latent with matrices of its own.
 
 From the mixer's input h: the query latent c_q = rms(W_dq h) w_q and q = W_uq c_q, laid out head by head as
-[``head_dim`` plain | ``rot_dim`` rotated]; W_dkv h = [``kv_rank`` | ``rot_dim``] rows, of which the first, RMS-normed with a
+[``head_dim`` plain | ``rot_dim`` rotated] (without ``q_rank`` there is no query latent: q = W_q h, rows of the first projection);
+W_dkv h = [``kv_rank`` | ``rot_dim``] rows, of which the first, RMS-normed with a
 weight, are the latent c and the last, rotated by the position encoding, the key part k_r shared by the heads.  Head h has
 k_h = W_uk_h c and v_h = W_uv_h c; its score is (q_plain_h . k_h + q_rot_h . k_r) * ``scale``, causal, over all earlier keys or
 the last ``window`` of them, plain softmax; the concatenated heads are multiplied by sigmoid(W_g h) (``gate`` true: one number
@@ -17,12 +18,15 @@ expanded per token, in prompts or in one-token steps.
 A layer with ``own_kv`` false has no W_dkv: it reads the cache rows of the schedule position named by ``LayerCall.cache_of``
 (which must have the same ``kv_rank``, ``rot_dim`` and rotation) under its own W_uk, W_uv, queries and everything else.
 
+A rotation of neighbouring pairs (2i, 2i + 1) becomes one of (i, i + dims / 2) when the weights are loaded: the rotated rows of the
+query's and of the shared key part's matrices are put in that order, which changes no score.
+
 Norms, rotation (float cos/sin table), scores, softmax and the gate are float; the query latent, the queries, the cache
 rows and the heads' outputs are rounded to the activation type between the products.
 
 Parameters: ``hidden_size``, ``num_heads``, ``head_dim``, ``rot_dim``, ``v_head_dim``, ``q_rank``, ``kv_rank``, ``scale``, ``eps``,
-``position`` (a position part over ``rot_dim``), ``window``, ``own_kv``, ``gate``, ``float_out``, and the tensor-name pieces ``dq``, ``uq``,
-``dkv``, ``uk``, ``uv``, ``g``, ``o``, ``weight_suffix``, ``norm_suffix``.
+``position`` (a position part over ``rot_dim``; either pairing), ``window``, ``own_kv``, ``gate``, ``float_out``, and the tensor-name pieces ``dq``, ``uq``
+(or ``q``), ``dkv``, ``uk``, ``uv``, ``g``, ``o``, ``weight_suffix``, ``norm_suffix``.
 """
 from __future__ import annotations
 
@@ -43,7 +47,7 @@ class LatentAttention:
         self.prefix, self.runtime, self.params = prefix, runtime, params
         self.hidden = int(params["hidden_size"])
         self.heads, self.d, self.rot, self.dv = (int(params[k]) for k in ("num_heads", "head_dim", "rot_dim", "v_head_dim"))
-        self.q_rank, self.rank = int(params["q_rank"]), int(params["kv_rank"])
+        self.q_rank, self.rank = int(params.get("q_rank") or 0), int(params["kv_rank"])      # q_rank 0: no query latent
         self.row = self.rank + self.rot                        # one cached row, and one head's query as the kernels see it
         if self.row > 640 or self.rank > 512:
             raise ValueError(f"{prefix}: a latent of {self.rank} + {self.rot} elements is beyond what the attention kernels take (512 + 128)")
@@ -55,21 +59,21 @@ class LatentAttention:
         self.window = int(params["window"]) if params.get("window") else None
         position_spec = params["position"]
         self.position = part_class("position", position_spec)(position_spec.params, runtime)
-        if getattr(self.position, "interleaved", False):
-            raise ValueError(f"{prefix}: the latent attention kernels rotate element i with element i + dims / 2")
+        self.interleaved = bool(getattr(self.position, "interleaved", False))
         self.cos_sin = None
-        self.at_kv = self.q_rank
-        self.at_gate = self.q_rank + (self.row if self.own_kv else 0)
+        self.at_kv = self.q_rank or self.heads * (self.d + self.rot)
+        self.at_gate = self.at_kv + (self.row if self.own_kv else 0)
         used = self.at_gate + (self.heads * (1 if self.head_gate else self.dv) if self.gated else 0)
         self.proj_rows = -(-used // 8) * 8
         self.proj = Linear("latent.proj" + ("" if self.own_kv else ".reader"), self.proj_rows, self.hidden, runtime, float_out=True, role="qkv")
         self.takes_scaled_rows = self.proj.fused_capable
-        self.uq = Linear("latent.uq", self.heads * (self.d + self.rot), self.q_rank, runtime)
+        self.uq = Linear("latent.uq", self.heads * (self.d + self.rot), self.q_rank, runtime) if self.q_rank else None
         float_out = bool(params.get("float_out", False))
         self.o = Linear("latent.o" + (".float" if float_out else ""), self.hidden, self.heads * self.dv, runtime, float_out=float_out, role="attn_out")
         ws = runtime.workspace
         tokens = runtime.max_step_tokens
-        ws.declare("latent.cq", tokens * self.q_rank, runtime.dtype)
+        if self.q_rank:
+            ws.declare("latent.cq", tokens * self.q_rank, runtime.dtype)
         ws.declare("latent.q", tokens * self.heads * self.row, runtime.dtype)
         ws.declare("latent.ctx", tokens * self.heads * self.rank, runtime.dtype)
         ws.declare("latent.heads", tokens * self.heads * self.dv, runtime.dtype)
@@ -81,18 +85,22 @@ class LatentAttention:
     @staticmethod
     def _names(params, prefix: str) -> dict[str, str]:
         w, nw = str(params.get("weight_suffix", ".weight")), str(params.get("norm_suffix", ".norm"))
-        n = {key: f"{prefix}.{params.get(key, key)}{w}" for key in ("dq", "uq", "dkv", "uk", "uv", "g", "o")}
+        n = {key: f"{prefix}.{params.get(key, key)}{w}" for key in ("dq", "uq", "q", "dkv", "uk", "uv", "g", "o")}
         n["dq_norm"], n["dkv_norm"] = f"{prefix}.{params.get('dq', 'dq')}{nw}", f"{prefix}.{params.get('dkv', 'dkv')}{nw}"
         return n
 
     @classmethod
     def expected_tensors(cls, params, prefix: str) -> dict[str, TensorSpec]:
         hidden, heads, d, rot, dv = (int(params[k]) for k in ("hidden_size", "num_heads", "head_dim", "rot_dim", "v_head_dim"))
-        q_rank, rank = int(params["q_rank"]), int(params["kv_rank"])
+        q_rank, rank = int(params.get("q_rank") or 0), int(params["kv_rank"])
         n = cls._names(params, prefix)
         std = float(params.get("init_std", 0.02))
-        out = {n["dq"]: TensorSpec((q_rank, hidden), init_std=std), n["dq_norm"]: TensorSpec((q_rank,), role="vector", init_std=0.1, init_mean=1.0),
-               n["uq"]: TensorSpec((heads * (d + rot), q_rank), init_std=std), n["uk"]: TensorSpec((heads * d, rank), init_std=std),
+        if q_rank:
+            out = {n["dq"]: TensorSpec((q_rank, hidden), init_std=std), n["dq_norm"]: TensorSpec((q_rank,), role="vector", init_std=0.1, init_mean=1.0),
+                   n["uq"]: TensorSpec((heads * (d + rot), q_rank), init_std=std)}
+        else:
+            out = {n["q"]: TensorSpec((heads * (d + rot), hidden), init_std=std)}
+        out |= {n["uk"]: TensorSpec((heads * d, rank), init_std=std),
                n["uv"]: TensorSpec((heads * dv, rank), init_std=std), n["o"]: TensorSpec((hidden, heads * dv), init_std=std)}
         if params.get("gate", True):
             out[n["g"]] = TensorSpec((heads * (1 if params.get("gate") == "head" else dv), hidden), init_std=std)
@@ -101,21 +109,32 @@ class LatentAttention:
             out[n["dkv_norm"]] = TensorSpec((rank,), role="vector", init_std=0.1, init_mean=1.0)
         return out
 
+    def _halves_order(self, weight: torch.Tensor, groups: int, plain: int) -> torch.Tensor:
+        """Rows stored as ``groups`` of [plain | rotated], the rotated ones of neighbouring pairs put in the order of a rotation of
+        halves: the even ones of the turning elements first, then the odd ones."""
+        if not self.interleaved:
+            return weight
+        turning = self.position.rotary_dim
+        place = torch.arange(plain + self.rot)
+        place[plain:plain + turning] = plain + torch.cat((torch.arange(0, turning, 2), torch.arange(1, turning, 2)))
+        return weight.view(groups, plain + self.rot, weight.shape[1])[:, place.to(weight.device)].reshape(weight.shape)
+
     def load(self, source) -> None:
         n = self._names(self.params, self.prefix)
         dtype, device = self.runtime.dtype, self.runtime.device
-        rows = [source(n["dq"]).to(dtype)]
+        rows = [source(n["dq"]).to(dtype) if self.q_rank else self._halves_order(source(n["q"]), self.heads, self.d).to(dtype)]
         if self.own_kv:
-            rows.append(source(n["dkv"]).to(dtype))
+            rows.append(self._halves_order(source(n["dkv"]), 1, self.rank).to(dtype))
         if self.gated:
             rows.append(source(n["g"]).to(dtype))
         used = sum(r.shape[0] for r in rows)
         if self.proj_rows > used:
             rows.append(torch.zeros(self.proj_rows - used, self.hidden, dtype=dtype, device=rows[0].device))
         self.proj.set_weight(torch.cat(rows, dim=0))
-        self.uq.set_weight(source(n["uq"]))
+        if self.q_rank:
+            self.uq.set_weight(self._halves_order(source(n["uq"]), self.heads, self.d))
+            self.q_norm = to_device(source(n["dq_norm"]), torch.float32, device)
         self.o.set_weight(source(n["o"]))
-        self.q_norm = to_device(source(n["dq_norm"]), torch.float32, device)
         if self.own_kv:
             self.kv_norm = to_device(source(n["dkv_norm"]), torch.float32, device)
         # W_uk per head, transposed: [heads, kv_rank, head_dim], the matrix of the product that carries a head's plain
@@ -158,12 +177,14 @@ class LatentAttention:
             raise ValueError(f"{self.prefix}: the cache rows it reads are not {self.rank} + {self.rot} elements long")
         table = ctx.block_table(cache.group)
         proj = self.proj.finished(x)
-        cq = ws.view("latent.cq", tokens, self.q_rank)
-        kernels.latent_prepare(proj, self.q_norm, self.kv_norm, self.eps, self.cos_sin, cq, cache.k if write else None, ctx.token_seq,
-                               ctx.token_pos, table if write else None, self.rank, self.rot, cache.page_tokens, cache.ring_tokens, write_kv=write)
-        q_full = self.uq(cq)                                                    # [*, T, heads * (d + rot)]
+        cq = ws.view("latent.cq", tokens, self.q_rank) if self.q_rank else None
+        if cq is not None or write:
+            kernels.latent_prepare(proj, self.q_norm, self.kv_norm, self.eps, self.cos_sin, cq, cache.k if write else None, ctx.token_seq,
+                                   ctx.token_pos, table if write else None, self.rank, self.rot, cache.page_tokens, cache.ring_tokens, write_kv=write,
+                                   at_kv=self.at_kv)
+        q_full = self.uq(cq) if cq is not None else proj                        # [*, T, heads * (d + rot)], or with the first projection's other columns behind
         q = ws.view("latent.q", tokens, self.heads, self.row)
-        kernels.head_product(q_full, self.uk_t, q, x_row=self.heads * (self.d + self.rot), x_head=self.d + self.rot)
+        kernels.head_product(q_full, self.uk_t, q, x_row=q_full.cols, x_head=self.d + self.rot)
         kernels.latent_query_rot(q_full, self.cos_sin, ctx.token_pos, q, self.heads, self.d, self.rot, self.rank)
         out = ws.view("latent.ctx", tokens, self.heads, self.rank)
         if ctx.is_decode:

@@ -43,7 +43,26 @@ class RMSNorm:
     def load(self, source) -> None:
         self.weight = to_device(source(self.tensor), torch.float32, self.runtime.device)
 
-    def apply(self, stream: ResidualStream, rows: torch.Tensor | None = None, lazy: bool = False):
+    def _apply_streams(self, stream: ResidualStream, rows, read):
+        """The same on a residual of several streams: the pending addition enters them as ``stream.write`` says, and what is normed
+        is their sum with the weights ``read`` (None: the plain sum)."""
+        if self.groups != 1:
+            raise RuntimeError(f"{self.name}: a norm in groups reads one stream, not {stream.residual.shape[1]}")
+        deferred = stream.take_deferred()
+        delta = stream.pending if deferred is None else deferred.linear.finished(deferred.x)
+        if delta is not None and stream.write is None:
+            raise RuntimeError(f"{self.name}: nothing says how the pending addition enters the {stream.residual.shape[1]} streams")
+        count = stream.residual.shape[0] if rows is None else rows.shape[0]
+        out = self.runtime.workspace.view("normed", count, self.size)
+        write = stream.write if delta is not None else None
+        kernels.streams_norm(stream.residual, delta, write.mix if write else None, write.out if write else None, read, self.weight, self.eps, out, rows)
+        if rows is None:
+            stream.pending = stream.write = None
+        else:
+            stream.pending = delta
+        return out
+
+    def apply(self, stream: ResidualStream, rows: torch.Tensor | None = None, lazy: bool = False, read: torch.Tensor | None = None):
         """Fold the pending delta into the stream and return the normed rows.
 
         With ``rows`` (int32 row numbers) only those rows are produced and the stream stays as it is.
@@ -59,6 +78,8 @@ class RMSNorm:
             raise RuntimeError(f"{self.name}: this norm folds one pending addition; the stream holds {1 + len(stream.more)}")
         if stream.post is not None:
             raise RuntimeError(f"{self.name}: the pending addition is to pass a norm of its own first, which this norm does not fold")
+        if stream.several:
+            return self._apply_streams(stream, rows, read)
         deferred = stream.take_deferred()
         if deferred is not None:
             count = stream.residual.shape[0]

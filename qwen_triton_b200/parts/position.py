@@ -30,16 +30,21 @@ class RotaryTable:
         self.angles = str(params.get("angles", "float32"))
         if self.angles not in ("float32", "float64"):
             raise ValueError(f"rotary angles in {self.angles!r} (float32 or float64)")
+        self.factor = float(params.get("factor", 1.0))                     # every frequency is divided by it (linear scaling)
+        if self.factor <= 0:
+            raise ValueError(f"rotary scaling by {self.factor}")
         self.runtime = runtime
 
     def key(self) -> tuple:
-        return ("rope", self.theta, self.rotary_dim, self.angles)          # the table does not depend on the pairing
+        return ("rope", self.theta, self.rotary_dim, self.angles, self.factor)          # the table does not depend on the pairing
 
     def table(self, max_positions: int) -> torch.Tensor:
         """float32 [max_positions, rotary_dim]: cos in the first half of each row, sin in the second."""
         work = torch.float64 if self.angles == "float64" else torch.float32
         exponent = torch.arange(0, self.rotary_dim, 2, dtype=work) / self.rotary_dim
         inv_freq = 1.0 / (self.theta ** exponent)
+        if self.factor != 1.0:
+            inv_freq = inv_freq / self.factor
         angles = torch.arange(max_positions, dtype=work)[:, None] * inv_freq[None, :]
         return torch.cat((angles.cos(), angles.sin()), dim=-1).to(torch.float32).contiguous().to(self.runtime.device)
 

@@ -33,7 +33,7 @@ import torch
 from ..ops import kernels
 from ..ops.kernels import GemmOut
 from ..weights.tensors import TensorSpec
-from .base import DeferredProduct, Runtime, StateRequest, register_mixer, to_device
+from .base import DeferredProduct, Runtime, StateRequest, part_class, register_mixer, to_device
 from .linear import Linear
 
 _UNIT_EPS = 1e-6      # inside the root of the unit norms of q and k
@@ -395,6 +395,107 @@ class GatedLinearAttention(_DecayedMixer):
         rows = proj if proj.n_splits == 1 else kernels.linear_attention_prepare(proj, self.at_gate, ws.view("gla.qkv", tokens, self.at_gate), False)
         read = ws.view("decayed.read", tokens, self.heads, self.vdim)
         kernels.decayed_attention(rows, 0, self.at_k, self.at_v, decay, cache.state, read, ctx, self.dim, self._scratch_views(),
+                                  out_scale=self.dim ** -0.5)
+        normed = ws.view("decayed.normed", tokens, width)
+        kernels.group_gate_norm(read.view(tokens, width), self.norm, self.eps, normed, groups=self.heads, proj=proj, at_gate=self.at_gate, gate="silu")
+        return self._output(normed, tokens)
+
+
+@register_mixer("retention")
+class Retention(_DecayedMixer):
+    """Linear attention with a fixed decay per head and rotated queries and keys ("retention"):
+
+        S <- decay_h S + k_t v_t^T;   o_t = dim^-1/2 S^T q_t
+
+    with q = R(W_q h), k = R(W_k h) ([heads, dim]) and v = W_v h ([heads, vdim]), R the rotation of the part ``position`` by the token's
+    position (pairs (i, i + dims / 2)).  Every head's o is divided by its root mean square over vdim (``eps`` inside the root, no
+    weight), the concatenated heads are multiplied by silu(W_g h) and projected by W_o.  Per sequence the mixer keeps the states,
+    float, zero for a new sequence, in the cache's per-slot state rows (stored transposed, [heads, vdim, dim]).  The four projections
+    of h run as one product with float sums; everything between it and the output projection is float
+    (``csrc/linear_attention.cu``, ``csrc/linear_attention_chunk.cu``: the kernels for decays that depend on the token, here given
+    the same logarithm for every token).
+
+    Parameters: ``hidden_size``, ``num_heads``, ``head_dim``, ``v_head_dim``, ``decay`` (one number per head, above 0 and at most 1),
+    ``position``, ``eps``, ``float_out``, ``init_std``, and the tensor-name pieces ``q``, ``k``, ``v``, ``g``, ``o``, ``weight_suffix``."""
+
+    def __init__(self, params, prefix: str, runtime: Runtime) -> None:
+        self.prefix, self.runtime, self.params = prefix, runtime, dict(params)
+        self.hidden = int(params["hidden_size"])
+        self.heads, self.dim = int(params["num_heads"]), int(params["head_dim"])
+        self.vdim = int(params.get("v_head_dim") or self.dim)
+        self.eps = float(params.get("eps", 1e-6))
+        self.decay_values = [float(d) for d in params["decay"]]
+        if len(self.decay_values) != self.heads or not all(0.0 < d <= 1.0 for d in self.decay_values):
+            raise ValueError(f"{prefix}: {self.heads} heads need as many decays above 0 and at most 1, not {self.decay_values}")
+        if self.dim > kernels.LINEAR_ATTENTION_MAX_DIM:
+            raise ValueError(f"{prefix}: {self.dim} key channels per head are beyond what the recurrence kernels hold "
+                             f"({kernels.LINEAR_ATTENTION_MAX_DIM})")
+        position_spec = params["position"]
+        self.position = part_class("position", position_spec)(position_spec.params, runtime)
+        if getattr(self.position, "interleaved", False):
+            raise ValueError(f"{prefix}: the recurrence's rotation pairs element i with element i + dims / 2")
+        self.cos_sin = None
+        self.at_k = self.heads * self.dim
+        self.at_v = 2 * self.heads * self.dim
+        self.at_gate = self.at_v + self.heads * self.vdim
+        self.proj_rows = -(-(self.at_gate + self.heads * self.vdim) // 8) * 8
+        self.proj = Linear("retention.proj", self.proj_rows, self.hidden, runtime, float_out=True, role="qkv")
+        self.takes_scaled_rows = self.proj.fused_capable
+        float_out = bool(params.get("float_out", False))
+        self.o = Linear("retention.o" + (".float" if float_out else ""), self.hidden, self.heads * self.vdim, runtime, float_out=float_out, role="attn_out")
+        runtime.workspace.declare("retention.qkv", runtime.max_step_tokens * self.at_gate, torch.float32)
+        self._declare_scratch(per_channel=False)
+        self.norm = self.log_decay = None
+
+    @staticmethod
+    def _names(params, prefix: str) -> dict[str, str]:
+        w = str(params.get("weight_suffix", ".weight"))
+        return {key: f"{prefix}.{params.get(key, key)}{w}" for key in ("q", "k", "v", "g", "o")}
+
+    @classmethod
+    def expected_tensors(cls, params, prefix: str) -> dict[str, TensorSpec]:
+        hidden, heads, dim = int(params["hidden_size"]), int(params["num_heads"]), int(params["head_dim"])
+        vdim = int(params.get("v_head_dim") or dim)
+        n = cls._names(params, prefix)
+        std = float(params.get("init_std", 0.02))
+        return {n["q"]: TensorSpec((heads * dim, hidden), init_std=std), n["k"]: TensorSpec((heads * dim, hidden), init_std=std),
+                n["v"]: TensorSpec((heads * vdim, hidden), init_std=std), n["g"]: TensorSpec((heads * vdim, hidden), init_std=std),
+                n["o"]: TensorSpec((hidden, heads * vdim), init_std=std)}
+
+    def load(self, source) -> None:
+        n = self._names(self.params, self.prefix)
+        dtype, device = self.runtime.dtype, self.runtime.device
+        rows = [source(n[key]).to(dtype) for key in ("q", "k", "v", "g")]
+        used = sum(r.shape[0] for r in rows)
+        if self.proj_rows > used:
+            rows.append(torch.zeros(self.proj_rows - used, self.hidden, dtype=dtype, device=rows[0].device))
+        self.proj.set_weight(torch.cat(rows, dim=0))
+        self.o.set_weight(source(n["o"]))
+        self.norm = torch.ones(self.vdim, dtype=torch.float32, device=device)
+        # the logarithms, formed in double, for as many tokens as a step may have
+        logs = torch.tensor(self.decay_values, dtype=torch.float64).log().to(torch.float32)
+        self.log_decay = logs.to(device).expand(self.runtime.max_step_tokens, self.heads).contiguous()
+        tables = self.runtime.options.setdefault("position_tables", {})
+        key = self.position.key() + (self.runtime.max_positions,)
+        if key not in tables:
+            tables[key] = self.position.table(self.runtime.max_positions)
+        self.cos_sin = tables[key]
+
+    def cache_request(self):
+        return StateRequest((self.heads, self.vdim, self.dim), torch.float32)
+
+    def forward(self, x, ctx, cache):
+        self._check(cache)
+        tokens, width = x.shape[0], self.heads * self.vdim
+        ws = self.runtime.workspace
+        proj = self.proj.finished(x)
+        if self.cos_sin is not None:
+            rows = kernels.linear_attention_rotate(proj, self.at_gate, ws.view("retention.qkv", tokens, self.at_gate), 2 * self.heads, self.dim, self.cos_sin,
+                                                   ctx.token_pos)
+        else:
+            rows = proj if proj.n_splits == 1 else kernels.linear_attention_prepare(proj, self.at_gate, ws.view("retention.qkv", tokens, self.at_gate), False)
+        read = ws.view("decayed.read", tokens, self.heads, self.vdim)
+        kernels.decayed_attention(rows, 0, self.at_k, self.at_v, self.log_decay[:tokens], cache.state, read, ctx, self.dim, self._scratch_views(),
                                   out_scale=self.dim ** -0.5)
         normed = ws.view("decayed.normed", tokens, width)
         kernels.group_gate_norm(read.view(tokens, width), self.norm, self.eps, normed, groups=self.heads, proj=proj, at_gate=self.at_gate, gate="silu")
