@@ -1,7 +1,7 @@
 """Decode and prefill throughput of the Qwen3-8B shape on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl b200|reference] [--temperature T]
-    python bench.py --workload 0.6b-unequal | 32b-long | lederax-layers | vunepel-layers | bisodra-layers | regupel-layers | misudra-layers
+    python bench.py --workload 0.6b-unequal | 32b-long | lederax-layers | vunepel-layers | bisodra-layers | regupel-layers | misudra-layers | bizurax-layers
 
 Prints ONE JSON line.  ``value`` is decoded tokens per second at batch 8 from a 2,048-token cache,
 timed on the device over the decode steps (step function plus greedy sampling kernel, tokens given
@@ -29,7 +29,10 @@ design: two parallel layers, windowed attention with kept first keys beside a li
 attention layers with a sink and a gate per head, each with routed experts and a shared expert, beside the Vunepel layers
 of equal size; the same three options), ``misudra-layers`` (four layers of the Misudra design: a gated linear attention with a
 dense feed-forward, a state-space layer, a windowed attention through a latent and a second gated linear attention with routed
-experts, the first two behind a map of the stream, beside Vunepel layers of equal size; the same three options).
+experts, the first two behind a map of the stream, beside Vunepel layers of equal size; the same three options), ``bizurax-layers``
+(four layers of the Bizurax design over a residual of parallel streams: a latent attention and an attention with capped scores and a
+sink, each with a dense feed-forward, and two retention layers with routed experts and a shared one, beside Misudra layers and Qwen3
+dense layers of equal size; the same three options).
 """
 from __future__ import annotations
 
@@ -63,9 +66,10 @@ def parse_args():
     parser.add_argument("--no-prefill", action="store_true")
     parser.add_argument("--min-seconds", type=float, default=2.0, help="a timed region lasts at least this long")
     parser.add_argument("--temperature", type=float, default=0.0, help="sampling temperature of the end-to-end run (0: greedy)")
-    parser.add_argument("--workload", default=None, choices=["0.6b-unequal", "32b-long", "lederax-layers", "vunepel-layers", "bisodra-layers", "regupel-layers", "misudra-layers"])
+    parser.add_argument("--workload", default=None, choices=["0.6b-unequal", "32b-long", "lederax-layers", "vunepel-layers", "bisodra-layers", "regupel-layers", "misudra-layers",
+                                                                  "bizurax-layers"])
     parser.add_argument("--size", default=None, help="vunepel-layers, bisodra-layers: only the size whose name starts with this")
-    parser.add_argument("--arm", default=None, choices=["vunepel", "bisodra", "regupel", "misudra", "dense"], help="vunepel-layers, bisodra-layers, regupel-layers: only this model")
+    parser.add_argument("--arm", default=None, choices=["vunepel", "bisodra", "regupel", "misudra", "bizurax", "dense"], help="vunepel-layers, bisodra-layers, regupel-layers: only this model")
     parser.add_argument("--phase", default=None, choices=["prefill", "decode8", "decode64"], help="vunepel-layers, bisodra-layers: only this measurement")
     return parser.parse_args()
 
@@ -654,6 +658,108 @@ def run_misudra_layers(args) -> dict:
             "sizes": out}
 
 
+# ----------------------------------------------------------------------------- the Bizurax design beside Misudra and the dense model
+BIZURAX_SIZES = (
+    # name, width, streams, attention heads, kv heads, head size, latent heads, plain, rotated and value sizes, latent size, retention heads,
+    # key and value channels, experts, top, expert width, shared width, dense width
+    ("w2048-s4-attn16x128-latent16-ret16x128-e16x1024-top2", 2048, 4, 16, 4, 128, 16, 128, 64, 128, 512, 16, 128, 128, 16, 2, 1024, 2048, 8192),
+    ("w4096-s4-attn32x128-latent32-ret32x128-e16x2048-top2", 4096, 4, 32, 8, 128, 32, 128, 64, 128, 512, 32, 128, 128, 16, 2, 2048, 2048, 16384),
+    ("w1024-s2-attn16x64-latent8-ret8x64-e8x2048-top1", 1024, 2, 16, 4, 64, 8, 64, 32, 64, 256, 8, 64, 128, 8, 1, 2048, 1024, 4096),
+)
+
+
+def run_bizurax_layers(args) -> dict:
+    """Prefill and one-token steps of four Bizurax layers at sizes that resemble a real model's (latent attention and a dense
+    feed-forward; retention with routed experts and a shared one; attention with capped scores and a sink and a dense
+    feed-forward; a second retention layer with experts), over a residual of parallel streams.  Beside them the layers of the two
+    designs that come closest: Misudra (the same latent attention without an effective window, recurrences with the same state
+    where the retention layers stand, experts, gated dense feed-forwards that read as many weights) and Qwen3 dense layers
+    (attention of the same heads and head size)."""
+    import torch
+
+    from qwen_triton_b200 import QwenB200ForCausalLM, config_from_dict
+
+    peak, peak_source = peaks()
+    vocab, prompt_len = 32768, args.prompt_len
+    out = []
+    for size in BIZURAX_SIZES:
+        (name, width, streams, heads, kv, dim, l_heads, plain, rot, l_vdim, latent, r_heads, r_dim, r_vdim, experts, top, ff, shared, dense) = size
+        if args.size and not name.startswith(args.size):
+            continue
+        gated = dense * 2 // 3 // 64 * 64                     # a gated feed-forward that reads as many weights as the dense one of two matrices
+        attention = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 30.0,
+                     "rot": {"base": 500000.0, "dims": dim, "scaling": {"factor": 4.0}}}
+        through = {"heads": l_heads, "dim": plain, "rot_dim": rot, "vdim": l_vdim, "kv_rank": latent, "scale": (plain + rot) ** -0.5,
+                   "rot": {"base": 500000.0, "dims": rot}}
+        keep = {"heads": r_heads, "dim": r_dim, "vdim": r_vdim, "decay": [1.0 - 2.0 ** (-5 - 7.0 * h / r_heads) for h in range(r_heads)],
+                "rot": {"base": 500000.0, "dims": r_dim}}
+        moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared}}
+        bizurax = {"architecture": "Bizurax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "streams": streams, "residual_mult": 0.5,
+                   "layers": [{"type": "latent_attention", "mixer": through, "mlp": {"kind": "dense", "ff": dense}}, {"type": "retention", "mixer": keep, "mlp": moe},
+                              {"type": "attention", "mixer": attention, "mlp": {"kind": "dense", "ff": dense}}, {"type": "retention", "mixer": keep, "mlp": moe}]}
+        m_through = {**through, "q_rank": 1536 * width // 4096, "mask": {"size": prompt_len + 512}}
+        m_moe = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": experts, "top": top}}
+        m_gla = {"heads": r_heads, "dim": r_dim, "vdim": r_vdim, "tau": 16.0, "ranks": {"decay": 16}}
+        m_space = {"heads": r_heads, "vdim": r_vdim, "state": r_dim, "groups": max(1, r_heads // 8), "conv": 4, "norm_groups": r_heads}
+        misudra = {"architecture": "Misudra", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "loop": {"start": 0, "stop": 4, "times": 1},
+                   "layers": [{"type": "latent_attention", "mixer": m_through, "mlp": {"kind": "dense", "ff": gated}}, {"type": "mamba2", "mixer": m_space, "mlp": m_moe},
+                              {"type": "latent_attention", "mixer": m_through, "mlp": {"kind": "dense", "ff": gated}}, {"type": "gla", "mixer": m_gla, "mlp": m_moe}]}
+        qwen3 = {"architectures": ["Qwen3ForCausalLM"], "model_type": "qwen3", "vocab_size": vocab, "hidden_size": width, "intermediate_size": gated,
+                 "num_hidden_layers": 4, "num_attention_heads": heads, "num_key_value_heads": kv, "head_dim": dim, "max_position_embeddings": 32768}
+        # weights a token multiplies with (the experts: the chosen ones)
+        attn_w = width * (2 * heads + 2 * kv) * dim
+        latent_w = width * (l_heads * (plain + rot) + latent + rot) + l_heads * (plain * latent + l_vdim * latent + l_vdim * width)
+        keep_w = width * r_heads * (2 * r_dim + 3 * r_vdim)
+        m_latent_w = latent_w - width * l_heads * (plain + rot) + m_through["q_rank"] * (width + l_heads * (plain + rot)) + width * l_heads
+        inner = r_heads * r_vdim
+        m_rec_w = width * (3 * inner + 2 * m_space["groups"] * r_dim + r_heads) + width * (r_heads * (2 * r_dim + 3 * r_vdim) + 16) + 16 * r_heads * r_dim
+
+        def moe_weights(count):
+            return 3 * width * ff * count + width * experts
+
+        states = 2 * 2 * 4 * r_heads * r_dim * r_vdim          # two layers' states, read and written
+        pair_latent, row_latent = 2 * l_heads * (2 * latent + rot), 2 * (latent + rot)
+        pair_attn, row_attn = 4 * heads * dim, 4 * kv * dim
+        # label, model, weights outside the experts, expert layers, FLOPs per visible pair, cached bytes per token, state bytes
+        arms = (("bizurax", bizurax, attn_w + latent_w + 2 * keep_w + 4 * width * dense + 6 * width * shared, 2, pair_latent + pair_attn, row_latent + row_attn, states),
+                ("misudra", misudra, 2 * m_latent_w + m_rec_w + 6 * width * gated + 2 * width * width, 2, 2 * pair_latent, 2 * row_latent, states),
+                ("dense", qwen3, 4 * (attn_w + 3 * width * gated), 0, 4 * pair_attn, 4 * row_attn, 0))
+        entry = {"size": name, "layers": 4}
+        for label, raw, weights, moes, pair_flops, key_bytes, state_bytes in arms:
+            if args.arm and label != args.arm:
+                continue
+            model = QwenB200ForCausalLM.from_config(config_from_dict(raw), seed=1, dtype="bf16",
+                                                    max_tokens=64 * (prompt_len + 512), max_seq_len=prompt_len + 512,
+                                                    max_step_tokens=max(4096, prompt_len), chunk_tokens=prompt_len)
+            result = {}
+            if args.phase in (None, "prefill"):
+                ms = time_prefill(model, prompt_len, vocab, repeats=args.steps if args.phase else 5, warmup=args.warmup if args.phase else 3)
+                flops = 2 * prompt_len * (weights + moes * moe_weights(top) + vocab * width / prompt_len) + pair_flops * prompt_len * (prompt_len + 1) // 2
+                result["prefill"] = {"tokens": prompt_len, "ms": round(ms, 3), "tokens_per_s": round(prompt_len * 1e3 / ms),
+                                     "tensor_fraction": round(flops / (ms * 1e-3) / (peak["bf16_tflops"] * 1e12), 4)}
+            for batch in (8, 64):
+                if args.phase not in (None, f"decode{batch}"):
+                    continue
+                prompts = random_prompts(batch, prompt_len, vocab, 300 + batch)
+                ms, launches, clocks, context, steps = time_decode(model, prompts, args.steps, args.warmup, vocab,
+                                                                   args.min_seconds / 4, 256)
+                read = 2 * (weights + moes * moe_weights(min(experts, batch * top)) + vocab * width) + batch * (key_bytes * context + state_bytes)
+                result[f"decode_batch{batch}"] = {"ms_per_step": round(ms, 4), "tokens_per_s": round(batch * 1e3 / ms),
+                                                   "launches_per_step": round(launches / steps, 1), "steps": steps,
+                                                   "hbm_fraction": round(read / (ms * 1e-3) / (peak["hbm_gbs"] * 1e9), 4),
+                                                   "clocks": clocks}
+            entry[label] = result
+            print(f"[bench] {name} {label}: " + json.dumps({k: {a: b for a, b in v.items() if a != 'clocks'} for k, v in result.items()}),
+                  file=sys.stderr, flush=True)
+            del model
+            torch.cuda.empty_cache()
+        out.append(entry)
+    return {"workload": args.workload, "impl": "b200", "dtype": "bf16", "data": "synthetic", "n_gpus": 1,
+            "config": {"prompt_len": prompt_len, "layers": 4, "vocab": vocab, "peaks": peak_source,
+                       "l2": "weights, caches and states of a step exceed L2 at every size but the smallest"},
+            "sizes": out}
+
+
 def time_prefill(model, tokens: int, vocab: int, repeats: int = 5, warmup: int = 3):
     import torch
     from qwen_triton_b200 import StepEntry
@@ -850,6 +956,8 @@ def run_workload(args) -> dict:
         return run_regupel_layers(args)
     if args.workload == "misudra-layers":
         return run_misudra_layers(args)
+    if args.workload == "bizurax-layers":
+        return run_bizurax_layers(args)
     import torch
 
     from qwen_triton_b200 import QwenB200ForCausalLM, StepEntry, load_preset
