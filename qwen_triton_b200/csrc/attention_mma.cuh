@@ -654,7 +654,8 @@ __global__ void __launch_bounds__(32 * WS_MAX_WARPS) attention_decode_ws_kernel(
     }
 }
 
-// One block per (sequence, head): out = sum_s acc_s e^{m_s - m} / sum_s l_s e^{m_s - m}; empty splits have m = -inf.
+// blockIdx.x is the (sequence, head), blockIdx.y a share of its columns: out = sum_s acc_s e^{m_s - m} / sum_s l_s e^{m_s - m};
+// empty splits have m = -inf.
 __global__ void attention_combine_mma_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                              __nv_bfloat16* __restrict__ out, int n_splits, int d, int sink,
                                              const float* __restrict__ sinks, int nq) {
@@ -687,10 +688,10 @@ __global__ void attention_combine_mma_kernel(const float* __restrict__ part_acc,
         l_all = l_all * factor + __expf(score - top);
     }
     const float* acc = part_acc + item * n_splits * d;
-    for (int c = threadIdx.x; c < d; c += blockDim.x) {
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < d; c += gridDim.y * blockDim.x) {
         float a = 0.f;
         if (kept) {                                                  // the loads do not wait for one another; an empty range's
-#pragma unroll 8                                                     // sums are read and dropped
+#pragma unroll 16                                                    // sums are read and dropped
             for (int s = 0; s < n_splits; ++s) {
                 const float v = acc[(size_t)s * d + c], f = factors[s];
                 a += f != 0.f ? v * f : 0.f;

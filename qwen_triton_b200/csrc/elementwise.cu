@@ -706,7 +706,8 @@ __global__ void __launch_bounds__(128) qk_norm_rope_pairs_kernel(const QkvParams
         if (is_q) dst = (TO*)p.q_out + ((size_t)t * p.nq + head) * p.d;
         else if (is_k) dst = (TO*)p.k_cache + cache_row + (size_t)(head - p.nq) * head_stride;
         else dst = (TO*)p.v_cache + cache_row + (size_t)(head - p.nq - p.nkv) * head_stride;
-        const bool normed = is_q ? p.q_weight != nullptr : (is_k && p.k_weight != nullptr);
+        const bool weighted = is_q ? p.q_weight != nullptr : (is_k && p.k_weight != nullptr);
+        const bool normed = weighted || (p.unit_norm && (is_q || is_k));
         float inv = 1.f;
         if (normed) {
             float sq = 0.f;
@@ -720,7 +721,10 @@ __global__ void __launch_bounds__(128) qk_norm_rope_pairs_kernel(const QkvParams
         for (int it = 0; it < IT; ++it) {
             const int j = (it * 32 + lane) * E;
             Piece<E> a = lo[hh][it], b = hi[hh][it];
-            if (normed) {
+            if (normed && !weighted) {
+#pragma unroll
+                for (int e = 0; e < E; ++e) { a.v[e] *= inv; b.v[e] *= inv; }
+            } else if (normed) {
 #pragma unroll
                 for (int e = 0; e < E; ++e) {
                     a.v[e] = a.v[e] * inv * (is_q ? wq_lo[it].v[e] : wk_lo[it].v[e]);
@@ -793,7 +797,7 @@ extern "C" int qt_qk_norm_rope_write(const void* qkv, int in_dtype, int n_splits
     const bool pair_aligned = split_stride % 2 == 0 && ((uintptr_t)qkv % 8 == 0) && ((uintptr_t)q_out % 8 == 0) && ((uintptr_t)cos_sin % 8 == 0) &&
                               (!q_weight || (uintptr_t)q_weight % 8 == 0) && (!k_weight || (uintptr_t)k_weight % 8 == 0) &&
                               (!write_kv || (((uintptr_t)k_cache % 8 == 0) && ((uintptr_t)v_cache % 8 == 0)));
-    if (pe && !own_values && !unit_norm && !whole_norm && !extra_cols && pair_aligned && n_tokens >= 256 && nq + 2 * nkv <= 65535 * 16 && (in_dtype == QT_F32 || in_dtype == QT_BF16) && out_dtype == QT_BF16) {
+    if (pe && !own_values && !(unit_norm && (q_weight || k_weight)) && !whole_norm && !extra_cols && pair_aligned && n_tokens >= 256 && nq + 2 * nkv <= 65535 * 16 && (in_dtype == QT_F32 || in_dtype == QT_BF16) && out_dtype == QT_BF16) {
         const int heads_total = nq + (kv_in_proj ? 2 * nkv : 0);
         const dim3 pgrid((unsigned)n_tokens, (unsigned)((heads_total + warps * HEADS_PER_WARP - 1) / (warps * HEADS_PER_WARP)));
 #define QT_LAUNCH_PAIRS(TI, E, IT) launch_kernel(qk_norm_rope_pairs_kernel<TI, __nv_bfloat16, E, IT>, pgrid, dim3(warps * 32), 0, s, p)

@@ -26,7 +26,7 @@ using namespace qt;
 
 constexpr int TILE = 128;      // weight rows (output columns) per tile
 
-enum Epilogue { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_SWIGLU = 2, EPI_QKV = 3 };
+enum Epilogue { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_SWIGLU = 2, EPI_QKV = 3, EPI_ACTIVATED = 4 };      // ACTIVATED: STORE with act(product)
 
 struct EpilogueParams {
     int M, N;
@@ -36,6 +36,7 @@ struct EpilogueParams {
     // STORE / SWIGLU
     void* out; int out_is_float; int act;      // act: the gate's activation, QT_ACT_*
     float limit;                               // of the capped gate (QT_ACT_CAPPED)
+    int activated;                             // STORE: act(product) is stored, not the product
     // RESIDUAL
     float* residual; const float* norm_w; __nv_bfloat16* xw; float* sq_out;
     // QKV
@@ -139,6 +140,10 @@ __device__ __forceinline__ void finish(const EpilogueParams& p, const Operands& 
             if (n + 2 < n_rows) v.z += p.bias[n + 2];
             if (n + 3 < n_rows) v.w += p.bias[n + 3];
         }
+        if (p.activated) {
+            v.x = gate_activation<true>(v.x, p.act); v.y = gate_activation<true>(v.y, p.act);
+            v.z = gate_activation<true>(v.z, p.act); v.w = gate_activation<true>(v.w, p.act);
+        }
         const float e[4] = {v.x, v.y, v.z, v.w};
         if (p.out_is_float) {
             float* dst = (float*)p.out + (size_t)m * n_rows + n;
@@ -206,6 +211,7 @@ inline int check_epilogue(const char* who, int epilogue, const EpilogueParams& p
         case EPI_STORE:
             QT_REQUIRE(p.out != nullptr && (out_dtype == QT_F32 || out_dtype == QT_BF16), "%s: the store epilogue needs a float or bfloat16 output", who);
             QT_REQUIRE((uintptr_t)p.out % 16 == 0, "%s: the output must be 16-byte aligned", who);
+            QT_REQUIRE(!p.activated || (p.act >= 0 && p.act < QT_ACT_COUNT), "%s: unknown activation code %d", who, p.act);
             break;
         case EPI_RESIDUAL:
             QT_REQUIRE(p.residual != nullptr && p.N % 4 == 0 && (uintptr_t)p.residual % 16 == 0, "%s: the residual epilogue needs an aligned stream whose width is a multiple of 4 (N=%d)", who, p.N);

@@ -292,6 +292,8 @@ extern "C" int qt_gemm_fused(const void* x, const void* w, int M, int N, int K, 
     e.token_seq = token_seq; e.token_pos = token_pos; e.block_table = block_table; e.max_blocks = max_blocks;
     e.q_w = q_w; e.k_w = k_w; e.qk_eps = qk_eps; e.cos_sin = cos_sin; e.rotary_dim = rotary_dim; e.max_pos = max_pos;
     e.nq = nq; e.nkv = nkv; e.d = d; e.page_tokens = page_tokens; e.ring_tokens = ring_tokens; e.write_kv = write_kv; e.interleaved = interleaved;
+    e.activated = epilogue == EPI_ACTIVATED;
+    if (e.activated) epilogue = EPI_STORE;
     int rc = check_epilogue("gemm_fused", epilogue, e, out_dtype);
     if (rc) return rc;
     CUtensorMap map_w, map_x;

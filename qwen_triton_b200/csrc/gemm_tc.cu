@@ -41,11 +41,14 @@ __device__ __forceinline__ void tile_coords(int t, int w_tiles, int x_tiles, int
     x = r / width;
 }
 
+// What an epilogue does with the sums: store them; gate them (below); store an activation of them (bfloat16, one K range).
+constexpr int PLAIN = 0, GATED = 1, ACTIVATED = 2;
+
 // GATED: the weight's rows alternate 16 of a gate projection and 16 of an up projection; the 32 accumulator lanes of
 // an epilogue warp are then the gate rows (lanes 0..15) and the up rows (16..31) of the same 16 features, and the
 // kernel stores act(gate) * up, [M, N / 2] (one K range only).  Of every two tokens the lower lanes finish the first
 // and the upper lanes the second: one exchange gives each half the value it lacks, and all 32 lanes compute and store.
-template <int BX, typename TO, bool GATED>
+template <int BX, typename TO, int MODE>
 __global__ void __launch_bounds__(THREADS) gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w,
                                                           const __grid_constant__ CUtensorMap map_x, TO* __restrict__ out,
                                                           int M, int N, int kb_total, int kb_per_split,
@@ -144,7 +147,7 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_kernel(const __grid_constant_
             for (int c = 0; c < BX; c += 16) {
                 uint32_t v[16];
                 tmem_load16(tmem_base + ((uint32_t)(quarter * 32) << 16) + (uint32_t)c, v);
-                if (GATED) {
+                if (MODE == GATED) {
                     const int features = N >> 1, feature = ((n - lane) >> 1) + (lane & 15);
                     const bool upper = (lane & 16) != 0;
 #pragma unroll
@@ -160,7 +163,8 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_kernel(const __grid_constant_
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
                         const int m = x0 + c + j;
-                        if (m < M) dst[(size_t)m * N + n] = from_float<TO>(__uint_as_float(v[j]) + add);
+                        const float y = __uint_as_float(v[j]) + add;
+                        if (m < M) dst[(size_t)m * N + n] = from_float<TO>(MODE == ACTIVATED ? gate_activation<true>(y, act) : y);
                     }
                 }
             }
@@ -300,7 +304,7 @@ struct PairWork {
 constexpr int PAIR_SLOT_FLOATS = PAIR_X * PAIR_W;    // one pair's accumulator tile in the scratch of the last wave
 constexpr int PAIR_FLAGS = 8;                       // per pair: one word per epilogue warp of its two blocks
 
-// SWIGLU: the weight's rows alternate 16 of a gate projection and 16 of an up projection (see swiglu in
+// GATED: the weight's rows alternate 16 of a gate projection and 16 of an up projection (see swiglu in
 // elementwise.cu); 32 accumulator columns of a token are then the gate and up values of 16 features, and the kernel
 // stores act(gate) * up, [M, N / 2], instead of the product itself.
 constexpr int SWIGLU_GROUP = 16;
@@ -320,7 +324,7 @@ template <> __device__ __forceinline__ void store8<__nv_bfloat16>(__nv_bfloat16*
     *reinterpret_cast<uint4*>(dst) = packed;
 }
 
-template <typename TO, bool SWIGLU>
+template <typename TO, int MODE>
 __global__ void __launch_bounds__(THREADS, 1) gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w,
                                                                   const __grid_constant__ CUtensorMap map_x, TO* __restrict__ out,
                                                                   int M, int N, int kb_total, int kb_per_split, int splits,
@@ -527,7 +531,7 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_tc_pair_kernel(const __grid_c
             const int m = x_tile * PAIR_X + slot_row;
             const int n0 = w_tile * PAIR_W;
             TO* __restrict__ plane = out + (size_t)item.split * split_stride;
-            TO* __restrict__ row = SWIGLU ? plane + (size_t)m * features + (n0 >> 1) : plane + (size_t)m * N + n0;
+            TO* __restrict__ row = MODE == GATED ? plane + (size_t)m * features + (n0 >> 1) : plane + (size_t)m * N + n0;
 #pragma unroll 1
             for (int c = 0; c < PAIR_W; c += 32) {
                 if (n0 + c >= N) break;
@@ -539,7 +543,7 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_tc_pair_kernel(const __grid_c
 #pragma unroll
                     for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(__uint_as_float(v[j]) + (n0 + c + j < N ? __ldg(bias + n0 + c + j) : 0.f));
                 }
-                if (SWIGLU) {
+                if (MODE == GATED) {
                     // columns c .. c + 15 are the gate rows of 16 features, c + 16 .. c + 31 the up rows of the same
                     const int f0 = (n0 + c) >> 1;
                     TO* dst = row + (c >> 1);
@@ -562,7 +566,10 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_tc_pair_kernel(const __grid_c
                     for (int h = 0; h < 4; ++h) {
                         float f[8];
 #pragma unroll
-                        for (int j = 0; j < 8; ++j) f[j] = __uint_as_float(v[8 * h + j]);
+                        for (int j = 0; j < 8; ++j) {
+                            const float y = __uint_as_float(v[8 * h + j]);
+                            f[j] = MODE == ACTIVATED ? gate_activation<true>(y, act) : y;
+                        }
                         if (vector_stores && n0 + c + 8 * h + 8 <= N) {
                             store8<TO>(row + c + 8 * h, f);
                         } else {
@@ -620,14 +627,14 @@ int pick_tail_tiles(long long n_tiles, int pairs, int kb_total, int tail, int ta
     return (whole - last_wave >= 3.0 && n_tiles > pairs) ? rest : 0;
 }
 
-template <typename TO, bool SWIGLU>
+template <typename TO, int MODE>
 int launch_pair(const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int M, int N, int kb_total, int splits,
                 size_t split_stride, int act, float limit, int tail, float* tail_scratch, int* tail_flags, int tail_pairs, const float* bias, int* status,
                 cudaStream_t stream) {
     const size_t smem = (size_t)PAIR_STAGES * PAIR_STAGE_BYTES + 1024 + (2 * PAIR_STAGES + 5) * 8 + 16;
     static int resident_pairs = 0;                           // pairs the device runs at once (one per TPC that can host a cluster)
     if (resident_pairs == 0) {
-        cudaError_t err = cudaFuncSetAttribute(gemm_tc_pair_kernel<TO, SWIGLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        cudaError_t err = cudaFuncSetAttribute(gemm_tc_pair_kernel<TO, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
         if (err != cudaSuccess) QT_FAIL(QT_ERR_LAUNCH, "gemm_tc_pair: cannot raise shared memory: %s", cudaGetErrorString(err));
         cudaLaunchConfig_t config = {};
         config.gridDim = dim3(2 * (unsigned)sm_count());
@@ -641,7 +648,7 @@ int launch_pair(const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int
         config.attrs = attribute;
         config.numAttrs = 1;
         int clusters = 0;
-        err = cudaOccupancyMaxActiveClusters(&clusters, gemm_tc_pair_kernel<TO, SWIGLU>, &config);
+        err = cudaOccupancyMaxActiveClusters(&clusters, gemm_tc_pair_kernel<TO, MODE>, &config);
         if (err != cudaSuccess || clusters < 1)
             QT_FAIL(QT_ERR_LAUNCH, "gemm_tc_pair: no cluster of two blocks fits the device (%s)", cudaGetErrorString(err));
         resident_pairs = clusters;
@@ -652,16 +659,16 @@ int launch_pair(const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int
     const int tail_tiles = splits == 1 && tail_scratch && tail_flags ? pick_tail_tiles(items, resident_pairs, kb_total, tail, tail_pairs) : 0;
     if (tail_tiles) pairs = (unsigned)resident_pairs;        // fewer tiles than pairs: all of them by K ranges over every pair
     // 16-byte stores need every output row (and plane) to start on a 16-byte boundary
-    const int per16 = 16 / (int)sizeof(TO), row_elems = SWIGLU ? N / 2 : N;
+    const int per16 = 16 / (int)sizeof(TO), row_elems = MODE == GATED ? N / 2 : N;
     const int vector_stores = ((uintptr_t)out % 16 == 0 && row_elems % per16 == 0 && split_stride % per16 == 0) ? 1 : 0;
-    launch_kernel_cluster(gemm_tc_pair_kernel<TO, SWIGLU>, dim3(2 * pairs), dim3(THREADS), smem, stream, 2, map_w, map_x, out, M, N, kb_total,
+    launch_kernel_cluster(gemm_tc_pair_kernel<TO, MODE>, dim3(2 * pairs), dim3(THREADS), smem, stream, 2, map_w, map_x, out, M, N, kb_total,
                           kb_per_split, splits, split_stride, act, limit, vector_stores, tail_tiles, tail_scratch, tail_flags, bias, status);
     QT_CHECK_LAUNCH("gemm_tc_pair");
     return QT_OK;
 }
 
 // ----------------------------------------------------------------------------- host side
-template <int BX, typename TO, bool GATED>
+template <int BX, typename TO, int MODE>
 int launch(const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int M, int N, int kb_total, int splits,
            size_t split_stride, int stages, int act, float limit, const float* bias, int* status, cudaStream_t stream) {
     constexpr uint32_t STAGE_BYTES = W_BYTES + BX * BK * 2;
@@ -682,27 +689,27 @@ int launch(const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int M, i
     const size_t smem = (size_t)stages * STAGE_BYTES + 1024 + (2 * stages + 1) * 8 + 16;
     static bool configured = false;
     if (!configured) {
-        cudaError_t err = cudaFuncSetAttribute(gemm_tc_kernel<BX, TO, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        cudaError_t err = cudaFuncSetAttribute(gemm_tc_kernel<BX, TO, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
         if (err != cudaSuccess) QT_FAIL(QT_ERR_LAUNCH, "gemm_tc: cannot raise shared memory: %s", cudaGetErrorString(err));
         configured = true;
     }
     const int kb_per_split = (kb_total + splits - 1) / splits;
     dim3 grid(((N + BW - 1) / BW) * ((M + BX - 1) / BX), 1, splits);
-    launch_kernel(gemm_tc_kernel<BX, TO, GATED>, dim3(grid), dim3(THREADS), smem, stream, map_w, map_x, out, M, N, kb_total, kb_per_split, split_stride, stages, act, limit, bias, status);
+    launch_kernel(gemm_tc_kernel<BX, TO, MODE>, dim3(grid), dim3(THREADS), smem, stream, map_w, map_x, out, M, N, kb_total, kb_per_split, split_stride, stages, act, limit, bias, status);
     QT_CHECK_LAUNCH("gemm_tc");
     return QT_OK;
 }
 
 
-template <typename TO, bool GATED>
+template <typename TO, int MODE>
 int dispatch_tile(int bx, const CUtensorMap& map_w, const CUtensorMap& map_x, TO* out, int M, int N, int kb_total, int splits,
                   size_t split_stride, int stages, int act, float limit, const float* bias, int* status, cudaStream_t stream) {
     switch (bx) {
-        case 16: return launch<16, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
-        case 32: return launch<32, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
-        case 64: return launch<64, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
-        case 128: return launch<128, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
-        case 256: return launch<256, TO, GATED>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
+        case 16: return launch<16, TO, MODE>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
+        case 32: return launch<32, TO, MODE>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
+        case 64: return launch<64, TO, MODE>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
+        case 128: return launch<128, TO, MODE>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
+        case 256: return launch<256, TO, MODE>(map_w, map_x, out, M, N, kb_total, splits, split_stride, stages, act, limit, bias, status, stream);
     }
     QT_FAIL(QT_ERR_ARG, "gemm_tc: token tile %d is not one of 16, 32, 64, 128, 256", bx);
 }
@@ -716,11 +723,13 @@ int dispatch_tile(int bx, const CUtensorMap& map_w, const CUtensorMap& map_x, TO
 // `stages` > 0 overrides the depth of the shared-memory ring (a tuning knob; 0 picks the default).
 // `bias` (or null): [N] float, added to the sums (to the first plane of split sums; ahead of the gate).
 // With `gated` the weight's rows alternate 16 of a gate and 16 of an up projection and `out` is [M, N / 2] bfloat16 =
-// act(gate) * up (`act`: one of QT_ACT_*; one K range only).
+// act(gate) * up (`act`: one of QT_ACT_*; one K range only).  `gated` 2: `out` [M, N] bfloat16 = act(product), one K range.
 extern "C" int qt_gemm_tc(const void* x, const void* w, void* out, int out_dtype, int M, int N, int K, int token_tile,
                           int splits, long long split_stride, int stages, int gated, int act, float limit, const float* bias, int* status,
                           void* stream) {
-    QT_REQUIRE(!gated || (splits == 1 && out_dtype == QT_BF16 && N % 32 == 0 && act >= 0 && act <= QT_ACT_CAPPED),
+    QT_REQUIRE(gated >= PLAIN && gated <= ACTIVATED && (gated != ACTIVATED || (splits == 1 && out_dtype == QT_BF16 && act >= 0 && act < QT_ACT_COUNT)),
+               "gemm_tc: an activation on the product writes bfloat16 from one K range (splits=%d, activation %d)", splits, act);
+    QT_REQUIRE(gated != GATED || (splits == 1 && out_dtype == QT_BF16 && N % 32 == 0 && act >= 0 && act <= QT_ACT_CAPPED),
                "gemm_tc: the gated epilogue writes bfloat16 from one K range of gate and up rows in groups of 16 (N=%d, splits=%d)", N, splits);
     QT_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_tc: bad sizes M=%d N=%d K=%d", M, N, K);
     QT_REQUIRE(K % 8 == 0, "gemm_tc: K=%d must be a multiple of 8 (rows must start on 16-byte boundaries for TMA)", K);
@@ -738,18 +747,20 @@ extern "C" int qt_gemm_tc(const void* x, const void* w, void* out, int out_dtype
     rc = tensor_map(&map_x, x, (uint64_t)M, (uint64_t)K, (uint32_t)token_tile);
     if (rc) return rc;
     cudaStream_t s = (cudaStream_t)stream;
-    if (gated)
-        return dispatch_tile<__nv_bfloat16, true>(token_tile, map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, stages, act, limit, bias, status, s);
+    if (gated == GATED)
+        return dispatch_tile<__nv_bfloat16, GATED>(token_tile, map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, stages, act, limit, bias, status, s);
+    if (gated == ACTIVATED)
+        return dispatch_tile<__nv_bfloat16, ACTIVATED>(token_tile, map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, stages, act, 0.f, bias, status, s);
     if (out_dtype == QT_BF16)
-        return dispatch_tile<__nv_bfloat16, false>(token_tile, map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, splits, (size_t)split_stride, stages, 0, 0.f, bias, status, s);
+        return dispatch_tile<__nv_bfloat16, PLAIN>(token_tile, map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, splits, (size_t)split_stride, stages, 0, 0.f, bias, status, s);
     if (out_dtype == QT_F32)
-        return dispatch_tile<float, false>(token_tile, map_w, map_x, (float*)out, M, N, kb_total, splits, (size_t)split_stride, stages, 0, 0.f, bias, status, s);
+        return dispatch_tile<float, PLAIN>(token_tile, map_w, map_x, (float*)out, M, N, kb_total, splits, (size_t)split_stride, stages, 0, 0.f, bias, status, s);
     QT_FAIL(QT_ERR_ARG, "gemm_tc: unknown output type %d", out_dtype);
 }
 
 // The same product by pairs of blocks (see gemm_tc_pair_kernel): bfloat16 or float output, meant for many tokens (a
 // pair covers 256 weight rows x 256 tokens); out[splits, M, N] in float when `splits` > 1, under the rule above.  With `swiglu` the weight's rows alternate 16 of a gate and
-// 16 of an up projection and `out` is [M, N / 2] = act(gate) * up (`act`: one of QT_ACT_*).  Codes in `status`: as above, 4 = the MMA issuer
+// 16 of an up projection and `out` is [M, N / 2] = act(gate) * up (`act`: one of QT_ACT_*); `swiglu` 2: `out` [M, N] = act(product).  Codes in `status`: as above, 4 = the MMA issuer
 // waiting for the epilogues to free an accumulator.
 // `tail`: 0 = every tile by one pair; -1 = the last wave's tiles by K ranges where that pays; 1 = wherever the tiles do
 // not divide by the pairs.  It needs `tail_scratch` (tail_pairs x 256 x 256 floats) and `tail_flags` (tail_pairs x 8
@@ -764,7 +775,8 @@ extern "C" int qt_gemm_tc_pair(const void* x, const void* w, void* out, int out_
     QT_REQUIRE(K % 8 == 0, "gemm_tc_pair: K=%d must be a multiple of 8 (rows must start on 16-byte boundaries for TMA)", K);
     QT_REQUIRE(((uintptr_t)x % 16 == 0) && ((uintptr_t)w % 16 == 0), "gemm_tc_pair: operands must be 16-byte aligned");
     QT_REQUIRE(status != nullptr, "gemm_tc_pair: a status word is required");
-    QT_REQUIRE(!swiglu || N % (2 * SWIGLU_GROUP) == 0, "gemm_tc_pair: N=%d is not gate and up rows in groups of %d", N, SWIGLU_GROUP);
+    QT_REQUIRE(swiglu >= PLAIN && swiglu <= ACTIVATED && (swiglu != ACTIVATED || act < QT_ACT_COUNT), "gemm_tc_pair: activation %d on mode %d", act, swiglu);
+    QT_REQUIRE(swiglu != GATED || N % (2 * SWIGLU_GROUP) == 0, "gemm_tc_pair: N=%d is not gate and up rows in groups of %d", N, SWIGLU_GROUP);
     const int kb_total = (K + BK - 1) / BK;
     QT_REQUIRE(splits >= 1 && splits <= kb_total, "gemm_tc_pair: splits=%d for %d K blocks", splits, kb_total);
     QT_REQUIRE((splits - 1) * ((kb_total + splits - 1) / splits) < kb_total, "gemm_tc_pair: splits=%d would leave a split without K blocks (%d blocks)", splits, kb_total);
@@ -776,9 +788,11 @@ extern "C" int qt_gemm_tc_pair(const void* x, const void* w, void* out, int out_
     rc = tensor_map(&map_x, x, (uint64_t)M, (uint64_t)K, (uint32_t)PAIR_HALF);
     if (rc) return rc;
     cudaStream_t s = (cudaStream_t)stream;
-    if (out_dtype == QT_BF16 && swiglu) return launch_pair<__nv_bfloat16, true>(map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, act, limit, tail, tail_scratch, tail_flags, tail_pairs, bias, status, s);
-    if (out_dtype == QT_BF16) return launch_pair<__nv_bfloat16, false>(map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, 0, 0.f, tail, tail_scratch, tail_flags, tail_pairs, bias, status, s);
-    if (out_dtype == QT_F32 && !swiglu) return launch_pair<float, false>(map_w, map_x, (float*)out, M, N, kb_total, splits, (size_t)split_stride, 0, 0.f, tail, tail_scratch, tail_flags, tail_pairs, bias, status, s);
+    if (out_dtype == QT_BF16 && swiglu == ACTIVATED)
+        return launch_pair<__nv_bfloat16, ACTIVATED>(map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, act, 0.f, tail, tail_scratch, tail_flags, tail_pairs, bias, status, s);
+    if (out_dtype == QT_BF16 && swiglu) return launch_pair<__nv_bfloat16, GATED>(map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, act, limit, tail, tail_scratch, tail_flags, tail_pairs, bias, status, s);
+    if (out_dtype == QT_BF16) return launch_pair<__nv_bfloat16, PLAIN>(map_w, map_x, (__nv_bfloat16*)out, M, N, kb_total, 1, 0, 0, 0.f, tail, tail_scratch, tail_flags, tail_pairs, bias, status, s);
+    if (out_dtype == QT_F32 && !swiglu) return launch_pair<float, PLAIN>(map_w, map_x, (float*)out, M, N, kb_total, splits, (size_t)split_stride, 0, 0.f, tail, tail_scratch, tail_flags, tail_pairs, bias, status, s);
     QT_FAIL(QT_ERR_ARG, "gemm_tc_pair: output type %d%s is not offered", out_dtype, swiglu ? " with the SiLU-gated epilogue" : "");
 }
 

@@ -1465,19 +1465,21 @@ def gemm_tc_supported(a: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: GemmOut, token_tile: int | None = None, stages: int = 0,
-            swiglu: bool = False, activation: str = "silu", limit: float = 0.0, bias: torch.Tensor | None = None) -> None:
+            swiglu: bool = False, activation: str = "silu", limit: float = 0.0, bias: torch.Tensor | None = None, activate: bool = False) -> None:
     """out = a [M, K] @ w [N, K]^T on the tcgen05 tensor cores; bfloat16 inputs, K a multiple of 8.
 
     ``out`` is [1, M, N] bfloat16 or float, or [splits, M, N] float for split-K partial sums.  With ``swiglu`` the
     rows of ``w`` alternate SWIGLU_GROUP of a gate and of an up projection and ``out`` [1, M, N / 2] (bfloat16)
     receives act(gate) * up from the epilogue.  ``bias`` [N] (float) is added to the sums (ahead of the gate).
+    With ``activate`` (and no gate) ``out`` [1, M, N] (bfloat16) receives act(product).
     """
     _need(a, "a", torch.bfloat16)
     _need(w, "w", torch.bfloat16)
     rows, k = a.shape
     cols = w.shape[0] // 2 if swiglu else w.shape[0]
     if k != w.shape[1] or (out.rows, out.cols) != (rows, cols) or (swiglu and (out.n_splits != 1 or w.shape[0] % (2 * SWIGLU_GROUP)
-                                                                                   or out.tensor.dtype != torch.bfloat16)):
+                                                                                   or out.tensor.dtype != torch.bfloat16)) \
+            or (activate and (swiglu or out.n_splits != 1 or out.tensor.dtype != torch.bfloat16)):
         raise KernelError(f"gemm: a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.tensor.shape)} do not fit")
     if rows == 0:
         return
@@ -1485,7 +1487,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: GemmOut, token_tile: int | No
         raise KernelError("gemm_tc: the output must be a bfloat16 or float32 CUDA tensor")
     tile = token_tile or tc_token_tile(rows)
     _call("gemm_tc", "qt_gemm_tc", _ptr(a), _ptr(w), _ptr(out.tensor), _code(out.tensor, "out"), rows, w.shape[0], k, tile,
-          out.n_splits, out.split_stride, int(stages), 1 if swiglu else 0, activation_code(activation, True) if swiglu else 0,
+          out.n_splits, out.split_stride, int(stages), 1 if swiglu else 2 if activate else 0, activation_code(activation, swiglu) if swiglu or activate else 0,
           float(limit), _ptr(_product_bias(bias, w)), _ptr(_status_word(a.device)), _stream())
 
 
@@ -1520,7 +1522,7 @@ def pair_tail_mode() -> int:
 
 
 def gemm_tc_pair(a: torch.Tensor, w: torch.Tensor, out: GemmOut, swiglu: bool = False, activation: str = "silu",
-                 tail: int | None = None, limit: float = 0.0, bias: torch.Tensor | None = None) -> None:
+                 tail: int | None = None, limit: float = 0.0, bias: torch.Tensor | None = None, activate: bool = False) -> None:
     """The same product by pairs of blocks on the two SMs of a TPC (tcgen05 cta_group::2): 256 weight rows x
     256 tokens per tile, each block staging half of both operands; one persistent pair per TPC with two
     accumulators in tensor memory.  Meant for many tokens; ``out`` may be [splits, M, N] float partial sums, which
@@ -1528,12 +1530,13 @@ def gemm_tc_pair(a: torch.Tensor, w: torch.Tensor, out: GemmOut, swiglu: bool = 
 
     With ``swiglu`` the rows of ``w`` alternate SWIGLU_GROUP of a gate and of an up projection
     (``interleave_gate_up``) and ``out`` [1, M, N / 2] receives act(gate) * up from the epilogue.  ``bias`` [N] (float) is
-    added to the sums (ahead of the gate)."""
+    added to the sums (ahead of the gate).  With ``activate`` (and no gate) ``out`` [1, M, N] (bfloat16) receives act(product)."""
     _need(a, "a", torch.bfloat16)
     _need(w, "w", torch.bfloat16)
     rows, k = a.shape
     cols = w.shape[0] // 2 if swiglu else w.shape[0]
-    if k != w.shape[1] or (out.rows, out.cols) != (rows, cols) or (swiglu and (out.n_splits != 1 or w.shape[0] % (2 * SWIGLU_GROUP))):
+    if k != w.shape[1] or (out.rows, out.cols) != (rows, cols) or (swiglu and (out.n_splits != 1 or w.shape[0] % (2 * SWIGLU_GROUP))) \
+            or (activate and (swiglu or out.n_splits != 1 or out.tensor.dtype != torch.bfloat16)):
         raise KernelError(f"gemm: a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.tensor.shape)} do not fit")
     if rows == 0:
         return
@@ -1542,7 +1545,7 @@ def gemm_tc_pair(a: torch.Tensor, w: torch.Tensor, out: GemmOut, swiglu: bool = 
     tail = pair_tail_mode() if tail is None else int(tail)
     slots, flags, pairs = _pair_tail(a.device) if tail != 0 and out.n_splits == 1 else (None, None, 0)
     _call("gemm_tc", "qt_gemm_tc_pair", _ptr(a), _ptr(w), _ptr(out.tensor), _code(out.tensor, "out"), rows, w.shape[0], k,
-          1 if swiglu else 0, activation_code(activation, True) if swiglu else 0, float(limit), out.n_splits, out.split_stride,
+          1 if swiglu else 2 if activate else 0, activation_code(activation, swiglu) if swiglu or activate else 0, float(limit), out.n_splits, out.split_stride,
           tail, _ptr(slots) if slots is not None else None, _ptr(flags) if flags is not None else None, pairs,
           _ptr(_product_bias(bias, w)), _ptr(_status_word(a.device)), _stream())
 
@@ -1575,7 +1578,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: GemmOut, bias: torch.Tensor | No
 # ----------------------------------------------------------------------------- products of a decode step, fused
 FUSED_MAX_ROWS = 128        # most tokens the fused product takes (one token tile per block)
 FUSED_MAX_SPLITS = 8        # blocks of a cluster that share a weight tile
-_EPI_STORE, _EPI_RESIDUAL, _EPI_SWIGLU, _EPI_QKV = 0, 1, 2, 3
+_EPI_STORE, _EPI_RESIDUAL, _EPI_SWIGLU, _EPI_QKV, _EPI_ACTIVATED = 0, 1, 2, 3, 4
 
 
 def fused_enabled(role: str) -> bool:
@@ -1644,10 +1647,13 @@ def _fused(x, w: torch.Tensor, splits: int, epilogue: int, *, out=None, residual
           1 if interleaved else 0, _ptr(_status_word(a.device)), _stream())
 
 
-def gemm_fused_store(x, w: torch.Tensor, out: torch.Tensor, splits: int = 1, stages: int = 0, bias: torch.Tensor | None = None) -> None:
-    """out [M, N] (float or bfloat16) = x w^T (+ ``bias``, float), times the rows' deferred norm factor if ``x`` is ``ScaledRows``."""
+def gemm_fused_store(x, w: torch.Tensor, out: torch.Tensor, splits: int = 1, stages: int = 0, bias: torch.Tensor | None = None,
+                     activation: str | None = None) -> None:
+    """out [M, N] (float or bfloat16) = x w^T (+ ``bias``, float), times the rows' deferred norm factor if ``x`` is ``ScaledRows``;
+    with ``activation`` that function of it."""
     _need(out, "out", shape=(x.shape[0], w.shape[0]))
-    _fused(x, w, splits, _EPI_STORE, out=out, stages=stages, bias=bias)
+    _fused(x, w, splits, _EPI_STORE if activation is None else _EPI_ACTIVATED, out=out, stages=stages, bias=bias,
+           act=0 if activation is None else activation_code(activation))
 
 
 def gemm_fused_residual(x, w: torch.Tensor, residual: torch.Tensor, norm_weight: torch.Tensor | None = None,

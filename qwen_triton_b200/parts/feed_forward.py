@@ -108,7 +108,8 @@ class PlainMLP:
 
     Parameters: ``hidden_size``, ``intermediate_size``, ``activation`` (one of ``kernels.ACTIVATIONS``, default the exact
     GELU), the tensor-name pieces ``up``, ``down``, ``weight_suffix`` (default ".weight"), ``float_out`` (the down
-    projection hands on float sums) and ``buffers``.  The activation is taken on the up product's sums in float."""
+    projection hands on float sums) and ``buffers``.  The activation is taken on the up product's sums in float, in that product's
+    epilogue where it is not cut over K (or is, on the chip: few tokens), else by a kernel behind it."""
 
     graph_safe = True
 
@@ -123,8 +124,9 @@ class PlainMLP:
         self.names = self._names(params)
         float_out = bool(params.get("float_out", False))
         key = str(params.get("buffers", "mlp"))
-        self.up = Linear(f"{key}.up.plain", self.inter, self.hidden, runtime)
-        self.down = Linear(f"{key}.down" + (".float" if float_out else ""), self.hidden, self.inter, runtime, float_out=float_out)
+        self.up = Linear(f"{key}.up.plain", self.inter, self.hidden, runtime, role="gate")
+        self.down = Linear(f"{key}.down" + (".float" if float_out else ""), self.hidden, self.inter, runtime, role="mlp_out", float_out=float_out)
+        self.takes_scaled_rows = self.up.fused_capable
         self.act_buffer = f"{key}.act"
         runtime.workspace.declare(self.act_buffer, runtime.max_step_tokens * self.inter, runtime.dtype)
 
@@ -149,8 +151,16 @@ class PlainMLP:
     def forward(self, x, ctx):
         tokens = x.shape[0]
         act = self.runtime.workspace.view(self.act_buffer, tokens, self.inter)
-        kernels.activation(self.up(x), act, self.activation)
-        return self.down(act)
+        if self.up.fusable(tokens):
+            self.up.into_activation(x, act, self.activation)
+        elif act.dtype == torch.bfloat16 and kernels.gemm_uses_pairs(x, self.up.weight):
+            kernels.gemm_tc_pair(x, self.up.weight, GemmOut(act.view(1, tokens, self.inter)), activate=True, activation=self.activation)
+        elif act.dtype == torch.bfloat16 and kernels.gemm_tc_supported(x, self.up.weight) and self.up.plan_splits(tokens) == 1:
+            kernels.gemm_tc(x, self.up.weight, GemmOut(act.view(1, tokens, self.inter)), activate=True, activation=self.activation)
+        else:
+            kernels.activation(self.up(x), act, self.activation)
+        # few tokens: left to the norm behind it
+        return DeferredProduct(self.down, act) if self.down.fusable(tokens) else self.down(act)
 
 
 # Most (token, expert) pairs that run as matrix-vector passes, each streaming its expert's rows once: up to two pairs

@@ -39,6 +39,9 @@ from .base import DeferredProduct, KVRequest, Runtime, part_class, register_mixe
 from .linear import Linear
 
 
+_MANY_TOKENS = 256       # steps of more tokens form the queries and the cache rows in products of their own (without a query latent)
+
+
 @register_mixer("latent_attention")
 class LatentAttention:
     graph_safe = True
@@ -67,6 +70,12 @@ class LatentAttention:
         self.proj_rows = -(-used // 8) * 8
         self.proj = Linear("latent.proj" + ("" if self.own_kv else ".reader"), self.proj_rows, self.hidden, runtime, float_out=True, role="qkv")
         self.takes_scaled_rows = self.proj.fused_capable
+        # Many tokens without a query latent: the queries are most of the first product's columns, and what reads them rounds them to
+        # the activation type anyway, so they are a product of their own that hands them on in it (over the same weight rows).
+        self.many = None
+        if not self.q_rank and runtime.dtype == torch.bfloat16 and self.hidden % 8 == 0 and runtime.max_step_tokens > _MANY_TOKENS and self.proj_rows > self.at_kv:
+            self.many = (Linear("latent.queries", self.at_kv, self.hidden, runtime),
+                         Linear("latent.rows", self.proj_rows - self.at_kv, self.hidden, runtime, float_out=True))
         self.uq = Linear("latent.uq", self.heads * (self.d + self.rot), self.q_rank, runtime) if self.q_rank else None
         float_out = bool(params.get("float_out", False))
         self.o = Linear("latent.o" + (".float" if float_out else ""), self.hidden, self.heads * self.dv, runtime, float_out=float_out, role="attn_out")
@@ -131,6 +140,8 @@ class LatentAttention:
         if self.proj_rows > used:
             rows.append(torch.zeros(self.proj_rows - used, self.hidden, dtype=dtype, device=rows[0].device))
         self.proj.set_weight(torch.cat(rows, dim=0))
+        if self.many is not None:
+            self.many[0].weight, self.many[1].weight = self.proj.weight[:self.at_kv], self.proj.weight[self.at_kv:]
         if self.q_rank:
             self.uq.set_weight(self._halves_order(source(n["uq"]), self.heads, self.d))
             self.q_norm = to_device(source(n["dq_norm"]), torch.float32, device)
@@ -176,13 +187,16 @@ class LatentAttention:
         if cache.k is None or cache.k.shape[-1] != self.row:
             raise ValueError(f"{self.prefix}: the cache rows it reads are not {self.rank} + {self.rot} elements long")
         table = ctx.block_table(cache.group)
-        proj = self.proj.finished(x)
+        own_queries = self.many is not None and tokens > _MANY_TOKENS
+        skipped = self.at_kv if own_queries else 0                              # columns that ``proj`` then lacks
+        proj = self.many[1](x) if own_queries else self.proj.finished(x)
         cq = ws.view("latent.cq", tokens, self.q_rank) if self.q_rank else None
         if cq is not None or write:
             kernels.latent_prepare(proj, self.q_norm, self.kv_norm, self.eps, self.cos_sin, cq, cache.k if write else None, ctx.token_seq,
                                    ctx.token_pos, table if write else None, self.rank, self.rot, cache.page_tokens, cache.ring_tokens, write_kv=write,
-                                   at_kv=self.at_kv)
-        q_full = self.uq(cq) if cq is not None else proj                        # [*, T, heads * (d + rot)], or with the first projection's other columns behind
+                                   at_kv=self.at_kv - skipped)
+        # [*, T, heads * (d + rot)], or with the first projection's other columns behind
+        q_full = self.uq(cq) if cq is not None else self.many[0](x) if own_queries else proj
         q = ws.view("latent.q", tokens, self.heads, self.row)
         kernels.head_product(q_full, self.uk_t, q, x_row=q_full.cols, x_head=self.d + self.rot)
         kernels.latent_query_rot(q_full, self.cos_sin, ctx.token_pos, q, self.heads, self.d, self.rot, self.rank)
@@ -196,7 +210,7 @@ class LatentAttention:
                                       cache.ring_tokens, self.window, self.scale, v_dim=self.rank)
         heads = ws.view("latent.heads", tokens, self.heads, self.dv)
         kernels.head_product(out, self.uv, heads, x_row=self.heads * self.rank, x_head=self.rank,
-                             gate=proj if self.gated else None, gate_offset=self.at_gate, gate_per_head=self.head_gate)
+                             gate=proj if self.gated else None, gate_offset=self.at_gate - skipped, gate_per_head=self.head_gate)
         heads = heads.view(tokens, self.heads * self.dv)
         # few tokens: the product is left to the block, whose next norm launches it with the residual addition in its epilogue
         return DeferredProduct(self.o, heads) if self.o.fusable(tokens) else self.o(heads)

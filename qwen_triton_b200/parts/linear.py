@@ -195,6 +195,11 @@ class Linear:
         kernels.gemm_fused_swiglu(x, self.weight, out, splits=self._fused_splits(x.shape[0]), stages=self._fused_stages(x.shape[0]),
                                   activation=activation, limit=limit, bias=bias)
 
+    def into_activation(self, x, out: torch.Tensor, activation: str) -> None:
+        """out = act(x W^T (+ bias)), the activation in the fused product's epilogue."""
+        kernels.gemm_fused_store(x, self.weight, out, splits=self._fused_splits(x.shape[0]), stages=self._fused_stages(x.shape[0]), bias=self._loaded_bias(),
+                                 activation=activation)
+
     def into_qkv(self, x, *args, **kwargs) -> None:
         kernels.gemm_fused_qkv(x, self.weight, *args, splits=self._fused_splits(x.shape[0]), stages=self._fused_stages(x.shape[0]), **kwargs)
 

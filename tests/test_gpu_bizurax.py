@@ -269,6 +269,26 @@ def test_squared_relu(dtype, rows, width):
     close(out, torch.relu(x.double().sum(0)).square(), dtype, "relu2")
 
 
+@pytest.mark.parametrize("activation, function", [("relu2", lambda z: torch.relu(z).square()), ("gelu", lambda z: 0.5 * z * (1 + torch.erf(z / math.sqrt(2.0))))])
+@pytest.mark.parametrize("rows", [1, 3, 16, 40, 300, 700])
+def test_an_activation_in_the_products_epilogues(rows, activation, function):
+    """Without a gate, in each tensor-core kernel; sizes whose last tiles are partial."""
+    torch.manual_seed(rows)
+    width, inter = 192, 172
+    x, w, b = torch.randn(rows, width).to(torch.bfloat16), (torch.randn(inter, width) * 0.1).to(torch.bfloat16), torch.randn(inter)
+    want = function(x.double() @ w.double().T + b.double())
+    out = torch.empty(rows, inter, dtype=torch.bfloat16, device=DEV)
+    for product in (kernels.gemm_tc, kernels.gemm_tc_pair):
+        out.fill_(float("nan"))
+        product(x.to(DEV), w.to(DEV), GemmOut(out.view(1, rows, inter)), activate=True, activation=activation, bias=b.to(DEV))
+        close(out, want, "bf16", product.__name__)
+    if rows <= 16:
+        out.fill_(float("nan"))
+        kernels.gemm_fused_store(x.to(DEV), w.to(DEV), out, splits=3, bias=b.to(DEV), activation=activation)
+        close(out, want, "bf16", "fused")
+    kernels.check_status(DEV)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("tokens", [3, 90, 400])
 def test_the_feed_forwards_alone(dtype, tokens):
