@@ -180,7 +180,8 @@ def attention_oracle(q, k, v, scale, softcap, sinks):
 @pytest.mark.parametrize("heads, kv_heads, d, dv, scale, softcap, unit, sink", [
     (4, 2, 64, 64, 0.11, 41.0, True, True), (4, 1, 128, 128, 0.25, 7.0, False, True), (6, 2, 128, 128, 0.0884, 15.0, True, True),
     (3, 3, 64, 64, 0.5, 2.0, False, False), (8, 2, 32, 32, 0.3, 12.0, True, True), (20, 1, 48, 48, 0.2, 3.0, False, True),
-    (2, 1, 40, 24, 0.4, 5.0, True, True), (4, 4, 10, 30, 0.7, 1.0, False, True), (4, 2, 64, 64, 0.2, None, False, True), (2, 2, 128, 128, 0.1, None, False, True)])
+    (2, 1, 40, 24, 0.4, 5.0, True, True), (4, 4, 10, 30, 0.7, 1.0, False, True), (4, 2, 64, 64, 0.2, None, False, True), (2, 2, 128, 128, 0.1, None, False, True), (4, 1, 96, 96, 0.15, 20.0, True, True),
+    (6, 3, 80, 80, 0.3, 4.0, False, True), (2, 1, 256, 256, 0.06, 9.0, False, True)])
 def test_attention_with_capped_scores_and_a_sink(dtype, heads, kv_heads, d, dv, scale, softcap, unit, sink):
     """300 positions over pages in no order: a prompt, a late portion of it, single tokens with several counts of key ranges.  Key
     5 is seen by every later query with a score far above all others (beyond the cap where queries and keys are not unit), and
@@ -200,7 +201,7 @@ def test_attention_with_capped_scores_and_a_sink(dtype, heads, kv_heads, d, dv, 
     k_pool, v_pool, table = paged(k, PAGE, order, store), paged(v, PAGE, order, store), as_int([order])
     on = dict(sinks=sinks.to(DEV) if sink else None, softcap=softcap)
     bound = d * scale if unit else None
-    tc = dtype == "bf16" and d == dv
+    tc = dtype == "bf16" and d == dv and d <= 128                # what the tensor-core kernels take, in steps of 16
     for begin in (0, 190, 298):
         for impl in [None, "generic"] + (["mma"] if tc and d % 16 == 0 else []) + (["tc"] if tc and d in (64, 128) else []):
             for known in {None, bound}:
