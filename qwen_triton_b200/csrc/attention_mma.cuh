@@ -691,7 +691,7 @@ __global__ void attention_combine_mma_kernel(const float* __restrict__ part_acc,
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < d; c += gridDim.y * blockDim.x) {
         float a = 0.f;
         if (kept) {                                                  // the loads do not wait for one another; an empty range's
-#pragma unroll 16                                                    // sums are read and dropped
+#pragma unroll 8                                                     // sums are read and dropped
             for (int s = 0; s < n_splits; ++s) {
                 const float v = acc[(size_t)s * d + c], f = factors[s];
                 a += f != 0.f ? v * f : 0.f;

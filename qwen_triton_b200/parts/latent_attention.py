@@ -76,6 +76,8 @@ class LatentAttention:
         if not self.q_rank and runtime.dtype == torch.bfloat16 and self.hidden % 8 == 0 and runtime.max_step_tokens > _MANY_TOKENS and self.proj_rows > self.at_kv:
             self.many = (Linear("latent.queries", self.at_kv, self.hidden, runtime),
                          Linear("latent.rows", self.proj_rows - self.at_kv, self.hidden, runtime, float_out=True))
+            # whole over K, or it would hand on float planes after all
+            self.many[0].split_plans = [(rows, splits) for rows, splits in self.many[0].split_plans if rows <= _MANY_TOKENS]
         self.uq = Linear("latent.uq", self.heads * (self.d + self.rot), self.q_rank, runtime) if self.q_rank else None
         float_out = bool(params.get("float_out", False))
         self.o = Linear("latent.o" + (".float" if float_out else ""), self.hidden, self.heads * self.dv, runtime, float_out=float_out, role="attn_out")
